@@ -48,6 +48,10 @@ extern "C" {
 #define LOOM_B200_ACT_RELU2 6
 #define LOOM_B200_ACT_LINEAR (-1)
 
+/* element types of float matrices */
+#define LOOM_B200_DTYPE_F32 0
+#define LOOM_B200_DTYPE_BF16 1
+
 typedef struct loom_b200_ctx loom_b200_ctx;       /* stands in for *poly.WGPUContext */
 typedef struct loom_b200_graph loom_b200_graph;   /* a recorded command buffer (one frame) */
 typedef struct loom_b200_weight loom_b200_weight; /* a packed ternary matrix resident in HBM:
@@ -106,6 +110,7 @@ void* loom_b200_ctx_stream(loom_b200_ctx* ctx);
  * and phase-trace code (1, default: +7 % decode tok/s) or the full kernels (0);
  * "tp_fused" 0/1 = row-parallel projections under the peer mailboxes as statistics kernel + GEMV + finalize kernel (0), or with the
  * exchange of the partial sums in the GEMV's epilogue (1, default);
+ * "dense_tc" 0/1 = token blocks of bf16 layer stacks run on the tensor cores (1, default) or as plain fused multiply-adds (0);
  * "prefill_gemm" 0/1 = prompts of 32 or more tokens
  * run their projections as token-block GEMMs on the tensor cores (1) or eight tokens at a time through the GEMV (0).  "gemm_cache" 0/1 = the token-block GEMM reads pre-expanded int8 codes (one byte per weight, built per
  * matrix the first time it meets the GEMM, four times its packed bytes; the device twin of ensureBitNetCodes,
@@ -378,6 +383,76 @@ int loom_b200_decoder_last_residual(loom_b200_decoder* dec, float* rows_host, in
  * {first-maximum token, forward it}.  The loop runs on the device; tokens come back once at the end. */
 int loom_b200_decoder_generate(loom_b200_decoder* dec, const int32_t* prompt, int n_prompt, int max_new,
                                int32_t* out_tokens, loom_b200_gen_metrics* metrics);
+
+/* ---- float matrices and layer stacks --------------------------------------------------------------
+ * No counterpart in the reference: decoders whose layers are described one by one -- a token mixer and a feed-forward,
+ * each with sizes and constants of its own -- over bf16 or float32 matrices.  They are loom_b200_decoder objects: forward,
+ * extend, generate, continue, select / step_batch / continue_batch, read_tokens and last_residual work on them as on the
+ * ternary decoder. */
+
+/* `groups` matrices of one shape [rows, cols] (the experts of a layer share one object; a plain matrix has one group),
+ * stored as bf16 or float32 in the blocked layout the kernels read.  put fills rows row0 .. row0+rows-1 of a group from
+ * row-major [rows, cols] values of either type (host memory, or device memory with src_on_device); rows that are never put
+ * are zero.  Stacking several projections of one input into one matrix is done with row0. */
+typedef struct loom_b200_matrix loom_b200_matrix;
+int loom_b200_matrix_create(loom_b200_ctx* ctx, int rows, int cols, int groups, int dtype, loom_b200_matrix** out);
+int loom_b200_matrix_put(loom_b200_ctx* ctx, loom_b200_matrix* m, int group, int row0, int rows, const void* src, int src_dtype,
+                         int src_on_device);
+int loom_b200_matrix_info(const loom_b200_matrix* m, int* rows, int* cols, int* groups, int* dtype);
+void loom_b200_matrix_free(loom_b200_ctx* ctx, loom_b200_matrix* m);
+
+#define LOOM_B200_MIXER_GLA 0    /* gated linear attention, one decay per key channel */
+#define LOOM_B200_MIXER_LATENT 1 /* softmax attention over cached latents, no positions */
+#define LOOM_B200_FFN_NONE 0
+#define LOOM_B200_FFN_DENSE 1    /* down(gelu(up h)), exact gelu */
+#define LOOM_B200_FFN_MOE 2      /* routed experts with the clamped gated unit; sigmoid scores, not renormalised, on the experts' input */
+
+typedef struct loom_b200_stack_dims {
+    int num_layers, width, vocab;
+    int max_seq_len;       /* positions of a sequence; <= 0 means 2048 */
+    int dtype;             /* LOOM_B200_DTYPE_*: matrices, activations of the products and the latent cache */
+    int conv_taps;         /* taps of the short convolution in front of a mixer (layers without weights for it have none) */
+    double norm_eps;       /* every RMS norm: x / sqrt(mean(x^2) + eps) */
+    double residual_mult;  /* x += residual_mult * branch */
+} loom_b200_stack_dims;
+
+typedef struct loom_b200_layer_spec {
+    int mixer;             /* LOOM_B200_MIXER_* */
+    int heads, dim, vdim;  /* per head: query/key and value dimensions */
+    int rank;              /* GLA: inner size of the low-rank decay projection; latent: size of the latent */
+    int kv_from;           /* latent: layer whose cached latents this one reads, or -1 for its own */
+    double tau;            /* GLA: decay = sigmoid(z)^(1/tau) */
+    double scale;          /* latent: factor of the scores */
+    int ffn;               /* LOOM_B200_FFN_* */
+    int ff;                /* inner size (of one expert) */
+    int experts, top;
+    double limit;          /* clamp of the gated unit */
+} loom_b200_layer_spec;
+
+/* Matrices are borrowed and must outlive the decoder; vectors are host float32 and are copied. */
+typedef struct loom_b200_layer_weights {
+    const loom_b200_matrix* in;   /* GLA: rows q, k [heads*dim], v, gate [heads*vdim], decay input [rank]; latent: q [heads*dim] and,
+                                     unless kv_from is set, the latent projection [rank] */
+    const loom_b200_matrix* out;  /* [width, heads*vdim] */
+    const loom_b200_matrix *up_k, *up_v;          /* latent: [heads*dim, rank], [heads*vdim, rank] */
+    const float* mixer_norm;      /* GLA: [vdim] norm of every head's output; latent: [rank] norm of the latent */
+    const float *decay_w, *decay_b;               /* GLA: [heads*dim, rank], [heads*dim] */
+    const float* conv_w;          /* [width, conv_taps] or NULL */
+    float norm1, norm2;           /* gains of the norms in front of the mixer and the feed-forward */
+    const loom_b200_matrix *router;               /* [experts, width] */
+    const loom_b200_matrix *gate, *up, *down;     /* dense: up [ff, width], down [width, ff]; experts: one group each */
+} loom_b200_layer_weights;
+
+int loom_b200_decoder_create_stack(loom_b200_ctx* ctx, const loom_b200_stack_dims* dims, loom_b200_decoder** out);
+/* after decoder_set_batch (if any): the states of every sequence are allocated here */
+int loom_b200_decoder_set_layer(loom_b200_decoder* dec, int layer, const loom_b200_layer_spec* spec, const loom_b200_layer_weights* weights);
+/* table: [vocab, width] in the stack's dtype, row-major device memory (borrowed); head [vocab, width] (borrowed) */
+int loom_b200_decoder_set_stack_embeddings(loom_b200_decoder* dec, const void* table_dev, float embed_norm, const loom_b200_matrix* head,
+                                           float final_norm);
+/* Appends n tokens to the selected sequence from whatever state it is in (reset starts it anew) and returns the logits after
+ * the tokens at places want[0..n_want) of this call (ascending), [n_want, vocab].  A prompt may be cut into calls anywhere.
+ * Ternary decoders take it too, with want empty or the last place only. */
+int loom_b200_decoder_extend(loom_b200_decoder* dec, const int32_t* tokens, int n, const int32_t* want, int n_want, float* logits_host);
 
 /* ---- tensor parallelism over the GPUs of one box --------------------------------------------------
  * The reference has no multi-device path (its only sharding notion is the per-layer tile size,

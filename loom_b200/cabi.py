@@ -15,6 +15,11 @@ _PKG = os.path.dirname(os.path.abspath(__file__))
 ACT_RELU, ACT_SILU, ACT_GELU, ACT_TANH, ACT_SIGMOID, ACT_LEAKY_RELU, ACT_RELU2, ACT_LINEAR = 0, 1, 2, 3, 4, 5, 6, -1
 
 
+DTYPE_F32, DTYPE_BF16 = 0, 1
+DTYPES = {"float32": DTYPE_F32, "bfloat16": DTYPE_BF16}
+MIXER_GLA, MIXER_LATENT = 0, 1
+FFN_NONE, FFN_DENSE, FFN_MOE = 0, 1, 2
+
 ERR_INVALID, ERR_CUDA, ERR_UNSUPPORTED, ERR_NO_DEVICE, ERR_TIMEOUT, ERR_COMM = -1, -2, -3, -4, -5, -6
 
 
@@ -108,6 +113,14 @@ SIGNATURES = {
     "loom_b200_decoder_step_launches": (_i, [_vp]),
     "loom_b200_decoder_linears_frame": (_i, [_vp]),
     "loom_b200_decoder_last_residual": (_i, [_vp, _vp, _i, C.POINTER(_i)]),
+    "loom_b200_matrix_create": (_i, [_vp, _i, _i, _i, _i, C.POINTER(_vp)]),
+    "loom_b200_matrix_put": (_i, [_vp, _vp, _i, _i, _i, _vp, _i, _i]),
+    "loom_b200_matrix_info": (_i, [_vp, C.POINTER(_i), C.POINTER(_i), C.POINTER(_i), C.POINTER(_i)]),
+    "loom_b200_matrix_free": (None, [_vp, _vp]),
+    "loom_b200_decoder_create_stack": (_i, [_vp, _vp, C.POINTER(_vp)]),
+    "loom_b200_decoder_set_layer": (_i, [_vp, _i, _vp, _vp]),
+    "loom_b200_decoder_set_stack_embeddings": (_i, [_vp, _vp, _f, _vp, _f]),
+    "loom_b200_decoder_extend": (_i, [_vp, _vp, _i, _vp, _i, _vp]),
     "loom_b200_tp_unique_id": (_i, [_vp]),
     "loom_b200_tp_init": (_i, [_vp, _i, _i, _vp]),
     "loom_b200_tp_peer_handle": (_i, [_vp, _vp]),
@@ -124,6 +137,21 @@ class DecoderDims(C.Structure):
     _fields_ = [("num_layers", _i), ("hidden", _i), ("num_heads", _i), ("num_kv_heads", _i), ("head_dim", _i),
                 ("intermediate", _i), ("vocab", _i), ("rms_eps", _d), ("rope_theta", _d), ("activation", _i),
                 ("max_seq_len", _i)]
+
+
+class StackDims(C.Structure):
+    _fields_ = [("num_layers", _i), ("width", _i), ("vocab", _i), ("max_seq_len", _i), ("dtype", _i), ("conv_taps", _i), ("norm_eps", _d),
+                ("residual_mult", _d)]
+
+
+class LayerSpec(C.Structure):
+    _fields_ = [("mixer", _i), ("heads", _i), ("dim", _i), ("vdim", _i), ("rank", _i), ("kv_from", _i), ("tau", _d), ("scale", _d), ("ffn", _i),
+                ("ff", _i), ("experts", _i), ("top", _i), ("limit", _d)]
+
+
+class LayerWeights(C.Structure):
+    _fields_ = [("in_", _vp), ("out", _vp), ("up_k", _vp), ("up_v", _vp), ("mixer_norm", _vp), ("decay_w", _vp), ("decay_b", _vp), ("conv_w", _vp),
+                ("norm1", _f), ("norm2", _f), ("router", _vp), ("gate", _vp), ("up", _vp), ("down", _vp)]
 
 
 class GenMetrics(C.Structure):
@@ -478,8 +506,46 @@ class MHA:
             pass
 
 
+def to_bf16(a: np.ndarray) -> np.ndarray:
+    """float32 -> bf16 bit patterns (round to nearest, ties to even)."""
+    u = np.ascontiguousarray(a, np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+class Matrix:
+    """bf16 or float32 matrices of one shape (`groups` of them) in the library's blocked layout."""
+
+    def __init__(self, ctx: "Context", rows: int, cols: int, groups: int = 1, dtype: int = DTYPE_BF16):
+        self.ctx, self.h = ctx, None
+        self.rows, self.cols, self.groups, self.dtype = rows, cols, groups, dtype
+        h = _vp()
+        ctx._check(lib().loom_b200_matrix_create(ctx.h, rows, cols, groups, dtype, C.byref(h)))
+        self.h = h
+
+    def put(self, src, dtype: int = DTYPE_F32, row0: int = 0, group: int = 0, rows: int | None = None):
+        """Rows row0 ... of a group from a host array (float32, or uint16 bit patterns with DTYPE_BF16) or a device tensor."""
+        on_device = hasattr(src, "data_ptr")
+        if not on_device:
+            src = np.ascontiguousarray(src)
+        n = rows if rows is not None else src.shape[0]
+        self.ctx._check(lib().loom_b200_matrix_put(self.ctx.h, self.h, group, row0, n, _ptr(src), dtype, 1 if on_device else 0))
+        return self
+
+    def free(self):
+        if self.h:
+            lib().loom_b200_matrix_free(self.ctx.h, self.h)
+            self.h = None
+
+    def __del__(self):
+        try:
+            self.free()
+        except Exception:
+            pass
+
+
 class Decoder:
-    """The ternary decoder stack on the device (InitHFDecoderBlocks + Transformer stand-in)."""
+    """A decoder on the device: the ternary stack (InitHFDecoderBlocks + Transformer stand-in), or with `Decoder.stack` layers that
+    are given one by one (`set_layer`)."""
 
     def __init__(self, ctx: Context, layers, hidden, heads, kv_heads, head_dim, inter, vocab, eps, theta,
                  act=ACT_SILU, max_seq_len=2048):
@@ -489,6 +555,47 @@ class Decoder:
         ctx._check(lib().loom_b200_decoder_create(ctx.h, C.byref(self.dims), C.byref(h)))
         self.h = h
         self._keep = []
+
+    @classmethod
+    def stack(cls, ctx: Context, layers, width, vocab, eps, residual_mult=1.0, conv_taps=0, dtype=DTYPE_BF16, max_seq_len=2048) -> "Decoder":
+        self = cls.__new__(cls)
+        self.ctx, self.h, self._keep = ctx, None, []
+        self.dims = DecoderDims(layers, width, 0, 0, 0, 0, vocab, eps, 0.0, ACT_LINEAR, max_seq_len)
+        d = StackDims(layers, width, vocab, max_seq_len, dtype, conv_taps, eps, residual_mult)
+        h = _vp()
+        ctx._check(lib().loom_b200_decoder_create_stack(ctx.h, C.byref(d), C.byref(h)))
+        self.h = h
+        return self
+
+    def set_layer(self, i: int, spec: dict, weights: dict):
+        """spec: fields of LayerSpec; weights: "in", "out", "up_k", "up_v", "router", "gate", "up", "down" as Matrix and the vectors and
+        gains of LayerWeights (absent = none)."""
+        s, w, keep = LayerSpec(**spec), LayerWeights(), []
+        for name, value in weights.items():
+            if value is None:
+                continue
+            if isinstance(value, Matrix):
+                self._keep.append(value)
+                value = value.h
+            elif name not in ("norm1", "norm2"):
+                value = _f32(value)
+                keep.append(value)
+                value = value.ctypes.data
+            setattr(w, "in_" if name == "in" else name, value)
+        self.ctx._check(lib().loom_b200_decoder_set_layer(self.h, i, C.byref(s), C.byref(w)))
+
+    def set_stack_embeddings(self, table_dev, embed_norm: float, head: Matrix, final_norm: float):
+        """table_dev: [vocab, width] on the device in the stack's dtype."""
+        self._keep += [table_dev, head]
+        self.ctx._check(lib().loom_b200_decoder_set_stack_embeddings(self.h, _ptr(table_dev), float(embed_norm), head.h, float(final_norm)))
+
+    def extend(self, tokens, want=()):
+        """Appends tokens to the selected sequence; the logits [len(want), vocab] after the tokens at the places `want` (ascending)."""
+        tokens = np.ascontiguousarray(tokens, np.int32).ravel()
+        w = np.ascontiguousarray(want, np.int32).ravel()
+        logits = np.empty((w.size, self.dims.vocab), np.float32)
+        self.ctx._check(lib().loom_b200_decoder_extend(self.h, tokens.ctypes.data, tokens.size, w.ctypes.data, w.size, logits.ctypes.data if w.size else None))
+        return logits
 
     def set_block(self, b, weights7, g1=None, g2=None, attn_inner=None, ffn_inner=None):
         assert len(weights7) == 7

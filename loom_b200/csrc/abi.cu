@@ -393,6 +393,8 @@ int loom_b200_ctx_set_option(loom_b200_ctx* ctx, const char* key, int value) {
         ctx->opt_prefill_gemm = value != 0;
     } else if (!strcmp(key, "tp_peer")) {
         ctx->opt_tp_peer = value != 0;
+    } else if (!strcmp(key, "dense_tc")) {
+        ctx->opt_dense_tc = value != 0;
     } else if (!strcmp(key, "tp_graph")) {
         ctx->opt_tp_graph = value != 0;
     } else {

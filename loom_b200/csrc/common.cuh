@@ -94,6 +94,7 @@ struct loom_b200_ctx {
     int opt_quant_regs = 1;        // the GEMM's quantizer keeps a token's row in registers (0: staged in shared memory)
     int opt_gemm_stream = 1;       // over pre-expanded codes the GEMM runs as a persistent kernel with two accumulator buffers (0: the one-shot kernel)
     int opt_gemm_cache = 1;        // the token-block GEMM reads pre-expanded int8 codes (built per matrix on first use) instead of expanding the 2-bit tiles in the kernel
+    int opt_dense_tc = 1;          // bf16 token blocks run on the tensor cores (0: plain fused multiply-adds)
     int opt_tp_graph = 1;          // record the sharded decode step (collectives included) as a graph
     void* nccl_comm = nullptr;
     // peer mailboxes (tp.cu): this rank's exchange buffer, the device table of every rank's buffer (own included) as

@@ -8,8 +8,11 @@
 // current token and the output cursor live in device memory, so the same frame replays for every token and
 // the greedy loop never waits for the host.
 #include "layers.cuh"
+#include "stack.cuh"
 
+#include <algorithm>
 #include <chrono>
+#include <cmath>
 #include <vector>
 
 struct loom_b200_graph;  // defined in abi.cu
@@ -27,6 +30,7 @@ struct loom_b200_decoder {
     loom_b200_ctx* ctx = nullptr;
     loom_b200_decoder_dims d{};
     std::vector<LbDecBlock> blocks;
+    LbStack* stack = nullptr;  // layers given one by one (stack.cu) instead of ternary blocks
     const float* emb = nullptr;  // borrowed device pointer [vocab, hidden]
     const loom_b200_weight* head_tern = nullptr;  // untied LM head as a packed ternary matrix [vocab, hidden] (borrowed), or null
     float* final_gain = nullptr;
@@ -118,7 +122,7 @@ void dec_point_at_lane(loom_b200_decoder* dec, int lane) {
     dec->step = dec->step_all + lane;
     dec->out_tokens = dec->out_tokens_all + (size_t)lane * dec->out_cap;
     dec->logits = dec->logits_all + (size_t)lane * dec->d.vocab;
-    dec->cur_tok = dec->batch > 1 ? dec->tok_all + lane : dec->tok;
+    dec->cur_tok = dec->batch > 1 || dec->stack ? dec->tok_all + lane : dec->tok;
     dec->kv_offset = dec->kv_offsets.empty() ? 0 : dec->kv_offsets[lane];
     for (size_t i = 0; i < dec->blocks.size(); ++i) {
         LbDecBlock& b = dec->blocks[i];
@@ -205,6 +209,60 @@ int dec_gather_logits(loom_b200_decoder* dec, float* logits_row) {
     if (!(dec->head_sharded && dec->fused_tail)) return 0;
     const int vl = dec->d.vocab / dec->tp_world;
     return lb_tp_allgather_f32(dec->ctx, logits_row + (size_t)dec->tp_rank * vl, logits_row, (size_t)vl);
+}
+
+// What a forward of a stack ends with: the first maximum of every row of logits becomes its sequence's next token, goes to
+// its output ring, and the position advances (the stack's counterpart of the head's greedy tail).
+int dec_stack_tail(loom_b200_decoder* dec, int lane0, int rows, int pos_delta) {
+    LbArgmaxParams a;
+    a.logits = dec->logits_all + (size_t)lane0 * dec->d.vocab;
+    a.stride = dec->d.vocab;
+    a.vocab = dec->d.vocab;
+    a.rows = rows;
+    a.tok = dec->tok_all + lane0;
+    a.out_tokens = dec->out_tokens_all + (size_t)lane0 * dec->out_cap;
+    a.out_cap = dec->out_cap;
+    a.step = dec->step_all + lane0;
+    a.pos = dec->pos_all + lane0;
+    a.pos_delta = pos_delta;
+    return lb_launch_argmax_rows(dec->ctx, a);
+}
+
+// M tokens (one of each of sequences lane0 ...) through a stack, head and tail included
+int dec_stack_step(loom_b200_decoder* dec, int lane0, int M) {
+    LbStack* st = dec->stack;
+    if (int rc = lb_stack_step(dec->ctx, st, dec->tok_all + lane0, dec->pos_all + lane0, lane0, M)) return rc;
+    if (int rc = lb_stack_head(dec->ctx, st, st->x, nullptr, M, dec->logits_all + (size_t)lane0 * dec->d.vocab, dec->d.vocab)) return rc;
+    dec->last_resid = st->x;
+    dec->last_resid_rows = M;
+    return dec_stack_tail(dec, lane0, M, 1);
+}
+
+// The next M tokens (already in pf_tok) of the selected sequence through a stack.  The logits at the n_want places in `want`
+// (of this block) go to the host; the last block of a call also runs the head on its last token and the greedy tail.
+int dec_stack_block(loom_b200_decoder* dec, int M, int pos0, bool last, const int32_t* want, int n_want, float* logits_host) {
+    loom_b200_ctx* ctx = dec->ctx;
+    LbStack* st = dec->stack;
+    const int V = dec->d.vocab;
+    if (int rc = lb_stack_block(ctx, st, M, pos0, dec->lane)) return rc;
+    dec->last_resid = st->pf_x;
+    dec->last_resid_rows = M;
+    if (n_want > 0) LB_CUDA(ctx, cudaMemcpyAsync(st->pf_rows, want, (size_t)n_want * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
+    for (int i0 = 0; i0 < n_want; i0 += kStackHeadRows) {
+        const int n = std::min(kStackHeadRows, n_want - i0);
+        if (i0 > 0)
+            LB_CUDA(ctx, cudaMemcpyAsync(st->pf_rows, want + i0, (size_t)n * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
+        if (n <= lb_dense_gemv_max_tokens(dec->d.hidden, st->d.dtype)) {
+            if (int rc = lb_stack_head(ctx, st, st->pf_x, st->pf_rows, n, st->pf_logits, st->ldl)) return rc;
+        } else if (int rc = lb_stack_head_block(ctx, st, n)) {
+            return rc;
+        }
+        LB_CUDA(ctx, cudaMemcpy2DAsync(logits_host + (size_t)i0 * V, (size_t)V * 4, st->pf_logits, (size_t)st->ldl * 4, (size_t)V * 4, n, cudaMemcpyDeviceToHost, ctx->stream));
+        if (int rc = lb_sync_checked(ctx)) return rc;
+    }
+    if (!last) return lb_launch_add_scalar(ctx, dec->pos, M);
+    if (int rc = lb_stack_head(ctx, st, st->pf_x + (size_t)(M - 1) * st->ldx, nullptr, 1, dec->logits, V)) return rc;
+    return dec_stack_tail(dec, dec->lane, 1, M);
 }
 
 // A block of M prompt tokens (already in pf_tok) at positions pos0..pos0+M-1 through the whole stack, every
@@ -403,6 +461,7 @@ int dec_prefill_block(loom_b200_decoder* dec, int M, int pos0, bool head) {
 int dec_forward_chunk(loom_b200_decoder* dec, int M, int splits, bool head, int head_row, bool linears_only = false, bool embed = true,
                       const int* tok_src = nullptr) {
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack) return dec_stack_step(dec, dec->lane, M);
     const loom_b200_decoder_dims& d = dec->d;
     if (!linears_only && embed)
         if (int rc = lb_launch_embed(ctx, dec->emb, d.vocab, d.hidden, tok_src ? tok_src : dec->tok, M, dec->x)) return rc;
@@ -475,6 +534,11 @@ int dec_forward_chunk(loom_b200_decoder* dec, int M, int splits, bool head, int 
 // table.  Its tail publishes every sequence's next token and advances its position.
 int dec_forward_lanes(loom_b200_decoder* dec, int lane0, int M) {
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack) {
+        for (int m0 = 0, per = lb_stack_max_lanes(dec->stack); m0 < M; m0 += per)
+            if (int rc = dec_stack_step(dec, lane0 + m0, std::min(per, M - m0))) return rc;
+        return 0;
+    }
     const loom_b200_decoder_dims& d = dec->d;
     const int H = d.hidden;
     if (int rc = lb_launch_embed(ctx, dec->emb, d.vocab, H, dec->tok_all + lane0, M, dec->x)) return rc;
@@ -544,6 +608,7 @@ int dec_forward_lanes(loom_b200_decoder* dec, int lane0, int M) {
 
 int dec_check_ready(loom_b200_decoder* dec) {
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack) return lb_stack_ready(ctx, dec->stack);
     LB_REQUIRE(ctx, dec->emb != nullptr, "decoder: embeddings are not set");
     for (size_t i = 0; i < dec->blocks.size(); ++i)
         LB_REQUIRE(ctx, dec->blocks[i].ready, "decoder: block %zu has no weights", i);
@@ -564,7 +629,7 @@ int dec_step(loom_b200_decoder* dec, bool host_token) {
     loom_b200_ctx* ctx = dec->ctx;
     const loom_b200_decoder_dims& d = dec->d;
     const bool in_frame = !dec->fused_tail;  // without the fused tail the gather is the first launch of the frame
-    if (dec->fused_tail && host_token)
+    if (dec->fused_tail && host_token && !dec->stack)  // (a stack's step starts with its own gather)
         if (int rc = lb_launch_embed(ctx, dec->emb, d.vocab, d.hidden, dec->cur_tok, 1, dec->x)) return rc;
     if (dec->step_graph) return loom_b200_graph_launch(ctx, dec->step_graph);
     if (dec->tp_world > 1 && !ctx->opt_tp_graph) return dec_forward_chunk(dec, 1, dec->decode_splits, true, 0, false, in_frame, dec->cur_tok);
@@ -585,9 +650,101 @@ int dec_step(loom_b200_decoder* dec, bool host_token) {
     return 0;
 }
 
+// Appends n tokens to the selected sequence; the logits at the places want[0..n_want) (ascending) go to the host.
+int dec_extend(loom_b200_decoder* dec, const int32_t* tokens, int n, const int32_t* want, int n_want, float* logits_host) {
+    loom_b200_ctx* ctx = dec->ctx;
+    const size_t V = (size_t)dec->d.vocab;
+    LB_REQUIRE(ctx, dec->kv_offset + n <= dec->d.max_seq_len, "decoder_forward: %d positions exceed MaxSeqLen %d", dec->kv_offset + n, dec->d.max_seq_len);
+    const bool want_last = n_want > 0 && want[n_want - 1] == n - 1;
+    if (dec->stack && n > 1) {
+        const int cap = std::min(n, kStackBlock);
+        if (int rc = lb_stack_ensure_block(ctx, dec->stack, cap)) return rc;
+        std::vector<int32_t> local(want, want + n_want);
+        int w = 0;
+        for (int s0 = 0; s0 < n; s0 += cap) {
+            const int M = std::min(cap, n - s0);
+            LB_CUDA(ctx, cudaMemcpyAsync(dec->stack->pf_tok, tokens + s0, (size_t)M * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
+            int w1 = w;
+            while (w1 < n_want && want[w1] < s0 + M) local[w1] = want[w1] - s0, ++w1;
+            if (int rc = dec_stack_block(dec, M, dec->kv_offset + s0, s0 + M == n, local.data() + w, w1 - w, logits_host ? logits_host + (size_t)w * V : nullptr)) return rc;
+            w = w1;
+        }
+        dec->kv_offset += n;
+        return 0;
+    }
+    if (n == 1) {
+        if (int rc = lb_launch_set_scalar(ctx, dec->cur_tok, tokens[0])) return rc;
+        if (int rc = dec_step(dec, true)) return rc;
+    } else if (n >= kGemmMinTokens && ctx->opt_prefill_gemm) {
+        const int cap = n < kPrefillBlock ? n : kPrefillBlock;
+        if (int rc = dec_ensure_prefill(dec, cap)) return rc;
+        for (int s0 = 0; s0 < n; s0 += cap) {
+            const int M = n - s0 < cap ? n - s0 : cap;
+            LB_CUDA(ctx, cudaMemcpyAsync(dec->pf_tok, tokens + s0, (size_t)M * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
+            if (int rc = dec_prefill_block(dec, M, dec->kv_offset + s0, s0 + M == n)) return rc;
+        }
+    } else {
+        // tokens per pass: what the widest input row (hidden, or this rank's slice of the intermediate) leaves room for
+        const int widest = dec->inter_l > dec->d.hidden ? dec->inter_l : dec->d.hidden;
+        const int chunk = lb_gemv_max_tokens(widest) < kChunkTokens ? lb_gemv_max_tokens(widest) : kChunkTokens;
+        for (int s0 = 0; s0 < n; s0 += chunk) {
+            const int M = n - s0 < chunk ? n - s0 : chunk;
+            LB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));  // h_tok is reused
+            for (int i = 0; i < M; ++i) dec->h_tok[i] = tokens[s0 + i];
+            LB_CUDA(ctx, cudaMemcpyAsync(dec->tok, dec->h_tok, M * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
+            const bool last = s0 + M == n;
+            if (int rc = dec_forward_chunk(dec, M, 1, last, M - 1)) return rc;
+        }
+    }
+    if (want_last) {
+        if (int rc = dec_gather_logits(dec, dec->logits)) return rc;
+        LB_CUDA(ctx, cudaMemcpyAsync(dec->h_logits, dec->logits, V * 4, cudaMemcpyDeviceToHost, ctx->stream));
+        if (int rc = lb_sync_checked(ctx)) return rc;
+        memcpy(logits_host + (size_t)(n_want - 1) * V, dec->h_logits, V * 4);
+    }
+    dec->kv_offset += n;
+    return 0;
+}
+
 }  // namespace
 
 extern "C" {
+
+// allocates the state every decoder has (dec->d, the ternary slices if any and ctx are set) and hands the decoder out
+static int dec_finish_create(loom_b200_decoder* dec, loom_b200_decoder** out) {
+    loom_b200_ctx* ctx = dec->ctx;
+    const loom_b200_decoder_dims& d = dec->d;
+    dec->out_cap = d.max_seq_len;
+    cudaError_t e = cudaSuccess;
+    auto A = [&](void** p, size_t bytes) {
+        if (e == cudaSuccess) e = cudaMalloc(p, bytes);
+        if (e == cudaSuccess) e = cudaMemsetAsync(*p, 0, bytes, ctx->stream);
+    };
+    A((void**)&dec->x, (size_t)kChunkTokens * d.hidden * 4);
+    if (!dec->stack) A((void**)&dec->prod, (size_t)kChunkTokens * dec->inter_l * 4);
+    A((void**)&dec->logits_all, (size_t)d.vocab * 4);
+    A((void**)&dec->hidden, (size_t)d.hidden * 4);
+    A((void**)&dec->tok, kChunkTokens * sizeof(int));
+    A((void**)&dec->pos_all, sizeof(int));
+    A((void**)&dec->step_all, sizeof(int));
+    A((void**)&dec->tok_all, sizeof(int));
+    A((void**)&dec->out_tokens_all, (size_t)dec->out_cap * sizeof(int));
+    dec->kv_offsets.assign(1, 0);
+    dec_point_at_lane(dec, 0);
+    if (dec->tp_world > 1) {
+        A((void**)&dec->tp_stats, 2 * kChunkTokens * sizeof(double));
+        A((void**)&dec->tp_acc, (size_t)kChunkTokens * d.hidden * sizeof(int32_t));
+    }
+    if (e == cudaSuccess) e = cudaMallocHost((void**)&dec->h_tok, kChunkTokens * sizeof(int));
+    if (e == cudaSuccess) e = cudaMallocHost((void**)&dec->h_logits, (size_t)d.vocab * 4);
+    if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
+    if (e != cudaSuccess) {
+        loom_b200_decoder_destroy(dec);
+        return lb_fail(ctx, LOOM_B200_ERR_CUDA, "decoder_create: %s", cudaGetErrorString(e));
+    }
+    *out = dec;
+    return 0;
+}
 
 int loom_b200_decoder_create(loom_b200_ctx* ctx, const loom_b200_decoder_dims* dims, loom_b200_decoder** out) {
     if (!ctx) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_create: ctx is NULL");
@@ -622,35 +779,66 @@ int loom_b200_decoder_create(loom_b200_ctx* ctx, const loom_b200_decoder_dims* d
     if (dec->decode_splits > 16) dec->decode_splits = 16;
     if (dec->decode_splits < 1) dec->decode_splits = 1;
     if (ctx->opt_decode_splits > 0) dec->decode_splits = ctx->opt_decode_splits;  // read when the decoder is created
-    dec->out_cap = dec->d.max_seq_len;
-    cudaError_t e = cudaSuccess;
-    auto A = [&](void** p, size_t bytes) {
-        if (e == cudaSuccess) e = cudaMalloc(p, bytes);
-        if (e == cudaSuccess) e = cudaMemsetAsync(*p, 0, bytes, ctx->stream);
-    };
-    A((void**)&dec->x, (size_t)kChunkTokens * d.hidden * 4);
-    A((void**)&dec->prod, (size_t)kChunkTokens * dec->inter_l * 4);
-    A((void**)&dec->logits_all, (size_t)d.vocab * 4);
-    A((void**)&dec->hidden, (size_t)d.hidden * 4);
-    A((void**)&dec->tok, kChunkTokens * sizeof(int));
-    A((void**)&dec->pos_all, sizeof(int));
-    A((void**)&dec->step_all, sizeof(int));
-    A((void**)&dec->tok_all, sizeof(int));
-    A((void**)&dec->out_tokens_all, (size_t)dec->out_cap * sizeof(int));
-    dec->kv_offsets.assign(1, 0);
-    dec_point_at_lane(dec, 0);
-    if (W > 1) {
-        A((void**)&dec->tp_stats, 2 * kChunkTokens * sizeof(double));
-        A((void**)&dec->tp_acc, (size_t)kChunkTokens * d.hidden * sizeof(int32_t));
-    }
-    if (e == cudaSuccess) e = cudaMallocHost((void**)&dec->h_tok, kChunkTokens * sizeof(int));
-    if (e == cudaSuccess) e = cudaMallocHost((void**)&dec->h_logits, (size_t)d.vocab * 4);
-    if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
-    if (e != cudaSuccess) {
-        loom_b200_decoder_destroy(dec);
-        return lb_fail(ctx, LOOM_B200_ERR_CUDA, "decoder_create: %s", cudaGetErrorString(e));
-    }
-    *out = dec;
+    return dec_finish_create(dec, out);
+}
+
+int loom_b200_decoder_create_stack(loom_b200_ctx* ctx, const loom_b200_stack_dims* dims, loom_b200_decoder** out) {
+    if (!ctx) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_create_stack: ctx is NULL");
+    LB_REQUIRE(ctx, dims && out, "decoder_create_stack: NULL argument");
+    *out = nullptr;
+    const loom_b200_stack_dims& d = *dims;
+    LB_REQUIRE(ctx, d.num_layers > 0 && d.width > 0 && d.vocab > 0, "decoder_create_stack: bad dimensions");
+    LB_REQUIRE(ctx, d.dtype == LOOM_B200_DTYPE_F32 || d.dtype == LOOM_B200_DTYPE_BF16, "decoder_create_stack: dtype %d", d.dtype);
+    LB_REQUIRE(ctx, d.conv_taps >= 0 && d.conv_taps <= 16, "decoder_create_stack: %d convolution taps (0..16)", d.conv_taps);
+    LB_REQUIRE(ctx, d.norm_eps >= 0, "decoder_create_stack: norm_eps %g", d.norm_eps);
+    if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_create_stack cannot be recorded");
+    if (ctx->tp_world > 1) return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "decoder_create_stack: not available under a tensor-parallel group");
+    if (int rc = lb_set_device(ctx)) return rc;
+    auto* dec = new loom_b200_decoder();
+    dec->ctx = ctx;
+    dec->d.num_layers = d.num_layers;
+    dec->d.hidden = d.width;
+    dec->d.vocab = d.vocab;
+    dec->d.max_seq_len = d.max_seq_len > 0 ? d.max_seq_len : 2048;
+    dec->d.rms_eps = d.norm_eps;
+    dec->stack = new LbStack();
+    dec->stack->d = d;
+    dec->stack->d.max_seq_len = dec->d.max_seq_len;
+    dec->stack->ldx = lb_round_up(d.width, 8);
+    dec->stack->layers.resize(d.num_layers);
+    dec->fused_tail = true;  // a stack's forward ends with its greedy tail
+    return dec_finish_create(dec, out);
+}
+
+int loom_b200_decoder_set_layer(loom_b200_decoder* dec, int layer, const loom_b200_layer_spec* spec, const loom_b200_layer_weights* weights) {
+    if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_set_layer: decoder is NULL");
+    loom_b200_ctx* ctx = dec->ctx;
+    LB_REQUIRE(ctx, dec->stack, "decoder_set_layer: not a layer stack");
+    LB_REQUIRE(ctx, spec && weights, "decoder_set_layer: NULL argument");
+    if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_set_layer cannot be recorded");
+    if (int rc = lb_set_device(ctx)) return rc;
+    dec_drop_graph(dec);
+    return lb_stack_set_layer(ctx, dec->stack, layer, *spec, *weights, dec->batch);
+}
+
+int loom_b200_decoder_set_stack_embeddings(loom_b200_decoder* dec, const void* table_dev, float embed_norm, const loom_b200_matrix* head,
+                                           float final_norm) {
+    if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_set_stack_embeddings: decoder is NULL");
+    loom_b200_ctx* ctx = dec->ctx;
+    LB_REQUIRE(ctx, dec->stack, "decoder_set_stack_embeddings: not a layer stack");
+    LB_REQUIRE(ctx, table_dev && head, "decoder_set_stack_embeddings: NULL argument");
+    LbStack* st = dec->stack;
+    LB_REQUIRE(ctx, head->rows == st->d.vocab && head->cols == st->d.width && head->dtype == st->d.dtype && head->groups == 1,
+               "decoder_set_stack_embeddings: head is %dx%d, expected %dx%d of the stack's dtype", head->rows, head->cols, st->d.vocab, st->d.width);
+    if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_set_stack_embeddings cannot be recorded");
+    if (int rc = lb_set_device(ctx)) return rc;
+    dec_drop_graph(dec);
+    st->table = table_dev;
+    st->head = head;
+    const float scal[2] = {embed_norm, final_norm};
+    if (!st->scal) LB_CUDA(ctx, cudaMalloc(&st->scal, sizeof(scal)));
+    LB_CUDA(ctx, cudaMemcpyAsync(st->scal, scal, sizeof(scal), cudaMemcpyHostToDevice, ctx->stream));
+    LB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
     return 0;
 }
 
@@ -671,6 +859,7 @@ void loom_b200_decoder_destroy(loom_b200_decoder* dec) {
         if (b.ffn_inner) cudaFree(b.ffn_inner);
     }
     dec_free_prefill(dec);
+    lb_stack_free(dec->stack);
     void* ptrs[] = {dec->final_gain, dec->x, dec->prod, dec->logits_all, dec->hidden, dec->tok, dec->pos_all, dec->step_all,
                     dec->tok_all, dec->out_tokens_all, dec->tp_stats, dec->tp_acc};
     for (void* p : ptrs)
@@ -686,6 +875,7 @@ int loom_b200_decoder_set_block(loom_b200_decoder* dec, int block, const float* 
                                 const float* ffn_inner_norm, int ffn_inner_len) {
     if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_set_block: decoder is NULL");
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack) return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "decoder_set_block: not for a layer stack");
     const loom_b200_decoder_dims& d = dec->d;
     LB_REQUIRE(ctx, block >= 0 && block < d.num_layers, "decoder_set_block: block %d out of range", block);
     LB_REQUIRE(ctx, w7 != nullptr, "decoder_set_block: weights are NULL");
@@ -750,6 +940,7 @@ int loom_b200_decoder_set_block(loom_b200_decoder* dec, int block, const float* 
 int loom_b200_decoder_set_embeddings(loom_b200_decoder* dec, const float* emb_dev, const float* final_gain) {
     if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_set_embeddings: decoder is NULL");
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack) return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "decoder_set_embeddings: not for a layer stack");
     LB_REQUIRE(ctx, emb_dev != nullptr, "decoder_set_embeddings: embeddings are NULL");
     if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_set_embeddings cannot be recorded");
     if (int rc = lb_set_device(ctx)) return rc;
@@ -767,6 +958,7 @@ int loom_b200_decoder_set_embeddings(loom_b200_decoder* dec, const float* emb_de
 int loom_b200_decoder_set_lm_head_ternary(loom_b200_decoder* dec, const loom_b200_weight* head) {
     if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_set_lm_head_ternary: decoder is NULL");
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack) return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "decoder_set_lm_head_ternary: not for a layer stack");
     if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_set_lm_head_ternary cannot be recorded");
     LB_REQUIRE(ctx, dec->emb != nullptr, "decoder_set_lm_head_ternary: set the embeddings first");
     LB_REQUIRE(ctx, dec->tp_world == 1 && dec->batch == 1, "decoder_set_lm_head_ternary: one GPU, one sequence");
@@ -808,45 +1000,29 @@ int loom_b200_decoder_forward(loom_b200_decoder* dec, const int32_t* tokens, int
     if (!incremental) {
         if (int rc = loom_b200_decoder_reset(dec)) return rc;
     }
-    LB_REQUIRE(ctx, dec->kv_offset + n <= dec->d.max_seq_len, "decoder_forward: %d positions exceed MaxSeqLen %d", dec->kv_offset + n, dec->d.max_seq_len);
-    if (n == 1) {
-        dec->h_tok[0] = tokens[0];
-        LB_CUDA(ctx, cudaMemcpyAsync(dec->cur_tok, dec->h_tok, sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
-        if (int rc = dec_step(dec, true)) return rc;
-    } else if (n >= kGemmMinTokens && ctx->opt_prefill_gemm) {
-        const int cap = n < kPrefillBlock ? n : kPrefillBlock;
-        if (int rc = dec_ensure_prefill(dec, cap)) return rc;
-        for (int s0 = 0; s0 < n; s0 += cap) {
-            const int M = n - s0 < cap ? n - s0 : cap;
-            LB_CUDA(ctx, cudaMemcpyAsync(dec->pf_tok, tokens + s0, (size_t)M * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
-            if (int rc = dec_prefill_block(dec, M, dec->kv_offset + s0, s0 + M == n)) return rc;
-        }
-    } else {
-        // tokens per pass: what the widest input row (hidden, or this rank's slice of the intermediate) leaves room for
-        const int widest = dec->inter_l > dec->d.hidden ? dec->inter_l : dec->d.hidden;
-        const int chunk = lb_gemv_max_tokens(widest) < kChunkTokens ? lb_gemv_max_tokens(widest) : kChunkTokens;
-        for (int s0 = 0; s0 < n; s0 += chunk) {
-            const int M = n - s0 < chunk ? n - s0 : chunk;
-            LB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));  // h_tok is reused
-            for (int i = 0; i < M; ++i) dec->h_tok[i] = tokens[s0 + i];
-            LB_CUDA(ctx, cudaMemcpyAsync(dec->tok, dec->h_tok, M * sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
-            const bool last = s0 + M == n;
-            if (int rc = dec_forward_chunk(dec, M, 1, last, M - 1)) return rc;
-        }
-    }
-    dec->kv_offset += n;
-    if (logits_host) {
-        if (int rc = dec_gather_logits(dec, dec->logits)) return rc;
-        LB_CUDA(ctx, cudaMemcpyAsync(dec->h_logits, dec->logits, (size_t)dec->d.vocab * 4, cudaMemcpyDeviceToHost, ctx->stream));
-        if (int rc = lb_sync_checked(ctx)) return rc;
-        memcpy(logits_host, dec->h_logits, (size_t)dec->d.vocab * 4);
-    }
-    return 0;
+    const int32_t place = n - 1;
+    return dec_extend(dec, tokens, n, &place, logits_host ? 1 : 0, logits_host);
+}
+
+int loom_b200_decoder_extend(loom_b200_decoder* dec, const int32_t* tokens, int n, const int32_t* want, int n_want, float* logits_host) {
+    if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_extend: decoder is NULL");
+    loom_b200_ctx* ctx = dec->ctx;
+    LB_REQUIRE(ctx, tokens && n > 0, "decoder_extend: no tokens");
+    LB_REQUIRE(ctx, n_want >= 0 && (n_want == 0 || (want && logits_host)), "decoder_extend: NULL buffer");
+    for (int i = 0; i < n_want; ++i)
+        LB_REQUIRE(ctx, want[i] >= 0 && want[i] < n && (i == 0 || want[i] > want[i - 1]), "decoder_extend: place %d of %d tokens (places ascend)", want[i], n);
+    if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_extend takes host buffers and cannot be recorded");
+    if (!dec->stack && n_want > 0 && (n_want > 1 || want[0] != n - 1))  // the greedy tail of a ternary decoder's head keeps one row
+        return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "decoder_extend: a ternary decoder returns the last token's logits only");
+    if (int rc = dec_check_ready(dec)) return rc;
+    if (int rc = lb_set_device(ctx)) return rc;
+    return dec_extend(dec, tokens, n, want, n_want, logits_host);
 }
 
 int loom_b200_decoder_last_hidden(loom_b200_decoder* dec, float* hidden_host) {
     if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_last_hidden: decoder is NULL");
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack) return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "decoder_last_hidden: not for a layer stack");
     LB_REQUIRE(ctx, hidden_host != nullptr, "decoder_last_hidden: NULL buffer");
     if (int rc = lb_set_device(ctx)) return rc;
     LB_CUDA(ctx, cudaMemcpyAsync(hidden_host, dec->hidden, (size_t)dec->d.hidden * 4, cudaMemcpyDeviceToHost, ctx->stream));
@@ -885,6 +1061,8 @@ int loom_b200_decoder_set_batch(loom_b200_decoder* dec, int batch) {
     LB_REQUIRE(ctx, dec->tp_world == 1 || (ctx->tp_peer && ctx->opt_tp_peer && dec->head_sharded),
                "decoder_set_batch: under a tensor-parallel group sequences in parallel need the peer-memory exchange (tp_attach_peers) and a vocabulary that divides by the group");
     for (auto& b : dec->blocks) LB_REQUIRE(ctx, !b.ready, "decoder_set_batch must be called before decoder_set_block");
+    if (dec->stack)
+        for (auto& l : dec->stack->layers) LB_REQUIRE(ctx, !l.ready, "decoder_set_batch must be called before decoder_set_layer");
     if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_set_batch cannot be recorded");
     if (int rc = lb_set_device(ctx)) return rc;
     LB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
@@ -1008,6 +1186,8 @@ int loom_b200_decoder_read_tokens_batch(loom_b200_decoder* dec, int32_t* tokens_
 int loom_b200_decoder_set_kv_offset(loom_b200_decoder* dec, int kv_offset) {
     if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_set_kv_offset: decoder is NULL");
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack && kv_offset != dec->kv_offset)
+        return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "decoder_set_kv_offset: the recurrent states of a layer stack cannot be cut back");
     LB_REQUIRE(ctx, kv_offset > 0 && kv_offset <= dec->kv_offset, "decoder_set_kv_offset: %d outside (0, %d]: a sequence can only be cut back", kv_offset, dec->kv_offset);
     if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_set_kv_offset cannot be recorded");
     if (int rc = lb_set_device(ctx)) return rc;
@@ -1022,6 +1202,7 @@ int loom_b200_decoder_step_launches(const loom_b200_decoder* dec) { return dec ?
 int loom_b200_decoder_linears_frame(loom_b200_decoder* dec) {
     if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_linears_frame: decoder is NULL");
     loom_b200_ctx* ctx = dec->ctx;
+    if (dec->stack) return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "decoder_linears_frame: not for a layer stack");
     if (int rc = dec_check_ready(dec)) return rc;
     LB_REQUIRE(ctx, dec->tp_world == 1, "decoder_linears_frame: not available under a tensor-parallel group");
     if (int rc = lb_set_device(ctx)) return rc;
@@ -1074,11 +1255,12 @@ int loom_b200_decoder_last_residual(loom_b200_decoder* dec, float* rows_host, in
     if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_last_residual: decoder is NULL");
     loom_b200_ctx* ctx = dec->ctx;
     LB_REQUIRE(ctx, rows_host && max_rows > 0, "decoder_last_residual: NULL buffer");
+    const size_t row_bytes = (size_t)dec->d.hidden * sizeof(float), ld_bytes = dec->stack ? (size_t)dec->stack->ldx * sizeof(float) : row_bytes;
     LB_REQUIRE(ctx, dec->last_resid && dec->last_resid_rows > 0, "decoder_last_residual: nothing has been forwarded yet");
     if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "decoder_last_residual takes host buffers and cannot be recorded");
     if (int rc = lb_set_device(ctx)) return rc;
     const int rows = dec->last_resid_rows < max_rows ? dec->last_resid_rows : max_rows;
-    LB_CUDA(ctx, cudaMemcpyAsync(rows_host, dec->last_resid, (size_t)rows * dec->d.hidden * sizeof(float), cudaMemcpyDeviceToHost, ctx->stream));
+    LB_CUDA(ctx, cudaMemcpy2DAsync(rows_host, row_bytes, dec->last_resid, ld_bytes, row_bytes, rows, cudaMemcpyDeviceToHost, ctx->stream));
     if (int rc = lb_sync_checked(ctx)) return rc;
     if (rows_out) *rows_out = rows;
     return 0;
@@ -1098,8 +1280,7 @@ int loom_b200_decoder_generate(loom_b200_decoder* dec, const int32_t* prompt, in
     // prefill: a one-token prompt still starts a fresh sequence
     if (n_prompt == 1) {
         if (int rc = loom_b200_decoder_reset(dec)) return rc;
-        dec->h_tok[0] = prompt[0];
-        LB_CUDA(ctx, cudaMemcpyAsync(dec->cur_tok, dec->h_tok, sizeof(int), cudaMemcpyHostToDevice, ctx->stream));
+        if (int rc = lb_launch_set_scalar(ctx, dec->cur_tok, prompt[0])) return rc;
         if (int rc = dec_step(dec, true)) return rc;
         dec->kv_offset = 1;
     } else {

@@ -434,14 +434,19 @@ __device__ __forceinline__ void argmax_merge(float& best, int& idx, float ov, in
     }
 }
 
-__global__ void __launch_bounds__(256) lb_argmax_advance_kernel(const float* __restrict__ logits, int vocab, int* tok,
-                                                                int* out_tokens, int out_cap, int* step, int* pos,
-                                                                float* part_val, int* part_idx, unsigned int* cnt) {
+constexpr int kArgmaxRows = 8;  // rows of one launch (grid y)
+
+__global__ void __launch_bounds__(256) lb_argmax_advance_kernel(const LbArgmaxParams p) {
     __shared__ float sv[8];
     __shared__ int si[8];
     __shared__ int s_last;
     lb_pdl_launch_dependents();
     lb_pdl_wait();
+    const int row = blockIdx.y, vocab = p.vocab;
+    const float* __restrict__ logits = p.logits + (size_t)row * p.stride;
+    float* part_val = p.part_val + row * kArgmaxCtas;
+    int* part_idx = p.part_idx + row * kArgmaxCtas;
+    unsigned int* cnt = p.cnt + row;
     const int per = (vocab + gridDim.x - 1) / gridDim.x;
     const int lo = blockIdx.x * per, hi = min(vocab, lo + per);
     float best = -INFINITY;
@@ -481,13 +486,13 @@ __global__ void __launch_bounds__(256) lb_argmax_advance_kernel(const float* __r
     }
     if (lane == 0) {
         if (idx == 0x7fffffff) idx = 0;  // only NaNs: the reference keeps index 0
-        tok[0] = idx;
-        if (out_tokens && step) {
-            int s = *step;
-            if (s < out_cap) out_tokens[s] = idx;
-            *step = s + 1;
+        p.tok[row] = idx;
+        if (p.out_tokens && p.step) {
+            int s = p.step[row];
+            if (s < p.out_cap) p.out_tokens[(size_t)row * p.out_cap + s] = idx;
+            p.step[row] = s + 1;
         }
-        if (pos) *pos += 1;
+        if (p.pos) p.pos[row] += p.pos_delta;
         *cnt = 0;
     }
 }
@@ -539,6 +544,12 @@ __global__ void lb_add_scalar_kernel(int* p, int delta) {
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     if (threadIdx.x == 0) *p += delta;
+}
+
+__global__ void lb_set_scalar_kernel(int* p, int value) {
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    if (threadIdx.x == 0) *p = value;
 }
 
 // Causal attention of a block of prompt tokens.  One CTA per (KV head, tile of query tokens): the 64 query rows of
@@ -867,26 +878,46 @@ int lb_launch_lm_head_legacy(loom_b200_ctx* ctx, const LbLmHeadParams& pin) {
 
 int lb_launch_argmax_advance(loom_b200_ctx* ctx, const float* logits, int vocab, int* tok, int* out_tokens, int out_cap,
                              int* step, int* pos) {
+    LbArgmaxParams p;
+    p.logits = logits;
+    p.vocab = vocab;
+    p.tok = tok;
+    p.out_tokens = out_tokens;
+    p.out_cap = out_cap;
+    p.step = step;
+    p.pos = pos;
+    return lb_launch_argmax_rows(ctx, p);
+}
+
+int lb_launch_argmax_rows(loom_b200_ctx* ctx, const LbArgmaxParams& pin) {
+    LbArgmaxParams p = pin;
+    LB_REQUIRE(ctx, p.rows >= 1 && p.rows <= kArgmaxRows, "argmax: %d rows", p.rows);
     // partial results live in the context scratch of the argmax (allocated once)
     if (!ctx->argmax_scratch) {
         if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "argmax scratch would be allocated while recording a graph");
-        LB_CUDA(ctx, cudaMalloc(&ctx->argmax_scratch, kArgmaxCtas * 8 + 16));
-        LB_CUDA(ctx, cudaMemsetAsync(ctx->argmax_scratch, 0, kArgmaxCtas * 8 + 16, ctx->stream));
+        const size_t bytes = (size_t)kArgmaxRows * (kArgmaxCtas * 8 + 4);
+        LB_CUDA(ctx, cudaMalloc(&ctx->argmax_scratch, bytes));
+        LB_CUDA(ctx, cudaMemsetAsync(ctx->argmax_scratch, 0, bytes, ctx->stream));
     }
-    float* pv = (float*)ctx->argmax_scratch;
-    int* pi = (int*)(pv + kArgmaxCtas);
-    unsigned int* cnt = (unsigned int*)(pi + kArgmaxCtas);
+    p.part_val = (float*)ctx->argmax_scratch;
+    p.part_idx = (int*)(p.part_val + kArgmaxRows * kArgmaxCtas);
+    p.cnt = (unsigned int*)(p.part_idx + kArgmaxRows * kArgmaxCtas);
     int grid = kArgmaxCtas;
-    if (grid > (vocab + 255) / 256) grid = (vocab + 255) / 256;
+    if (grid > (p.vocab + 255) / 256) grid = (p.vocab + 255) / 256;
     if (grid < 1) grid = 1;
-    LB_CUDA(ctx, launch_pdl(ctx, lb_argmax_advance_kernel, dim3(grid), dim3(256), 0, logits, vocab, tok, out_tokens, out_cap,
-                            step, pos, pv, pi, cnt));
+    LB_CUDA(ctx, launch_pdl(ctx, lb_argmax_advance_kernel, dim3(grid, p.rows), dim3(256), 0, p));
     ctx->launches++;
     return 0;
 }
 
 int lb_launch_add_scalar(loom_b200_ctx* ctx, int* pos, int delta) {
     LB_CUDA(ctx, launch_pdl(ctx, lb_add_scalar_kernel, dim3(1), dim3(32), 0, pos, delta));
+    ctx->launches++;
+    return 0;
+}
+
+int lb_launch_set_scalar(loom_b200_ctx* ctx, int* p, int value) {
+    LB_CUDA(ctx, launch_pdl(ctx, lb_set_scalar_kernel, dim3(1), dim3(32), 0, p, value));
     ctx->launches++;
     return 0;
 }

@@ -111,5 +111,22 @@ int lb_lm_head_rows_per_pass(const loom_b200_ctx* ctx, const float* head, int hi
 // out_tokens[*step]; then *step += 1 and *pos += 1 so that a recorded frame can be replayed as is.
 int lb_launch_argmax_advance(loom_b200_ctx* ctx, const float* logits, int vocab, int* tok, int* out_tokens,
                              int out_cap, int* step, int* pos);
+// The same for several sequences, one row of logits each: tok[r], out_tokens[r * out_cap + step[r]], step[r] += 1 and
+// pos[r] += pos_delta.
+struct LbArgmaxParams {
+    const float* logits = nullptr;
+    long long stride = 0;
+    int rows = 1, vocab = 0;
+    int *tok = nullptr, *out_tokens = nullptr;
+    int out_cap = 0;
+    int *step = nullptr, *pos = nullptr;
+    int pos_delta = 1;
+    float* part_val = nullptr;  // scratch, set by the launcher
+    int* part_idx = nullptr;
+    unsigned int* cnt = nullptr;
+};
+int lb_launch_argmax_rows(loom_b200_ctx* ctx, const LbArgmaxParams& p);
 // *pos += delta (after a prefill chunk)
 int lb_launch_add_scalar(loom_b200_ctx* ctx, int* pos, int delta);
+// *p = value, the value travelling as a kernel argument: calls may follow one another without waiting for a staging buffer
+int lb_launch_set_scalar(loom_b200_ctx* ctx, int* p, int value);

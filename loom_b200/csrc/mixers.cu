@@ -1,0 +1,711 @@
+// mixers.cu -- kernels of mixers.cuh.
+#include "mixers.cuh"
+
+namespace {
+
+// ---- embedding, norms, short convolution --------------------------------------------------------------------
+
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_embed_norm_kernel(const WT* __restrict__ table, int vocab, int width, const int* tok, const float* gain,
+                                                            float eps, float* __restrict__ x, int ldx) {
+    __shared__ float red[8];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = tok[blockIdx.x];
+    float* out = x + (size_t)blockIdx.x * ldx;
+    const bool ok = t >= 0 && t < vocab;
+    const WT* row = table + (size_t)(ok ? t : 0) * width;
+    float ss = 0.f;
+    for (int k = threadIdx.x; k < width; k += blockDim.x) {
+        const float v = ok ? (float)row[k] : 0.f;
+        ss = fmaf(v, v, ss);
+    }
+    ss = lb_block_sumf(ss, red);
+    const float r = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)width), eps))) * *gain;
+    for (int k = threadIdx.x; k < width; k += blockDim.x) out[k] = ok ? (float)row[k] * r : 0.f;
+}
+
+constexpr int kNormTokens = 16;  // tokens of a CTA
+constexpr int kMaxTaps = 16;
+
+__device__ __forceinline__ float row_rstd(const float* row, int width, float eps, int lane) {  // a warp per row
+    float ss = 0.f;
+    for (int k = lane; k < width; k += 32) ss = fmaf(row[k], row[k], ss);
+    ss = lb_warp_sumf(ss);
+    return __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)width), eps)));
+}
+
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p) {
+    constexpr int C = LbElem<WT>::kChunk;
+    __shared__ float s_r[kNormTokens + kMaxTaps];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * kNormTokens, t1 = min(p.T, t0 + kNormTokens);
+    const int back = p.conv_w ? p.taps - 1 : 0;
+    const float gain = *p.gain;
+    for (int i = warp; i < t1 - t0 + back; i += 8) {
+        const int t = t0 - back + i;
+        if (t < 0) continue;
+        const int src = p.row_idx ? p.row_idx[t] : t;
+        const float r = row_rstd(p.x + (size_t)src * p.ldx, p.width, p.eps, lane) * gain;
+        if (lane == 0) s_r[i] = r;
+    }
+    __syncthreads();
+    const int chunks = p.slices * 8;
+    for (int i = threadIdx.x; i < (t1 - t0) * chunks; i += blockDim.x) {
+        const int tt = i / chunks, c = i - tt * chunks, t = t0 + tt;
+        const int src = p.row_idx ? p.row_idx[t] : t;
+        float f[C];
+#pragma unroll
+        for (int e = 0; e < C; ++e) {
+            const int k = c * C + e;
+            f[e] = k < p.width ? p.x[(size_t)src * p.ldx + k] * s_r[tt + back] : 0.f;
+        }
+        if (p.conv_w) {
+            float a[C];
+#pragma unroll
+            for (int e = 0; e < C; ++e) a[e] = 0.f;
+            for (int j = 0; j < p.taps; ++j) {  // tap j looks back taps - 1 - j positions
+                const int ts = t - back + j;
+                if (p.pos0 + ts < 0) continue;
+#pragma unroll
+                for (int e = 0; e < C; ++e) {
+                    const int k = c * C + e;
+                    if (k >= p.width) continue;
+                    const float h = ts >= 0 ? p.x[(size_t)ts * p.ldx + k] * s_r[tt + j] : p.ring[(size_t)((p.pos0 + ts) % p.taps) * p.ring_ld + k];
+                    a[e] = fmaf(p.conv_w[(size_t)k * p.taps + j], h, a[e]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < C; ++e) f[e] += a[e];
+        }
+        *reinterpret_cast<uint4*>(p.img + lb_img_chunk(t, c, p.slices)) = lb_pack_chunk<WT>(f);
+    }
+}
+
+__global__ void __launch_bounds__(256) lb_conv_commit_kernel(const LbNormBlock p) {
+    __shared__ float red[8];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = p.T - 1 - (int)blockIdx.x;
+    if (t < 0) return;
+    const float* row = p.x + (size_t)t * p.ldx;
+    float ss = 0.f;
+    for (int k = threadIdx.x; k < p.width; k += blockDim.x) ss = fmaf(row[k], row[k], ss);
+    ss = lb_block_sumf(ss, red);
+    const float r = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)p.width), p.eps))) * *p.gain;
+    float* out = p.ring + (size_t)((p.pos0 + t) % p.taps) * p.ring_ld;
+    for (int k = threadIdx.x; k < p.width; k += blockDim.x) out[k] = row[k] * r;
+}
+
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_rows_image_kernel(const float* __restrict__ x, int ldx, int cols, int slices, uint8_t* __restrict__ img) {
+    constexpr int C = LbElem<WT>::kChunk;
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = blockIdx.x;
+    for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
+        float f[C];
+#pragma unroll
+        for (int e = 0; e < C; ++e) f[e] = c * C + e < cols ? x[(size_t)t * ldx + c * C + e] : 0.f;
+        *reinterpret_cast<uint4*>(img + lb_img_chunk(t, c, slices)) = lb_pack_chunk<WT>(f);
+    }
+}
+
+// ---- gated linear attention -------------------------------------------------------------------------------------
+
+__device__ __forceinline__ float gla_alpha(const LbGla& p, const float* low, int ch) {
+    const int hd = p.heads * p.dim;
+    float z = 0.f;
+    for (int r = 0; r < p.rank; ++r) z = fmaf(p.a2t[(size_t)r * hd + ch], low[r], z);
+    return expf(lb_log_sigmoidf(z + p.a2b[ch]) * p.inv_tau);
+}
+
+// one new token per sequence: CTA = (32 value columns, head, sequence); warps split the key channels
+__global__ void __launch_bounds__(256) lb_gla_step_kernel(const LbGla p, const int* pos, int lane0) {
+    extern __shared__ float sm[];
+    __shared__ float part[8][32];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int h = blockIdx.y, m = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int HD = p.heads * p.dim, HV = p.heads * p.vdim;
+    float *sq = sm, *sk = sm + p.dim, *sa = sk + p.dim, *low = sa + p.dim;
+    const float* row = p.proj + (size_t)m * p.ldp;
+    for (int r = threadIdx.x; r < p.rank; r += blockDim.x) low[r] = row[2 * HD + 2 * HV + r];
+    __syncthreads();
+    for (int d = threadIdx.x; d < p.dim; d += blockDim.x) {
+        sq[d] = row[h * p.dim + d] * p.qscale;
+        sk[d] = row[HD + h * p.dim + d];
+        sa[d] = gla_alpha(p, low, h * p.dim + d);
+    }
+    __syncthreads();
+    const int v = blockIdx.x * 32 + lane;
+    const bool fresh = pos[m] == 0;
+    float acc = 0.f;
+    if (v < p.vdim) {
+        float* S = p.state + (((size_t)(lane0 + m) * p.heads + h) * p.dim) * p.vdim + v;
+        const float vv = row[2 * HD + h * p.vdim + v];
+#pragma unroll 4
+        for (int d = warp; d < p.dim; d += 8) {
+            const float old = fresh ? 0.f : S[(size_t)d * p.vdim];
+            const float s = fmaf(sa[d], old, sk[d] * vv);
+            S[(size_t)d * p.vdim] = s;
+            acc = fmaf(sq[d], s, acc);
+        }
+    }
+    part[warp][lane] = acc;
+    __syncthreads();
+    if (warp == 0 && v < p.vdim) {
+        float o = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) o += part[w][lane];
+        p.o[(size_t)m * HV + h * p.vdim + v] = o;
+    }
+}
+
+__global__ void __launch_bounds__(256) lb_gla_decay_kernel(const LbGla p, float* __restrict__ alpha) {
+    extern __shared__ float low[];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = blockIdx.x, HD = p.heads * p.dim, HV = p.heads * p.vdim;
+    const float* row = p.proj + (size_t)t * p.ldp + 2 * HD + 2 * HV;
+    for (int r = threadIdx.x; r < p.rank; r += blockDim.x) low[r] = row[r];
+    __syncthreads();
+    for (int ch = threadIdx.x; ch < HD; ch += blockDim.x) alpha[(size_t)t * HD + ch] = gla_alpha(p, low, ch);
+}
+
+// The recurrence over a chunk of tokens in registers.  A thread owns 16 key channels x 4 value columns of the state, G lanes
+// share a column group.  The channels of lane g are 4 (i G + g) + j, so that the lanes' float4 reads of a token's q, k and
+// decay are consecutive.  kOut = false: the chunk's end state from a zero start, and the product of its decays.
+// kOut = true: outputs from the state in front of the chunk; the last chunk leaves the sequence's state.
+constexpr int kGlaThreads = 128;
+constexpr int kGlaStage = 16;  // tokens staged in shared memory at a time
+
+template <bool kOut>
+__global__ void __launch_bounds__(kGlaThreads) lb_gla_chunk_kernel(const LbGla p, int T, int C, int G, const float* __restrict__ alpha,
+                                                                   float* chunk_state, float* chunk_decay, int fresh) {
+    extern __shared__ __align__(16) float sm[];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int h = blockIdx.y, ch = blockIdx.z, tid = threadIdx.x;
+    const int HD = p.heads * p.dim, HV = p.heads * p.vdim, DP = 16 * G, cols = 4 * (kGlaThreads / G);
+    const int g = tid % G, v0 = blockIdx.x * cols + (tid / G) * 4;
+    float *sq = sm, *sk = sq + kGlaStage * DP, *sa = sk + kGlaStage * DP, *sv = sa + kGlaStage * DP;
+    const int t0 = ch * C, t1 = min(T, t0 + C);
+    const size_t mat = (size_t)p.dim * p.vdim;
+    float s[16][4];
+    const bool one = gridDim.z == 1;
+    const float* Sin = one ? p.state + (size_t)h * mat : chunk_state + ((size_t)ch * p.heads + h) * mat;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const int d = 4 * ((i >> 2) * G + g) + (i & 3);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) s[i][c] = kOut && !(one && fresh) && d < p.dim && v0 + c < p.vdim ? Sin[(size_t)d * p.vdim + v0 + c] : 0.f;
+    }
+    float decay = 1.f;
+    for (int ts = t0; ts < t1; ts += kGlaStage) {
+        const int n = min(kGlaStage, t1 - ts);
+        __syncthreads();
+        for (int i = tid; i < n * DP; i += kGlaThreads) {
+            const int t = i / DP, d = i - t * DP;
+            const float* row = p.proj + (size_t)(ts + t) * p.ldp;
+            const bool ok = d < p.dim;
+            if (kOut) sq[i] = ok ? row[h * p.dim + d] * p.qscale : 0.f;
+            sk[i] = ok ? row[HD + h * p.dim + d] : 0.f;
+            sa[i] = ok ? alpha[(size_t)(ts + t) * HD + h * p.dim + d] : 0.f;
+        }
+        for (int i = tid; i < n * cols; i += kGlaThreads) {
+            const int t = i / cols, v = blockIdx.x * cols + (i - t * cols);
+            sv[i] = v < p.vdim ? p.proj[(size_t)(ts + t) * p.ldp + 2 * HD + h * p.vdim + v] : 0.f;
+        }
+        __syncthreads();
+        for (int t = 0; t < n; ++t) {
+            const float4 v4 = *reinterpret_cast<const float4*>(sv + t * cols + (tid / G) * 4);
+            const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
+            float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int i4 = 0; i4 < 4; ++i4) {
+                const int at = t * DP + 4 * (i4 * G + g);
+                const float4 k4 = *reinterpret_cast<const float4*>(sk + at), a4 = *reinterpret_cast<const float4*>(sa + at);
+                const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, aa[4] = {a4.x, a4.y, a4.z, a4.w};
+                float qq[4];
+                if (kOut) {
+                    const float4 q4 = *reinterpret_cast<const float4*>(sq + at);
+                    qq[0] = q4.x;
+                    qq[1] = q4.y;
+                    qq[2] = q4.z;
+                    qq[3] = q4.w;
+                }
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) {
+                        float& st = s[i4 * 4 + j][c];
+                        st = fmaf(aa[j], st, kk[j] * vv[c]);
+                        if (kOut) o[c] = fmaf(qq[j], st, o[c]);
+                    }
+            }
+            if (kOut) {
+                for (int off = 1; off < G; off <<= 1) {
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) o[c] += __shfl_xor_sync(0xffffffffu, o[c], off);
+                }
+                if (g == 0) {
+                    float* out = p.o + (size_t)(ts + t) * HV + h * p.vdim;
+#pragma unroll
+                    for (int c = 0; c < 4; ++c)
+                        if (v0 + c < p.vdim) out[v0 + c] = o[c];
+                }
+            }
+        }
+        if (!kOut && blockIdx.x == 0)
+            for (int d = tid, q = 0; d < p.dim && q < 1; d += kGlaThreads, ++q)
+                for (int t = 0; t < n; ++t) decay *= sa[t * DP + d];
+    }
+    if (!kOut && blockIdx.x == 0) {
+        float* dec = chunk_decay + ((size_t)ch * p.heads + h) * p.dim;
+        if (tid < p.dim) dec[tid] = decay;
+        for (int d = tid + kGlaThreads; d < p.dim; d += kGlaThreads) {  // channels beyond one per thread: straight from memory
+            float a = 1.f;
+            for (int t = t0; t < t1; ++t) a *= alpha[(size_t)t * HD + h * p.dim + d];
+            dec[d] = a;
+        }
+    }
+    if (!kOut || ch == (int)gridDim.z - 1) {
+        float* Sout = kOut ? p.state + (size_t)h * mat : chunk_state + ((size_t)ch * p.heads + h) * mat;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            const int d = 4 * ((i >> 2) * G + g) + (i & 3);
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+                if (d < p.dim && v0 + c < p.vdim) Sout[(size_t)d * p.vdim + v0 + c] = s[i][c];
+        }
+    }
+}
+
+// chunk end states (from zero) -> state in front of every chunk, in place
+__global__ void __launch_bounds__(256) lb_gla_scan_kernel(const LbGla p, int chunks, float* chunk_state, const float* chunk_decay, int fresh) {
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const size_t all = (size_t)p.heads * p.dim * p.vdim, i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= all) return;
+    const int hd = (int)(i / p.vdim);  // head * dim + channel
+    float s = fresh ? 0.f : p.state[i];
+    for (int c = 0; c < chunks; ++c) {
+        const float end = chunk_state[(size_t)c * all + i];
+        chunk_state[(size_t)c * all + i] = s;
+        s = fmaf(chunk_decay[(size_t)c * p.heads * p.dim + hd], s, end);
+    }
+}
+
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_gated_heads_kernel(const float* __restrict__ o, const float* __restrict__ gate, int ldg, int heads, int vdim,
+                                                             const float* __restrict__ w, float eps, int slices, uint8_t* __restrict__ img) {
+    extern __shared__ float s_r[];
+    constexpr int C = LbElem<WT>::kChunk;
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, HV = heads * vdim;
+    const float* row = o + (size_t)t * HV;
+    for (int h = warp; h < heads; h += 8) {
+        const float r = row_rstd(row + (size_t)h * vdim, vdim, eps, lane);
+        if (lane == 0) s_r[h] = r;
+    }
+    __syncthreads();
+    for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
+        float f[C];
+#pragma unroll
+        for (int e = 0; e < C; ++e) {
+            const int k = c * C + e;
+            f[e] = 0.f;
+            if (k < HV) {
+                const int h = k / vdim;
+                f[e] = row[k] * s_r[h] * w[k - h * vdim] * lb_siluf(gate[(size_t)t * ldg + k]);
+            }
+        }
+        *reinterpret_cast<uint4*>(img + lb_img_chunk(t, c, slices)) = lb_pack_chunk<WT>(f);
+    }
+}
+
+// ---- latent attention ---------------------------------------------------------------------------------------------
+
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_latent_store_kernel(const LbLatent p, const float* __restrict__ raw, int ldr, const float* __restrict__ w, float eps) {
+    constexpr int C = LbElem<WT>::kChunk;
+    __shared__ float red[8];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = blockIdx.x;
+    const int pos = p.pos ? p.pos[t] : p.pos0 + t, lane = p.pos ? p.lane0 + t : p.lane0;
+    if (pos >= p.max_seq) return;
+    const float* row = raw + (size_t)t * ldr;
+    float ss = 0.f;
+    for (int k = threadIdx.x; k < p.rank; k += blockDim.x) ss = fmaf(row[k], row[k], ss);
+    ss = lb_block_sumf(ss, red);
+    const float r = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)p.rank), eps)));
+    uint8_t* img = p.cache + (size_t)lane * p.lane_bytes;
+    for (int c = threadIdx.x; c < p.slices * 8; c += blockDim.x) {
+        float f[C];
+#pragma unroll
+        for (int e = 0; e < C; ++e) f[e] = c * C + e < p.rank ? row[c * C + e] * r * w[c * C + e] : 0.f;
+        *reinterpret_cast<uint4*>(img + lb_img_chunk(pos, c, p.slices)) = lb_pack_chunk<WT>(f);
+    }
+}
+
+// CTA = (32 chunks of the latent, head, token): thread = (row % 8, chunk), the rows of the head in groups of eight
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_absorb_q_kernel(const LbLatent p, float* __restrict__ ql) {
+    extern __shared__ float sm[];
+    constexpr int C = LbElem<WT>::kChunk;
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int h = blockIdx.y, t = blockIdx.z;
+    const int r8 = threadIdx.x & 7, chunk = blockIdx.x * 32 + (threadIdx.x >> 3);
+    float* sq = sm;  // [dim]
+    for (int d = threadIdx.x; d < p.dim; d += blockDim.x) sq[d] = p.q[(size_t)t * p.ldq + h * p.dim + d] * p.scale;
+    __syncthreads();
+    float acc[C];
+#pragma unroll
+    for (int e = 0; e < C; ++e) acc[e] = 0.f;
+    if (chunk < p.slices * 8) {
+#pragma unroll 4
+        for (int d = r8; d < p.dim; d += 8) {
+            float f[C];
+            lb_unpack_chunk<WT>(__ldg(reinterpret_cast<const uint4*>(p.uk + lb_img_chunk(h * p.dim + d, chunk, p.slices))), f);
+#pragma unroll
+            for (int e = 0; e < C; ++e) acc[e] = fmaf(sq[d], f[e], acc[e]);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < C; ++e) {
+        acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], 1);
+        acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], 2);
+        acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], 4);
+    }
+    if (r8 == 0 && chunk < p.slices * 8) {
+        float* out = ql + ((size_t)t * p.heads + h) * p.rank;
+#pragma unroll
+        for (int e = 0; e < C; ++e)
+            if (chunk * C + e < p.rank) out[chunk * C + e] = acc[e];
+    }
+}
+
+// CTA = (32 value rows, head, token): a warp per row
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_absorb_v_kernel(const LbLatent p, const float* __restrict__ ol, float* __restrict__ out, int ldo) {
+    extern __shared__ float sm[];
+    constexpr int C = LbElem<WT>::kChunk;
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int h = blockIdx.y, t = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float* row = ol + ((size_t)t * p.heads + h) * p.rank;
+    for (int k = threadIdx.x; k < p.slices * 8 * C; k += blockDim.x) sm[k] = k < p.rank ? row[k] : 0.f;
+    __syncthreads();
+    for (int i = warp; i < 32; i += 8) {
+        const int v = blockIdx.x * 32 + i;
+        if (v >= p.vdim) break;
+        float a = 0.f;
+        for (int c = lane; c < p.slices * 8; c += 32) {
+            float f[C];
+            lb_unpack_chunk<WT>(__ldg(reinterpret_cast<const uint4*>(p.uv + lb_img_chunk(h * p.vdim + v, c, p.slices))), f);
+#pragma unroll
+            for (int e = 0; e < C; ++e) a = fmaf(f[e], sm[c * C + e], a);
+        }
+        a = lb_warp_sumf(a);
+        if (lane == 0) out[(size_t)t * ldo + h * p.vdim + v] = a;
+    }
+}
+
+// One CTA per (head, token), any precision: tiles of 256 positions, a thread per position for the scores, then a thread per
+// (latent chunk, position group) for the weighted sum; running maximum and sum over the tiles.
+constexpr int kLatTile = 256;
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_latent_attn_kernel(const LbLatent p, const float* __restrict__ ql, float* __restrict__ ol, int PG) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int C = LbElem<WT>::kChunk;
+    __shared__ float sw[kLatTile], red[8];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, chunks = p.slices * 8;
+    const int pos = p.pos ? p.pos[t] : p.pos0 + t, seq = p.pos ? p.lane0 + t : p.lane0;
+    const uint8_t* img = p.cache + (size_t)seq * p.lane_bytes;
+    float* sq = sm;                 // [chunks * C]
+    float* so = sm + chunks * C;    // [chunks * C] (times PG for the final sum)
+    for (int k = tid; k < chunks * C; k += 256) sq[k] = k < p.rank ? ql[((size_t)t * p.heads + h) * p.rank + k] : 0.f;
+    const int pg = tid % PG, c0 = tid / PG;
+    float acc[C];
+#pragma unroll
+    for (int e = 0; e < C; ++e) acc[e] = 0.f;
+    float mx = -INFINITY, den = 0.f;
+    __syncthreads();
+    for (int j0 = 0; j0 <= pos; j0 += kLatTile) {
+        const int j = j0 + tid;
+        float sc = -INFINITY;
+        if (j <= pos) {
+            sc = 0.f;
+#pragma unroll 4
+            for (int c = 0; c < chunks; ++c) {
+                float f[C];
+                lb_unpack_chunk<WT>(*reinterpret_cast<const uint4*>(img + lb_img_chunk(j, c, p.slices)), f);
+#pragma unroll
+                for (int e = 0; e < C; ++e) sc = fmaf(f[e], sq[c * C + e], sc);
+            }
+        }
+        float m = sc;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        if ((tid & 31) == 0) red[tid >> 5] = m;
+        __syncthreads();
+        for (int i = 0; i < 8; ++i) m = fmaxf(m, red[i]);
+        const float nm = fmaxf(mx, m), f = expf(mx - nm), w = j <= pos ? expf(sc - nm) : 0.f;
+        mx = nm;
+        sw[tid] = w;
+        den = den * f + lb_block_sumf(w, red);  // (its barriers also publish sw)
+        if (c0 < chunks) {
+#pragma unroll
+            for (int e = 0; e < C; ++e) acc[e] *= f;
+            const int n = min(kLatTile, pos + 1 - j0);
+#pragma unroll 4
+            for (int i = pg; i < n; i += PG) {
+                float c[C];
+                lb_unpack_chunk<WT>(*reinterpret_cast<const uint4*>(img + lb_img_chunk(j0 + i, c0, p.slices)), c);
+#pragma unroll
+                for (int e = 0; e < C; ++e) acc[e] = fmaf(sw[i], c[e], acc[e]);
+            }
+        }
+        __syncthreads();
+    }
+    if (c0 < chunks) {
+#pragma unroll
+        for (int e = 0; e < C; ++e) so[((size_t)pg * chunks + c0) * C + e] = acc[e];
+    }
+    __syncthreads();
+    for (int k = tid; k < p.rank; k += 256) {
+        float o = 0.f;
+        for (int g = 0; g < PG; ++g) o += so[(size_t)g * chunks * C + k];
+        ol[((size_t)t * p.heads + h) * p.rank + k] = __fdiv_rn(o, den);
+    }
+}
+
+// ---- routing ----------------------------------------------------------------------------------------------------
+
+__global__ void __launch_bounds__(256) lb_route_topk_kernel(const LbRouteBlock p) {
+    extern __shared__ float sm[];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 8 + warp;
+    if (t >= p.T) return;
+    float* row = sm + (size_t)warp * p.experts;
+    for (int e = lane; e < p.experts; e += 32) row[e] = p.logits[(size_t)t * p.ldl + e];
+    __syncwarp();
+    for (int j = 0; j < p.top; ++j) {
+        float best = -INFINITY;
+        int bi = 0x7fffffff;
+        for (int e = lane; e < p.experts; e += 32)
+            if (row[e] > best) {
+                best = row[e];
+                bi = e;
+            }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (ov > best || (ov == best && oi < bi)) {
+                best = ov;
+                bi = oi;
+            }
+        }
+        if (bi >= p.experts) bi = 0;  // only NaNs left
+        if (lane == 0) {
+            row[bi] = -INFINITY;
+            p.idx[(size_t)t * p.top + j] = bi;
+            p.score[(size_t)t * p.top + j] = lb_sigmoidf(p.logits[(size_t)t * p.ldl + bi]);
+            p.slot[(size_t)t * p.top + j] = atomicAdd(p.count + bi, 1);  // the order inside an expert does not matter: its rows are independent
+        }
+        __syncwarp();
+    }
+}
+
+__global__ void __launch_bounds__(256) lb_route_plan_kernel(const LbRouteBlock p) {
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    if (threadIdx.x == 0) {
+        int b = 0;
+        for (int e = 0; e < p.experts; ++e) {
+            p.offset[e] = b * kImgRows;
+            const int n = lb_ceil_div(p.count[e], kImgRows);
+            for (int i = 0; i < n; ++i) p.block_group[b + i] = e;
+            b += n;
+            p.count[e] = 0;  // zero between launches
+        }
+        *p.nblocks = b;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < p.T * p.top; i += blockDim.x) p.slot[i] += p.offset[p.idx[i]];
+}
+
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_route_gather_kernel(const LbRouteBlock p, const float* __restrict__ x, int ldx, int width, const float* gain,
+                                                              float eps, int slices, uint8_t* __restrict__ img) {
+    constexpr int C = LbElem<WT>::kChunk;
+    __shared__ float red[8];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = blockIdx.x;
+    const float* row = x + (size_t)t * ldx;
+    float ss = 0.f;
+    for (int k = threadIdx.x; k < width; k += blockDim.x) ss = fmaf(row[k], row[k], ss);
+    ss = lb_block_sumf(ss, red);
+    const float r = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)width), eps))) * *gain;
+    for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
+        float h[C];
+#pragma unroll
+        for (int e = 0; e < C; ++e) h[e] = c * C + e < width ? row[c * C + e] * r : 0.f;
+        for (int j = 0; j < p.top; ++j) {
+            const float w = p.score[(size_t)t * p.top + j];
+            float f[C];
+#pragma unroll
+            for (int e = 0; e < C; ++e) f[e] = w * h[e];
+            *reinterpret_cast<uint4*>(img + lb_img_chunk(p.slot[(size_t)t * p.top + j], c, slices)) = lb_pack_chunk<WT>(f);
+        }
+    }
+}
+
+__global__ void __launch_bounds__(256) lb_route_combine_kernel(const LbRouteBlock p, const float* __restrict__ y, int ldy, float mult, int width,
+                                                               float* __restrict__ x, int ldx) {
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = blockIdx.x;
+    for (int k = threadIdx.x; k < width; k += blockDim.x) {
+        float a = 0.f;
+        for (int j = 0; j < p.top; ++j) a += y[(size_t)p.slot[(size_t)t * p.top + j] * ldy + k];
+        float* o = x + (size_t)t * ldx + k;
+        *o = fmaf(mult, a, *o);
+    }
+}
+
+bool bf16(int dtype) { return dtype == LOOM_B200_DTYPE_BF16; }
+#define LB_TYPED(dtype, kern_f, kern_b, grid, block, smem, ...)         \
+    do {                                                                \
+        if (bf16(dtype))                                                \
+            LB_LAUNCH(ctx, kern_b, grid, block, smem, __VA_ARGS__);     \
+        else                                                            \
+            LB_LAUNCH(ctx, kern_f, grid, block, smem, __VA_ARGS__);     \
+    } while (0)
+
+}  // namespace
+
+int lb_embed_norm(loom_b200_ctx* ctx, int dtype, const void* table, int vocab, int width, const int* tok, int n, const float* gain, float eps,
+                  float* x, int ldx) {
+    if (bf16(dtype))
+        LB_LAUNCH(ctx, lb_embed_norm_kernel<__nv_bfloat16>, dim3(n), dim3(256), 0, static_cast<const __nv_bfloat16*>(table), vocab, width, tok, gain, eps, x, ldx);
+    else
+        LB_LAUNCH(ctx, lb_embed_norm_kernel<float>, dim3(n), dim3(256), 0, static_cast<const float*>(table), vocab, width, tok, gain, eps, x, ldx);
+    return 0;
+}
+
+int lb_norm_block(loom_b200_ctx* ctx, int dtype, const LbNormBlock& p) {
+    LB_REQUIRE(ctx, p.taps >= 1 && p.taps <= kMaxTaps, "norm_block: %d taps (1..%d)", p.taps, kMaxTaps);
+    LB_TYPED(dtype, lb_norm_block_kernel<float>, lb_norm_block_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.T, kNormTokens)), dim3(256), 0, p);
+    return 0;
+}
+
+int lb_conv_commit(loom_b200_ctx* ctx, const LbNormBlock& p) {
+    if (p.taps < 2) return 0;
+    LB_LAUNCH(ctx, lb_conv_commit_kernel, dim3(p.taps - 1), dim3(256), 0, p);
+    return 0;
+}
+
+int lb_rows_image(loom_b200_ctx* ctx, int dtype, const float* x, int ldx, int T, int cols, int slices, uint8_t* img) {
+    LB_TYPED(dtype, lb_rows_image_kernel<float>, lb_rows_image_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, x, ldx, cols, slices, img);
+    return 0;
+}
+
+int lb_gla_step(loom_b200_ctx* ctx, const LbGla& p, const int* pos, int lane0, int M) {
+    const size_t smem = (size_t)(3 * p.dim + p.rank) * sizeof(float);
+    LB_REQUIRE(ctx, smem <= 48 * 1024, "gla: %d key channels, decay rank %d", p.dim, p.rank);
+    LB_LAUNCH(ctx, lb_gla_step_kernel, dim3(lb_ceil_div(p.vdim, 32), p.heads, M), dim3(256), smem, p, pos, lane0);
+    return 0;
+}
+
+int lb_gla_block(loom_b200_ctx* ctx, const LbGla& p, int T, int pos0, float* alpha, float* chunk_state, float* chunk_decay) {
+    int G = 1;
+    while (16 * G < p.dim) G *= 2;
+    LB_REQUIRE(ctx, G <= 32, "gla: %d key channels (at most 512)", p.dim);
+    const int cols = 4 * (kGlaThreads / G), vt = lb_ceil_div(p.vdim, cols);
+    // chunks: long ones unless they leave the device half empty
+    const int C = (long long)vt * p.heads * lb_ceil_div(T, kGlaChunk) >= 2 * ctx->sm_count ? kGlaChunk : kGlaChunk / 2;
+    const int chunks = lb_ceil_div(T, C), fresh = pos0 == 0 ? 1 : 0;
+    LB_LAUNCH(ctx, lb_gla_decay_kernel, dim3(T), dim3(256), (size_t)p.rank * sizeof(float), p, alpha);
+    const size_t smem = (size_t)kGlaStage * (3 * 16 * G + cols) * sizeof(float);
+    LB_REQUIRE(ctx, smem <= 200 * 1024, "gla: %d key channels", p.dim);
+    if (smem > 48 * 1024) {
+        LB_BIG_SMEM(ctx, lb_gla_chunk_kernel<true>, 200 * 1024);
+        LB_BIG_SMEM(ctx, lb_gla_chunk_kernel<false>, 200 * 1024);
+    }
+    const dim3 grid(vt, p.heads, chunks);
+    if (chunks > 1) {
+        LB_LAUNCH(ctx, lb_gla_chunk_kernel<false>, grid, dim3(kGlaThreads), smem, p, T, C, G, alpha, chunk_state, chunk_decay, fresh);
+        const size_t all = (size_t)p.heads * p.dim * p.vdim;
+        LB_LAUNCH(ctx, lb_gla_scan_kernel, dim3((unsigned)((all + 255) / 256)), dim3(256), 0, p, chunks, chunk_state, chunk_decay, fresh);
+    }
+    LB_LAUNCH(ctx, lb_gla_chunk_kernel<true>, grid, dim3(kGlaThreads), smem, p, T, C, G, alpha, chunk_state, chunk_decay, fresh);
+    return 0;
+}
+
+int lb_gated_heads_image(loom_b200_ctx* ctx, int dtype, const float* o, const float* gate, int ldg, int T, int heads, int vdim, const float* head_w,
+                         float eps, int slices, uint8_t* img) {
+    LB_TYPED(dtype, lb_gated_heads_kernel<float>, lb_gated_heads_kernel<__nv_bfloat16>, dim3(T), dim3(256), (size_t)heads * sizeof(float), o, gate, ldg,
+             heads, vdim, head_w, eps, slices, img);
+    return 0;
+}
+
+int lb_latent_store(loom_b200_ctx* ctx, int dtype, const LbLatent& p, const float* raw, int ldr, const float* weight, float eps, int tokens) {
+    LB_TYPED(dtype, lb_latent_store_kernel<float>, lb_latent_store_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, p, raw, ldr, weight, eps);
+    return 0;
+}
+
+int lb_latent_absorb_q(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tokens, float* ql) {
+    LB_REQUIRE(ctx, p.dim <= 8192, "latent attention: query dimension %d", p.dim);
+    LB_TYPED(dtype, lb_absorb_q_kernel<float>, lb_absorb_q_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.slices * 8, 32), p.heads, tokens), dim3(256),
+             (size_t)p.dim * sizeof(float), p, ql);
+    return 0;
+}
+
+int lb_latent_absorb_v(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tokens, const float* ol, float* out, int ldo) {
+    const size_t smem = (size_t)p.slices * lb_slice_cols(dtype) * sizeof(float);
+    LB_REQUIRE(ctx, smem <= 48 * 1024, "latent attention: latent size %d", p.rank);
+    LB_TYPED(dtype, lb_absorb_v_kernel<float>, lb_absorb_v_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.vdim, 32), p.heads, tokens), dim3(256), smem, p, ol, out, ldo);
+    return 0;
+}
+
+int lb_latent_attention(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tokens, const float* ql, float* ol) {
+    const int chunks = p.slices * 8;
+    LB_REQUIRE(ctx, chunks <= 256, "latent attention: latent size %d", p.rank);
+    int PG = 1;
+    while (PG * 2 * chunks <= 256) PG *= 2;
+    const size_t smem = (size_t)chunks * (16 / (bf16(dtype) ? 2 : 4)) * (1 + PG) * sizeof(float);
+    LB_TYPED(dtype, lb_latent_attn_kernel<float>, lb_latent_attn_kernel<__nv_bfloat16>, dim3(p.heads, tokens), dim3(256), smem, p, ql, ol, PG);
+    return 0;
+}
+
+int lb_route_block(loom_b200_ctx* ctx, const LbRouteBlock& p) {
+    const size_t smem = (size_t)8 * p.experts * sizeof(float);
+    LB_REQUIRE(ctx, smem <= 48 * 1024, "routing: %d experts", p.experts);
+    LB_LAUNCH(ctx, lb_route_topk_kernel, dim3(lb_ceil_div(p.T, 8)), dim3(256), smem, p);
+    LB_LAUNCH(ctx, lb_route_plan_kernel, dim3(1), dim3(256), 0, p);
+    return 0;
+}
+
+int lb_route_gather(loom_b200_ctx* ctx, int dtype, const LbRouteBlock& p, const float* x, int ldx, int width, const float* gain, float eps, int slices,
+                    uint8_t* img) {
+    LB_TYPED(dtype, lb_route_gather_kernel<float>, lb_route_gather_kernel<__nv_bfloat16>, dim3(p.T), dim3(256), 0, p, x, ldx, width, gain, eps, slices, img);
+    return 0;
+}
+
+int lb_route_combine(loom_b200_ctx* ctx, const LbRouteBlock& p, const float* y, int ldy, float mult, int width, float* x, int ldx) {
+    LB_LAUNCH(ctx, lb_route_combine_kernel, dim3(p.T), dim3(256), 0, p, y, ldy, mult, width, x, ldx);
+    return 0;
+}
