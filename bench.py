@@ -104,7 +104,7 @@ def algorithmic_bytes(shape, ctx_len):
     return ternary, kv, head
 
 
-def build_model(ctx, torch, shape, seed):
+def build_model(ctx, torch, shape, seed, batch=1):
     from loom_b200 import cabi
     dev = torch.device("cuda", ctx.device)
     g = torch.Generator(device=dev)
@@ -114,6 +114,8 @@ def build_model(ctx, torch, shape, seed):
     dims = ((qd, H), (kvd, H), (kvd, H), (H, qd), (I, H), (I, H), (H, I))
     dec = cabi.Decoder(ctx, shape["layers"], H, shape["heads"], shape["kv_heads"], hd, I, shape["vocab"], shape["eps"],
                        shape["theta"], cabi.ACT_SILU, shape["max_seq_len"])
+    if batch > 1:
+        dec.set_batch(batch)
     weights = []
     for b in range(shape["layers"]):
         ws = []
@@ -775,6 +777,150 @@ def batch_mode(args):
     return 0
 
 
+# Layer stacks (`--mode stack`): a Zitupel of each size beside a ternary decoder of the same width, depth, vocabulary and -- for the
+# dense size -- feed-forward.  Every fourth layer is latent attention, and every second of those reads the latents of the one before.
+STACK_SHAPES = {
+    "2b": dict(layers=8, width=2560, vocab=128256, gla=(10, 128, 256, 16), latent=(20, 128, 128, 512), ff=6912, experts=0, top=0,
+               ternary=dict(heads=20, kv_heads=5, inter=6912)),
+    "8b": dict(layers=8, width=4096, vocab=128256, gla=(16, 128, 256, 16), latent=(32, 128, 128, 512), ff=14336, experts=0, top=0,
+               ternary=dict(heads=32, kv_heads=8, inter=14336)),
+    "8b-moe": dict(layers=8, width=4096, vocab=128256, gla=(16, 128, 256, 16), latent=(32, 128, 128, 512), ff=1792, experts=32, top=4,
+                   ternary=dict(heads=32, kv_heads=8, inter=7168)),  # the experts a token goes through add up to inter
+}
+
+
+def stack_config(sh):
+    layers, last = [], None
+    for i in range(sh["layers"]):
+        mlp = {"kind": "dense", "ff": sh["ff"]}
+        if sh["experts"]:
+            mlp = {"kind": "moe", "expert": {"ff": sh["ff"], "limit": 7.0}, "router": {"experts": sh["experts"], "top": sh["top"]}}
+        if i % 4 == 3:
+            h, dim, vdim, rank = sh["latent"]
+            m = {"heads": h, "dim": dim, "vdim": vdim, "kv_rank": rank, "scale": dim ** -0.5}
+            if last is not None:
+                m["kv_from"], last = last, None
+            else:
+                last = i
+            layers.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+        else:
+            h, dim, vdim, _ = sh["gla"]
+            layers.append({"type": "gla", "mixer": {"heads": h, "dim": dim, "vdim": vdim, "tau": 16.0}, "mlp": mlp})
+    return {"architecture": "Zitupel", "canon": {"taps": 4}, "layers": layers, "norm": {"eps": 1e-5}, "residual_mult": 0.7,
+            "vocab": sh["vocab"], "width": sh["width"]}
+
+
+class RandomWeights:
+    """Seeded random tensors under a checkpoint's interface, made on the device as they are asked for."""
+
+    def __init__(self, torch, device, sizes, seed):
+        self.torch, self.dev, self.sizes = torch, device, sizes
+        self.g = torch.Generator(device=device)
+        self.g.manual_seed(seed)
+
+    def shape(self, name):
+        return self.sizes[name.rsplit(".", 1)[-1]]
+
+    def raw(self, name, shape):
+        from loom_b200 import cabi
+        t = self.torch.randn(*shape, device=self.dev, generator=self.g, dtype=self.torch.float32) * shape[-1] ** -0.5
+        t = t.to(self.torch.bfloat16)
+        self.torch.cuda.synchronize(self.dev)  # the library copies on a stream of its own
+        return t, cabi.DTYPE_BF16
+
+    def f32(self, name, shape):
+        t = self.torch.randn(*shape, device=self.dev, generator=self.g, dtype=self.torch.float32) * 0.1
+        return (t + (1.0 if name.endswith("norm") else 3.0 if name.endswith(".b") else 0.0)).cpu().numpy()
+
+    def scalar(self, name):
+        return 1.0
+
+
+def stack_measure(torch, ctx, dec, vocab, prompt_len, steps, warmup, batch, reps):
+    """Prompt and decode rates of any decoder: CUDA events on the context's stream, `reps` prompts per sequence slot, then K greedy
+    steps of every sequence together."""
+    rng = np.random.default_rng(5)
+    s = torch.cuda.ExternalStream(ctx.stream)
+
+    def timed(fn):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        ctx.sync()
+        e0.record(s)
+        fn()
+        e1.record(s)
+        ctx.sync()
+        return e0.elapsed_time(e1)
+
+    prompts = [rng.integers(0, vocab, prompt_len).astype(np.int32) for _ in range(batch)]
+
+    def prompt(i):
+        dec.select(i)
+        dec.reset()
+        dec.extend(prompts[i])
+
+    prompt(0)
+    prompt(0)
+    pf = [timed(lambda: prompt(0)) for _ in range(reps)]
+    for i in range(batch):
+        prompt(i)
+    go = dec.continue_greedy if batch == 1 else dec.continue_batch
+    go(warmup)
+    dc = [timed(lambda: go(steps)) / steps for _ in range(reps)]
+    return float(np.median(pf)), float(np.median(dc))
+
+
+def stack_mode(args):
+    """A layer stack and a ternary decoder of equal size, one after the other on one GPU: prompt tok/s and greedy decode tok/s for
+    one and for `--batch` sequences.  The value is the stack's batch-1 decode rate."""
+    import torch
+
+    import loom_b200
+    from loom_b200 import cabi, models
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    steps, warm, reps = args.steps, max(args.warmup, 3), max(args.reps, 1)
+    sh = dict(STACK_SHAPES[args.stack_shape])
+    if args.layers != SHAPE["layers"]:
+        sh["layers"] = args.layers
+    if args.vocab != SHAPE["vocab"]:
+        sh["vocab"] = args.vocab
+    msl = args.prompt + warm + steps * reps + 8
+    clocks = ClockSampler(0)
+    clocks.start()
+    out, launches = {}, 0
+    for batch in sorted({1, args.batch}):
+        for kind in ("stack", "ternary"):
+            if args.only and kind != args.only:
+                continue
+            ctx = loom_b200.Context(0)
+            apply_opts(ctx, args)
+            if kind == "stack":
+                dec = models.build(ctx, stack_config(sh), RandomWeights(torch, dev, {"a1": (sh["gla"][3], sh["width"])}, args.seed),
+                                   models.LoadOptions(cabi.DTYPES[args.dtype], msl, batch))
+                keep = None
+            else:
+                t = sh["ternary"]
+                shape = dict(layers=sh["layers"], hidden=sh["width"], heads=t["heads"], kv_heads=t["kv_heads"], head_dim=sh["width"] // t["heads"],
+                             inter=t["inter"], vocab=sh["vocab"], eps=1e-5, theta=500000.0, max_seq_len=msl)
+                dec, *keep = build_model(ctx, torch, shape, args.seed, batch)
+            pf, dc = stack_measure(torch, ctx, dec, sh["vocab"], args.prompt, steps, warm, batch, reps)
+            launches += ctx.launch_count
+            out.setdefault(kind, {})["batch%d" % batch] = {"prompt_ms": pf, "prompt_tok_per_s": args.prompt / pf * 1e3, "step_ms": dc,
+                                                           "decode_tok_per_s": batch / dc * 1e3}
+            dec.close()
+            del dec, keep
+            ctx.close()
+            torch.cuda.empty_cache()
+    first = out.get("stack", out.get("ternary"))["batch1"]
+    print(json.dumps({"metric": "decode tok/s (Zitupel, %s-shape layers, bs=1) beside a ternary decoder of equal size" % args.stack_shape,
+                      "value": first["decode_tok_per_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warm, "ms_per_step": first["step_ms"],
+                      "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": args.dtype, "data": "synthetic",
+                      "config": {"shape": args.stack_shape, "layers": sh["layers"], "width": sh["width"], "prompt": args.prompt, "vocab": sh["vocab"],
+                                 "batch": args.batch, "l2": "weights of a step exceed L2"},
+                      "rates": out, "gpu_launches": launches, "clocks": clocks.stop()}))
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -788,13 +934,17 @@ def main():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--batch", type=int, default=16, help="batch mode: independent sequences")
     ap.add_argument("--opt", action="append", default=[], help="context option key=value (repeatable), e.g. --opt tp_fused=0")
-    ap.add_argument("--mode", default="decode", choices=["decode", "gemm", "tp", "sweep", "batch"],
+    ap.add_argument("--mode", default="decode", choices=["decode", "gemm", "tp", "sweep", "batch", "stack"],
                     help="gemm: the batched-prefill GEMM microbenchmark; tp: tensor-parallel decode of --shape under torchrun; "
                          "sweep: GEMV vs GEMM over batch sizes for the gate/down projections of --shape")
     ap.add_argument("--shape", default="8b", choices=sorted(TP_SHAPES) + ["2b"])
     ap.add_argument("--tp-exchange", default="peer", choices=["peer", "nccl"],
                     help="tp mode: how the row-parallel projections exchange their partial results")
     ap.add_argument("--tokens", type=int, default=512)
+    ap.add_argument("--stack-shape", default="2b", choices=sorted(STACK_SHAPES), help="stack mode: a layer stack and a ternary decoder of equal size")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="stack mode: element type of the stack")
+    ap.add_argument("--reps", type=int, default=5, help="stack mode: repetitions of a timed region (the median counts)")
+    ap.add_argument("--only", default="", choices=["", "stack", "ternary"], help="stack mode: one of the two models (profiling)")
     ap.add_argument("--no-tp-section", action="store_true", help="multi-GPU runs: skip the tensor-parallel decode after the replica measurement")
     args = ap.parse_args()
     if args.mode == "gemm":
@@ -803,6 +953,8 @@ def main():
         return tp_mode(args)
     if args.mode == "batch":
         return batch_mode(args)
+    if args.mode == "stack":
+        return stack_mode(args)
     if args.mode == "sweep":
         args.steps = min(args.steps, 20)
         return sweep_mode(args)

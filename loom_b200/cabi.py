@@ -712,7 +712,8 @@ class Decoder:
 
     def close(self):
         if self.h:
-            lib().loom_b200_decoder_destroy(self.h)
+            if self.ctx.h:  # (a decoder must go before its context; one that did not is left to the process's end)
+                lib().loom_b200_decoder_destroy(self.h)
             self.h = None
 
     def __del__(self):

@@ -53,7 +53,7 @@ class Checkpoint:
             raise ValueError("tensor '%s' is %s, expected %s" % (name, list(a.shape), list(shape)))
         if e["dtype"] == "BF16":
             return a, cabi.DTYPE_BF16
-        return np.ascontiguousarray(a, np.float32), cabi.DTYPE_F32
+        return a.astype(np.float32, copy=False), cabi.DTYPE_F32
 
     def f32(self, name: str, shape=None) -> np.ndarray:
         a, code = self.raw(name, shape)

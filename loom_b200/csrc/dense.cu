@@ -157,11 +157,11 @@ __device__ __forceinline__ void load_batch(GemvBatch<NB>& w, const uint8_t* stri
 
 // KW warps share a strip of 16 rows by K slices, 8/KW strips run side by side in a CTA.
 template <typename WT, int PRO, int EPI>
-__global__ void __launch_bounds__(kGemvThreads) lb_dense_gemv_kernel(const LbDenseGemv p, int Mp, int KW) {
+__global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const LbDenseGemv p, int Mp, int KW, bool vec) {
     extern __shared__ __align__(16) uint8_t smem[];
     constexpr int C = LbElem<WT>::kChunk;
     constexpr bool kDual = EPI == LB_DEPI_GLU;
-    constexpr int NB = kDual ? 2 : 4;
+    constexpr int NB = kDual ? 1 : 2;
     __shared__ float red[kGemvWarps][128];
     __shared__ float red2[kDual ? kGemvWarps : 1][128];
     __shared__ float s_stat[kGemvWarps];
@@ -298,33 +298,51 @@ __global__ void __launch_bounds__(kGemvThreads) lb_dense_gemv_kernel(const LbDen
         if (PRO == LB_DPRO_CONV && live) pos = p.pos[m];
         for (int c = lt; c < chunks; c += nt) {
             float f[C];
+            const int k0 = c * C;
+            if (live && k0 < p.K) {
+                lb_load_cols<C>(xr, k0, p.K, vec, f);
+                if (PRO == LB_DPRO_NORM || PRO == LB_DPRO_CONV || PRO == LB_DPRO_MOE) {
 #pragma unroll
-            for (int i = 0; i < C; ++i) {
-                const int k = c * C + i;
-                float v = 0.f;
-                if (live && k < p.K) {
-                    if (PRO == LB_DPRO_PLAIN) v = xr[k];
-                    if (PRO == LB_DPRO_NORM) v = xr[k] * rstd * gain;
-                    if (PRO == LB_DPRO_MOE) v = s_w[m] * (xr[k] * rstd * gain);
-                    if (PRO == LB_DPRO_GATED) {
-                        const int h = k / p.head_dim;
-                        v = xr[k] * s_head[h] * p.head_w[k - h * p.head_dim] * lb_siluf(p.gate[(size_t)m * p.gate_ld + k]);
-                    }
-                    if (PRO == LB_DPRO_CONV) {
-                        const float h = xr[k] * rstd * gain;
-                        const float* cw = p.conv_w + (size_t)k * p.taps;
-                        float* ring = p.conv_ring + (size_t)seq * p.taps * p.ring_ld + k;
-                        float a = 0.f;
-                        for (int j = 0; j + 1 < p.taps; ++j) {  // tap j looks back taps - 1 - j positions
-                            const int ps = pos - (p.taps - 1) + j;
-                            if (ps >= 0) a = fmaf(cw[j], ring[(size_t)(ps % p.taps) * p.ring_ld], a);
-                        }
-                        a = fmaf(cw[p.taps - 1], h, a);
-                        if (blockIdx.x == 0) ring[(size_t)(pos % p.taps) * p.ring_ld] = h;  // no CTA of this launch reads this slot
-                        v = h + a;
+                    for (int i = 0; i < C; ++i) f[i] = f[i] * rstd * gain;
+                }
+                if (PRO == LB_DPRO_MOE) {
+#pragma unroll
+                    for (int i = 0; i < C; ++i) f[i] *= s_w[m];
+                }
+                if (PRO == LB_DPRO_GATED) {
+                    float gt[C];
+                    lb_load_cols<C>(p.gate + (size_t)m * p.gate_ld, k0, p.K, vec, gt);
+#pragma unroll
+                    for (int i = 0; i < C; ++i) {
+                        const int k = k0 + i, h = k / p.head_dim;
+                        if (k < p.K) f[i] = f[i] * s_head[h] * p.head_w[k - h * p.head_dim] * lb_siluf(gt[i]);
                     }
                 }
-                f[i] = v;
+                if (PRO == LB_DPRO_CONV) {
+                    float* ring = p.conv_ring + (size_t)seq * p.taps * p.ring_ld;
+                    float a[C], w[C], y[C];
+#pragma unroll
+                    for (int i = 0; i < C; ++i) a[i] = 0.f;
+                    for (int j = 0; j + 1 < p.taps; ++j) {  // tap j looks back taps - 1 - j positions
+                        const int ps = pos - (p.taps - 1) + j;
+                        if (ps < 0) continue;
+                        lb_load_cols<C>(p.conv_w + (size_t)j * p.ring_ld, k0, p.K, vec, w);
+                        lb_load_cols<C>(ring + (size_t)(ps % p.taps) * p.ring_ld, k0, p.K, vec, y);
+#pragma unroll
+                        for (int i = 0; i < C; ++i) a[i] = fmaf(w[i], y[i], a[i]);
+                    }
+                    lb_load_cols<C>(p.conv_w + (size_t)(p.taps - 1) * p.ring_ld, k0, p.K, vec, w);
+                    float* slot = ring + (size_t)(pos % p.taps) * p.ring_ld + k0;  // no CTA of this launch reads this slot
+#pragma unroll
+                    for (int i = 0; i < C; ++i) {
+                        a[i] = fmaf(w[i], f[i], a[i]);
+                        if (blockIdx.x == 0 && k0 + i < p.K) slot[i] = f[i];
+                        f[i] += a[i];
+                    }
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < C; ++i) f[i] = 0.f;
             }
             xs[(size_t)c * Mp + m] = lb_pack_chunk<WT>(f);
         }
@@ -341,17 +359,16 @@ __global__ void __launch_bounds__(kGemvThreads) lb_dense_gemv_kernel(const LbDen
             if (PRO != LB_DPRO_PAIRS) {
                 const uint8_t* s1 = strip_ptr(w1, strip);
                 const uint8_t* s2 = kDual ? strip_ptr(w2, strip) : nullptr;
-                const bool loaded = strip == (int)blockIdx.x * SP + sp && (kEarly || PRO == LB_DPRO_MOE);
-                if (!loaded) {
-                    load_batch(cur, s1, kw, KW, p.slices, g, t);
-                    if (kDual) load_batch(cur2, s2, kw, KW, p.slices, g, t);
-                }
+                const int next = strip + (int)gridDim.x * SP;
                 for (int s = kw; s < p.slices; s += NB * KW) {
                     GemvBatch<NB> now = cur, now2;
                     if (kDual) now2 = cur2;
                     if (s + NB * KW < p.slices) {
                         load_batch(cur, s1, s + NB * KW, KW, p.slices, g, t);
                         if (kDual) load_batch(cur2, s2, s + NB * KW, KW, p.slices, g, t);
+                    } else if (next < strips) {  // the next strip's first batch travels while this strip's sums meet
+                        load_batch(cur, strip_ptr(w1, next), kw, KW, p.slices, g, t);
+                        if (kDual) load_batch(cur2, strip_ptr(w2, next), kw, KW, p.slices, g, t);
                     }
 #pragma unroll
                     for (int u = 0; u < NB; ++u) {
@@ -429,9 +446,15 @@ int gemv_launch(loom_b200_ctx* ctx, const LbDenseGemv& p) {
     LB_REQUIRE(ctx, p.M >= 1 && p.M <= kMaxLanesPerPass, "dense_gemv: %d tokens", p.M);
     int Mp = 1;
     while (Mp < p.M) Mp *= 2;
+    const int strips = lb_ceil_div(p.rows, 16), cap = ctx->sm_count * 2;
     int KW = 1;
     while (KW < kGemvWarps && KW * 2 <= p.slices) KW *= 2;
-    const int SP = kGemvWarps / KW, strips = lb_ceil_div(p.rows, 16);
+    // many strips per CTA: fewer warps per strip, so that a warp streams longer runs between two meetings of the sums
+    while (KW > 1 && (long long)strips >= 6ll * (2 * kGemvWarps / KW) * cap) KW /= 2;
+    const int SP = kGemvWarps / KW;
+    bool vec = lb_vec_rows(p.x, p.ldx);
+    if (PRO == LB_DPRO_GATED) vec = vec && lb_vec_rows(p.gate, p.gate_ld);
+    if (PRO == LB_DPRO_CONV) vec = vec && lb_vec_rows(p.conv_w, p.ring_ld) && lb_vec_rows(p.conv_ring, p.ring_ld);
     size_t smem = PRO == LB_DPRO_PAIRS ? 0 : (size_t)p.slices * 8 * Mp * 16;
     if (PRO == LB_DPRO_MOE) smem += (size_t)p.M * p.experts * 4 + (size_t)p.M * p.top * 4;
     if (PRO == LB_DPRO_GATED) smem += (size_t)Mp * (p.K / p.head_dim) * 4;
@@ -439,9 +462,8 @@ int gemv_launch(loom_b200_ctx* ctx, const LbDenseGemv& p) {
     if (smem > 48 * 1024) LB_BIG_SMEM(ctx, (lb_dense_gemv_kernel<WT, PRO, EPI>), kGemvSmemX + 16 * 1024);
     int gx = lb_ceil_div(strips, SP);
     const int gy = PRO == LB_DPRO_MOE ? p.M * p.top : 1;
-    const int cap = ctx->sm_count * 2;
     if (gx > cap) gx = lb_ceil_div(gx, lb_ceil_div(gx, cap));  // equal numbers of strips per CTA
-    LB_LAUNCH(ctx, (lb_dense_gemv_kernel<WT, PRO, EPI>), dim3(gx, gy), dim3(kGemvThreads), smem, p, Mp, KW);
+    LB_LAUNCH(ctx, (lb_dense_gemv_kernel<WT, PRO, EPI>), dim3(gx, gy), dim3(kGemvThreads), smem, p, Mp, KW, vec);
     return 0;
 }
 
@@ -536,7 +558,11 @@ __global__ void __launch_bounds__(256) lb_dense_gemm_simt_kernel(const LbDenseGe
                 if (EPI == LB_DEPI_GELU) f[j] = lb_gelu_erff(acc[i][j]);
                 if (EPI == LB_DEPI_GLU) f[j] = lb_clamped_glu(acc[i][j], acc2[i][j], p.limit);
             }
-            if (r / LbElem<WT>::kSlice < p.img_slices) lb_img_store8<WT>(p.img, tok, r, p.img_slices, f);
+            if (EPI == LB_DEPI_HEADS) {
+                if (r < p.rows) *reinterpret_cast<uint4*>(p.img + lb_heads_chunk(tok, r, p.heads, p.head_dim, p.head_chunks)) = lb_pack_chunk<__nv_bfloat16>(f);
+            } else if (r / LbElem<WT>::kSlice < p.img_slices) {
+                lb_img_store8<WT>(p.img, tok, r, p.img_slices, f);
+            }
         }
     }
 }
@@ -557,6 +583,7 @@ int gemm_simt(loom_b200_ctx* ctx, int epi, const LbDenseGemm& p) {
     LB_CASE(LB_DEPI_GELU)
     LB_CASE(LB_DEPI_GLU)
     LB_CASE(LB_DEPI_IMG)
+    LB_CASE(LB_DEPI_HEADS)
 #undef LB_CASE
     return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "dense_gemm: epilogue %d is not built", epi);
 }

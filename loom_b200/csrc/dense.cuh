@@ -87,6 +87,30 @@ __device__ __forceinline__ void lb_img_store8(uint8_t* img, int row, int col0, i
         *reinterpret_cast<uint4*>(img + lb_img_chunk(row, col0 / C + i, slices)) = lb_pack_chunk<WT>(f + i * C);
 }
 
+// C floats of a row from column k on, zero from column n on; vec: the row starts on a 16-byte boundary
+template <int C>
+__device__ __forceinline__ void lb_load_cols(const float* row, int k, int n, bool vec, float* f) {
+    if (vec && k + C <= n) {
+#pragma unroll
+        for (int i = 0; i < C; i += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(row + k + i);
+            f[i] = v.x;
+            f[i + 1] = v.y;
+            f[i + 2] = v.z;
+            f[i + 3] = v.w;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < C; ++i) f[i] = k + i < n ? row[k + i] : 0.f;
+    }
+}
+static inline bool lb_vec_rows(const float* p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; }
+// chunk of eight columns of a token's row in the per-head blocks
+__device__ __forceinline__ size_t lb_heads_chunk(int row, int col, int heads, int head_dim, int head_chunks) {
+    const int h = col / head_dim, d = col - h * head_dim;
+    return ((size_t)(row >> 7) * heads + h) * head_chunks * 2048 + (size_t)((row & 127) >> 3) * head_chunks * 128 + (size_t)(d >> 3) * 128 + (size_t)(row & 7) * 16;
+}
+
 __device__ __forceinline__ float lb_warp_sumf(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -131,6 +155,7 @@ enum LbDenseEpi : int {
     LB_DEPI_GELU = 2,   // exact gelu (GEMV: float rows, GEMM: image)
     LB_DEPI_GLU = 3,    // clamped gated unit of two products (GEMV: rows of WT per pair, GEMM: image)
     LB_DEPI_IMG = 4,    // GEMM only: image
+    LB_DEPI_HEADS = 5,  // GEMM only: per-head blocks [token block of 128][head][token/8][chunk][token%8][16 B]
 };
 
 // What the first expert product leaves for the second: the distinct experts of this pass and, per expert and token, the
@@ -154,7 +179,7 @@ struct LbDenseGemv {
     const int* row_idx = nullptr;  // token m reads row row_idx[m] of x (null: m)
     const float* gain = nullptr;   // one float
     float eps = 0.f;
-    // convolution: weights [K][taps], ring [lane][taps][ring_ld] of normed inputs (slot = position % taps)
+    // convolution: weights [taps][ring_ld], ring [lane][taps][ring_ld] of normed inputs (slot = position % taps)
     const float* conv_w = nullptr;
     float* conv_ring = nullptr;
     int taps = 0, ring_ld = 0;
@@ -196,6 +221,7 @@ struct LbDenseGemm {
     float* out = nullptr;
     uint8_t* img = nullptr;
     int ldo = 0, img_slices = 0;
+    int heads = 0, head_dim = 0, head_chunks = 0;  // per-head blocks: head_dim % 8 == 0, head_chunks 16-byte chunks per row
     float mult = 1.f, limit = 0.f;
     int* status = nullptr;
 };

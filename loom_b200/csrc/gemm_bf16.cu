@@ -177,7 +177,7 @@ __global__ void __launch_bounds__(kThreads, 1) lb_gemm_bf16_kernel(const LbDense
                             o[1] = y;
                         }
                     } else {
-                        if (r / 64 >= p.img_slices) continue;
+                        if (EPI == LB_DEPI_HEADS ? r >= p.rows : r / 64 >= p.img_slices) continue;
                         float f[8];
 #pragma unroll
                         for (int j = 0; j < 8; ++j) {
@@ -185,7 +185,10 @@ __global__ void __launch_bounds__(kThreads, 1) lb_gemm_bf16_kernel(const LbDense
                             if (EPI == LB_DEPI_GELU) f[j] = lb_gelu_erff(v8[j]);
                             if (EPI == LB_DEPI_GLU) f[j] = lb_clamped_glu(v8[j], u8[j], p.limit);
                         }
-                        lb_img_store8<__nv_bfloat16>(p.img, tok, r, p.img_slices, f);
+                        if (EPI == LB_DEPI_HEADS)
+                            *reinterpret_cast<uint4*>(p.img + lb_heads_chunk(tok, r, p.heads, p.head_dim, p.head_chunks)) = lb_pack_chunk<__nv_bfloat16>(f);
+                        else
+                            lb_img_store8<__nv_bfloat16>(p.img, tok, r, p.img_slices, f);
                     }
                 }
             }
@@ -231,6 +234,7 @@ int lb_gemm_bf16_run(loom_b200_ctx* ctx, int epi, const LbDenseGemm& p) {
         case LB_DEPI_RESID: return launch_plain<LB_DEPI_RESID>(ctx, p);
         case LB_DEPI_GELU: return launch_plain<LB_DEPI_GELU>(ctx, p);
         case LB_DEPI_IMG: return launch_plain<LB_DEPI_IMG>(ctx, p);
+        case LB_DEPI_HEADS: return launch_plain<LB_DEPI_HEADS>(ctx, p);
         case LB_DEPI_GLU: return launch<2, LB_DEPI_GLU>(ctx, p);
     }
     return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "gemm_bf16: epilogue %d is not built", epi);

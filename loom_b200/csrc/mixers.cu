@@ -25,7 +25,7 @@ __global__ void __launch_bounds__(256) lb_embed_norm_kernel(const WT* __restrict
     for (int k = threadIdx.x; k < width; k += blockDim.x) out[k] = ok ? (float)row[k] * r : 0.f;
 }
 
-constexpr int kNormTokens = 16;  // tokens of a CTA
+constexpr int kNormTokens = 8;  // tokens of a CTA
 constexpr int kMaxTaps = 16;
 
 __device__ __forceinline__ float row_rstd(const float* row, int width, float eps, int lane) {  // a warp per row
@@ -36,7 +36,7 @@ __device__ __forceinline__ float row_rstd(const float* row, int width, float eps
 }
 
 template <typename WT>
-__global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p) {
+__global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p, bool vec) {
     constexpr int C = LbElem<WT>::kChunk;
     __shared__ float s_r[kNormTokens + kMaxTaps];
     lb_pdl_launch_dependents();
@@ -55,28 +55,29 @@ __global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p)
     __syncthreads();
     const int chunks = p.slices * 8;
     for (int i = threadIdx.x; i < (t1 - t0) * chunks; i += blockDim.x) {
-        const int tt = i / chunks, c = i - tt * chunks, t = t0 + tt;
+        const int tt = i / chunks, c = i - tt * chunks, t = t0 + tt, k0 = c * C;
         const int src = p.row_idx ? p.row_idx[t] : t;
         float f[C];
+        lb_load_cols<C>(p.x + (size_t)src * p.ldx, k0, p.width, vec, f);
 #pragma unroll
-        for (int e = 0; e < C; ++e) {
-            const int k = c * C + e;
-            f[e] = k < p.width ? p.x[(size_t)src * p.ldx + k] * s_r[tt + back] : 0.f;
-        }
-        if (p.conv_w) {
-            float a[C];
+        for (int e = 0; e < C; ++e) f[e] *= s_r[tt + back];
+        if (p.conv_w && k0 < p.width) {
+            float a[C], w[C], h[C];
 #pragma unroll
             for (int e = 0; e < C; ++e) a[e] = 0.f;
             for (int j = 0; j < p.taps; ++j) {  // tap j looks back taps - 1 - j positions
                 const int ts = t - back + j;
                 if (p.pos0 + ts < 0) continue;
+                lb_load_cols<C>(p.conv_w + (size_t)j * p.ring_ld, k0, p.width, vec, w);
+                if (ts >= 0) {
+                    lb_load_cols<C>(p.x + (size_t)ts * p.ldx, k0, p.width, vec, h);
 #pragma unroll
-                for (int e = 0; e < C; ++e) {
-                    const int k = c * C + e;
-                    if (k >= p.width) continue;
-                    const float h = ts >= 0 ? p.x[(size_t)ts * p.ldx + k] * s_r[tt + j] : p.ring[(size_t)((p.pos0 + ts) % p.taps) * p.ring_ld + k];
-                    a[e] = fmaf(p.conv_w[(size_t)k * p.taps + j], h, a[e]);
+                    for (int e = 0; e < C; ++e) h[e] *= s_r[tt + j];
+                } else {
+                    lb_load_cols<C>(p.ring + (size_t)((p.pos0 + ts) % p.taps) * p.ring_ld, k0, p.width, vec, h);
                 }
+#pragma unroll
+                for (int e = 0; e < C; ++e) a[e] = fmaf(w[e], h[e], a[e]);
             }
 #pragma unroll
             for (int e = 0; e < C; ++e) f[e] += a[e];
@@ -108,222 +109,33 @@ __global__ void __launch_bounds__(256) lb_rows_image_kernel(const float* __restr
     const int t = blockIdx.x;
     for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
         float f[C];
-#pragma unroll
-        for (int e = 0; e < C; ++e) f[e] = c * C + e < cols ? x[(size_t)t * ldx + c * C + e] : 0.f;
+        lb_load_cols<C>(x + (size_t)t * ldx, c * C, cols, ldx % 4 == 0, f);
         *reinterpret_cast<uint4*>(img + lb_img_chunk(t, c, slices)) = lb_pack_chunk<WT>(f);
     }
 }
 
-// ---- gated linear attention -------------------------------------------------------------------------------------
-
-__device__ __forceinline__ float gla_alpha(const LbGla& p, const float* low, int ch) {
-    const int hd = p.heads * p.dim;
-    float z = 0.f;
-    for (int r = 0; r < p.rank; ++r) z = fmaf(p.a2t[(size_t)r * hd + ch], low[r], z);
-    return expf(lb_log_sigmoidf(z + p.a2b[ch]) * p.inv_tau);
-}
-
-// one new token per sequence: CTA = (32 value columns, head, sequence); warps split the key channels
-__global__ void __launch_bounds__(256) lb_gla_step_kernel(const LbGla p, const int* pos, int lane0) {
-    extern __shared__ float sm[];
-    __shared__ float part[8][32];
-    lb_pdl_launch_dependents();
-    lb_pdl_wait();
-    const int h = blockIdx.y, m = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int HD = p.heads * p.dim, HV = p.heads * p.vdim;
-    float *sq = sm, *sk = sm + p.dim, *sa = sk + p.dim, *low = sa + p.dim;
-    const float* row = p.proj + (size_t)m * p.ldp;
-    for (int r = threadIdx.x; r < p.rank; r += blockDim.x) low[r] = row[2 * HD + 2 * HV + r];
-    __syncthreads();
-    for (int d = threadIdx.x; d < p.dim; d += blockDim.x) {
-        sq[d] = row[h * p.dim + d] * p.qscale;
-        sk[d] = row[HD + h * p.dim + d];
-        sa[d] = gla_alpha(p, low, h * p.dim + d);
-    }
-    __syncthreads();
-    const int v = blockIdx.x * 32 + lane;
-    const bool fresh = pos[m] == 0;
-    float acc = 0.f;
-    if (v < p.vdim) {
-        float* S = p.state + (((size_t)(lane0 + m) * p.heads + h) * p.dim) * p.vdim + v;
-        const float vv = row[2 * HD + h * p.vdim + v];
-#pragma unroll 4
-        for (int d = warp; d < p.dim; d += 8) {
-            const float old = fresh ? 0.f : S[(size_t)d * p.vdim];
-            const float s = fmaf(sa[d], old, sk[d] * vv);
-            S[(size_t)d * p.vdim] = s;
-            acc = fmaf(sq[d], s, acc);
-        }
-    }
-    part[warp][lane] = acc;
-    __syncthreads();
-    if (warp == 0 && v < p.vdim) {
-        float o = 0.f;
-#pragma unroll
-        for (int w = 0; w < 8; ++w) o += part[w][lane];
-        p.o[(size_t)m * HV + h * p.vdim + v] = o;
-    }
-}
-
-__global__ void __launch_bounds__(256) lb_gla_decay_kernel(const LbGla p, float* __restrict__ alpha) {
-    extern __shared__ float low[];
-    lb_pdl_launch_dependents();
-    lb_pdl_wait();
-    const int t = blockIdx.x, HD = p.heads * p.dim, HV = p.heads * p.vdim;
-    const float* row = p.proj + (size_t)t * p.ldp + 2 * HD + 2 * HV;
-    for (int r = threadIdx.x; r < p.rank; r += blockDim.x) low[r] = row[r];
-    __syncthreads();
-    for (int ch = threadIdx.x; ch < HD; ch += blockDim.x) alpha[(size_t)t * HD + ch] = gla_alpha(p, low, ch);
-}
-
-// The recurrence over a chunk of tokens in registers.  A thread owns 16 key channels x 4 value columns of the state, G lanes
-// share a column group.  The channels of lane g are 4 (i G + g) + j, so that the lanes' float4 reads of a token's q, k and
-// decay are consecutive.  kOut = false: the chunk's end state from a zero start, and the product of its decays.
-// kOut = true: outputs from the state in front of the chunk; the last chunk leaves the sequence's state.
-constexpr int kGlaThreads = 128;
-constexpr int kGlaStage = 16;  // tokens staged in shared memory at a time
-
-template <bool kOut>
-__global__ void __launch_bounds__(kGlaThreads) lb_gla_chunk_kernel(const LbGla p, int T, int C, int G, const float* __restrict__ alpha,
-                                                                   float* chunk_state, float* chunk_decay, int fresh) {
-    extern __shared__ __align__(16) float sm[];
-    lb_pdl_launch_dependents();
-    lb_pdl_wait();
-    const int h = blockIdx.y, ch = blockIdx.z, tid = threadIdx.x;
-    const int HD = p.heads * p.dim, HV = p.heads * p.vdim, DP = 16 * G, cols = 4 * (kGlaThreads / G);
-    const int g = tid % G, v0 = blockIdx.x * cols + (tid / G) * 4;
-    float *sq = sm, *sk = sq + kGlaStage * DP, *sa = sk + kGlaStage * DP, *sv = sa + kGlaStage * DP;
-    const int t0 = ch * C, t1 = min(T, t0 + C);
-    const size_t mat = (size_t)p.dim * p.vdim;
-    float s[16][4];
-    const bool one = gridDim.z == 1;
-    const float* Sin = one ? p.state + (size_t)h * mat : chunk_state + ((size_t)ch * p.heads + h) * mat;
-#pragma unroll
-    for (int i = 0; i < 16; ++i) {
-        const int d = 4 * ((i >> 2) * G + g) + (i & 3);
-#pragma unroll
-        for (int c = 0; c < 4; ++c) s[i][c] = kOut && !(one && fresh) && d < p.dim && v0 + c < p.vdim ? Sin[(size_t)d * p.vdim + v0 + c] : 0.f;
-    }
-    float decay = 1.f;
-    for (int ts = t0; ts < t1; ts += kGlaStage) {
-        const int n = min(kGlaStage, t1 - ts);
-        __syncthreads();
-        for (int i = tid; i < n * DP; i += kGlaThreads) {
-            const int t = i / DP, d = i - t * DP;
-            const float* row = p.proj + (size_t)(ts + t) * p.ldp;
-            const bool ok = d < p.dim;
-            if (kOut) sq[i] = ok ? row[h * p.dim + d] * p.qscale : 0.f;
-            sk[i] = ok ? row[HD + h * p.dim + d] : 0.f;
-            sa[i] = ok ? alpha[(size_t)(ts + t) * HD + h * p.dim + d] : 0.f;
-        }
-        for (int i = tid; i < n * cols; i += kGlaThreads) {
-            const int t = i / cols, v = blockIdx.x * cols + (i - t * cols);
-            sv[i] = v < p.vdim ? p.proj[(size_t)(ts + t) * p.ldp + 2 * HD + h * p.vdim + v] : 0.f;
-        }
-        __syncthreads();
-        for (int t = 0; t < n; ++t) {
-            const float4 v4 = *reinterpret_cast<const float4*>(sv + t * cols + (tid / G) * 4);
-            const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
-            float o[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int i4 = 0; i4 < 4; ++i4) {
-                const int at = t * DP + 4 * (i4 * G + g);
-                const float4 k4 = *reinterpret_cast<const float4*>(sk + at), a4 = *reinterpret_cast<const float4*>(sa + at);
-                const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, aa[4] = {a4.x, a4.y, a4.z, a4.w};
-                float qq[4];
-                if (kOut) {
-                    const float4 q4 = *reinterpret_cast<const float4*>(sq + at);
-                    qq[0] = q4.x;
-                    qq[1] = q4.y;
-                    qq[2] = q4.z;
-                    qq[3] = q4.w;
-                }
-#pragma unroll
-                for (int j = 0; j < 4; ++j)
-#pragma unroll
-                    for (int c = 0; c < 4; ++c) {
-                        float& st = s[i4 * 4 + j][c];
-                        st = fmaf(aa[j], st, kk[j] * vv[c]);
-                        if (kOut) o[c] = fmaf(qq[j], st, o[c]);
-                    }
-            }
-            if (kOut) {
-                for (int off = 1; off < G; off <<= 1) {
-#pragma unroll
-                    for (int c = 0; c < 4; ++c) o[c] += __shfl_xor_sync(0xffffffffu, o[c], off);
-                }
-                if (g == 0) {
-                    float* out = p.o + (size_t)(ts + t) * HV + h * p.vdim;
-#pragma unroll
-                    for (int c = 0; c < 4; ++c)
-                        if (v0 + c < p.vdim) out[v0 + c] = o[c];
-                }
-            }
-        }
-        if (!kOut && blockIdx.x == 0)
-            for (int d = tid, q = 0; d < p.dim && q < 1; d += kGlaThreads, ++q)
-                for (int t = 0; t < n; ++t) decay *= sa[t * DP + d];
-    }
-    if (!kOut && blockIdx.x == 0) {
-        float* dec = chunk_decay + ((size_t)ch * p.heads + h) * p.dim;
-        if (tid < p.dim) dec[tid] = decay;
-        for (int d = tid + kGlaThreads; d < p.dim; d += kGlaThreads) {  // channels beyond one per thread: straight from memory
-            float a = 1.f;
-            for (int t = t0; t < t1; ++t) a *= alpha[(size_t)t * HD + h * p.dim + d];
-            dec[d] = a;
-        }
-    }
-    if (!kOut || ch == (int)gridDim.z - 1) {
-        float* Sout = kOut ? p.state + (size_t)h * mat : chunk_state + ((size_t)ch * p.heads + h) * mat;
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-            const int d = 4 * ((i >> 2) * G + g) + (i & 3);
-#pragma unroll
-            for (int c = 0; c < 4; ++c)
-                if (d < p.dim && v0 + c < p.vdim) Sout[(size_t)d * p.vdim + v0 + c] = s[i][c];
-        }
-    }
-}
-
-// chunk end states (from zero) -> state in front of every chunk, in place
-__global__ void __launch_bounds__(256) lb_gla_scan_kernel(const LbGla p, int chunks, float* chunk_state, const float* chunk_decay, int fresh) {
-    lb_pdl_launch_dependents();
-    lb_pdl_wait();
-    const size_t all = (size_t)p.heads * p.dim * p.vdim, i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= all) return;
-    const int hd = (int)(i / p.vdim);  // head * dim + channel
-    float s = fresh ? 0.f : p.state[i];
-    for (int c = 0; c < chunks; ++c) {
-        const float end = chunk_state[(size_t)c * all + i];
-        chunk_state[(size_t)c * all + i] = s;
-        s = fmaf(chunk_decay[(size_t)c * p.heads * p.dim + hd], s, end);
-    }
-}
-
 template <typename WT>
-__global__ void __launch_bounds__(256) lb_gated_heads_kernel(const float* __restrict__ o, const float* __restrict__ gate, int ldg, int heads, int vdim,
+__global__ void __launch_bounds__(256) lb_gated_heads_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, bool vec, int heads, int vdim,
                                                              const float* __restrict__ w, float eps, int slices, uint8_t* __restrict__ img) {
     extern __shared__ float s_r[];
     constexpr int C = LbElem<WT>::kChunk;
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, HV = heads * vdim;
-    const float* row = o + (size_t)t * HV;
+    const float* row = o + (size_t)t * ldo;
     for (int h = warp; h < heads; h += 8) {
         const float r = row_rstd(row + (size_t)h * vdim, vdim, eps, lane);
         if (lane == 0) s_r[h] = r;
     }
     __syncthreads();
     for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
-        float f[C];
+        float f[C], g[C];
+        lb_load_cols<C>(row, c * C, HV, vec, f);
+        lb_load_cols<C>(gate + (size_t)t * ldg, c * C, HV, vec, g);
 #pragma unroll
         for (int e = 0; e < C; ++e) {
-            const int k = c * C + e;
-            f[e] = 0.f;
-            if (k < HV) {
-                const int h = k / vdim;
-                f[e] = row[k] * s_r[h] * w[k - h * vdim] * lb_siluf(gate[(size_t)t * ldg + k]);
-            }
+            const int k = c * C + e, h = k / vdim;
+            f[e] = k < HV ? f[e] * s_r[h] * w[k - h * vdim] * lb_siluf(g[e]) : 0.f;
         }
         *reinterpret_cast<uint4*>(img + lb_img_chunk(t, c, slices)) = lb_pack_chunk<WT>(f);
     }
@@ -561,8 +373,9 @@ __global__ void __launch_bounds__(256) lb_route_gather_kernel(const LbRouteBlock
     const float r = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)width), eps))) * *gain;
     for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
         float h[C];
+        lb_load_cols<C>(row, c * C, width, ldx % 4 == 0, h);
 #pragma unroll
-        for (int e = 0; e < C; ++e) h[e] = c * C + e < width ? row[c * C + e] * r : 0.f;
+        for (int e = 0; e < C; ++e) h[e] *= r;
         for (int j = 0; j < p.top; ++j) {
             const float w = p.score[(size_t)t * p.top + j];
             float f[C];
@@ -608,7 +421,8 @@ int lb_embed_norm(loom_b200_ctx* ctx, int dtype, const void* table, int vocab, i
 
 int lb_norm_block(loom_b200_ctx* ctx, int dtype, const LbNormBlock& p) {
     LB_REQUIRE(ctx, p.taps >= 1 && p.taps <= kMaxTaps, "norm_block: %d taps (1..%d)", p.taps, kMaxTaps);
-    LB_TYPED(dtype, lb_norm_block_kernel<float>, lb_norm_block_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.T, kNormTokens)), dim3(256), 0, p);
+    LB_TYPED(dtype, lb_norm_block_kernel<float>, lb_norm_block_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.T, kNormTokens)), dim3(256), 0, p,
+             lb_vec_rows(p.x, p.ldx) && (!p.conv_w || (lb_vec_rows(p.conv_w, p.ring_ld) && lb_vec_rows(p.ring, p.ring_ld))));
     return 0;
 }
 
@@ -623,42 +437,10 @@ int lb_rows_image(loom_b200_ctx* ctx, int dtype, const float* x, int ldx, int T,
     return 0;
 }
 
-int lb_gla_step(loom_b200_ctx* ctx, const LbGla& p, const int* pos, int lane0, int M) {
-    const size_t smem = (size_t)(3 * p.dim + p.rank) * sizeof(float);
-    LB_REQUIRE(ctx, smem <= 48 * 1024, "gla: %d key channels, decay rank %d", p.dim, p.rank);
-    LB_LAUNCH(ctx, lb_gla_step_kernel, dim3(lb_ceil_div(p.vdim, 32), p.heads, M), dim3(256), smem, p, pos, lane0);
-    return 0;
-}
-
-int lb_gla_block(loom_b200_ctx* ctx, const LbGla& p, int T, int pos0, float* alpha, float* chunk_state, float* chunk_decay) {
-    int G = 1;
-    while (16 * G < p.dim) G *= 2;
-    LB_REQUIRE(ctx, G <= 32, "gla: %d key channels (at most 512)", p.dim);
-    const int cols = 4 * (kGlaThreads / G), vt = lb_ceil_div(p.vdim, cols);
-    // chunks: long ones unless they leave the device half empty
-    const int C = (long long)vt * p.heads * lb_ceil_div(T, kGlaChunk) >= 2 * ctx->sm_count ? kGlaChunk : kGlaChunk / 2;
-    const int chunks = lb_ceil_div(T, C), fresh = pos0 == 0 ? 1 : 0;
-    LB_LAUNCH(ctx, lb_gla_decay_kernel, dim3(T), dim3(256), (size_t)p.rank * sizeof(float), p, alpha);
-    const size_t smem = (size_t)kGlaStage * (3 * 16 * G + cols) * sizeof(float);
-    LB_REQUIRE(ctx, smem <= 200 * 1024, "gla: %d key channels", p.dim);
-    if (smem > 48 * 1024) {
-        LB_BIG_SMEM(ctx, lb_gla_chunk_kernel<true>, 200 * 1024);
-        LB_BIG_SMEM(ctx, lb_gla_chunk_kernel<false>, 200 * 1024);
-    }
-    const dim3 grid(vt, p.heads, chunks);
-    if (chunks > 1) {
-        LB_LAUNCH(ctx, lb_gla_chunk_kernel<false>, grid, dim3(kGlaThreads), smem, p, T, C, G, alpha, chunk_state, chunk_decay, fresh);
-        const size_t all = (size_t)p.heads * p.dim * p.vdim;
-        LB_LAUNCH(ctx, lb_gla_scan_kernel, dim3((unsigned)((all + 255) / 256)), dim3(256), 0, p, chunks, chunk_state, chunk_decay, fresh);
-    }
-    LB_LAUNCH(ctx, lb_gla_chunk_kernel<true>, grid, dim3(kGlaThreads), smem, p, T, C, G, alpha, chunk_state, chunk_decay, fresh);
-    return 0;
-}
-
-int lb_gated_heads_image(loom_b200_ctx* ctx, int dtype, const float* o, const float* gate, int ldg, int T, int heads, int vdim, const float* head_w,
+int lb_gated_heads_image(loom_b200_ctx* ctx, int dtype, const float* o, int ldo, const float* gate, int ldg, int T, int heads, int vdim, const float* head_w,
                          float eps, int slices, uint8_t* img) {
-    LB_TYPED(dtype, lb_gated_heads_kernel<float>, lb_gated_heads_kernel<__nv_bfloat16>, dim3(T), dim3(256), (size_t)heads * sizeof(float), o, gate, ldg,
-             heads, vdim, head_w, eps, slices, img);
+    LB_TYPED(dtype, lb_gated_heads_kernel<float>, lb_gated_heads_kernel<__nv_bfloat16>, dim3(T), dim3(256), (size_t)heads * sizeof(float), o, ldo, gate, ldg,
+             lb_vec_rows(o, ldo) && lb_vec_rows(gate, ldg), heads, vdim, head_w, eps, slices, img);
     return 0;
 }
 

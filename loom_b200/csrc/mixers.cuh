@@ -16,7 +16,7 @@ struct LbNormBlock {
     int T = 0, width = 0, slices = 0;
     const float* gain = nullptr;
     float eps = 0.f;
-    const float* conv_w = nullptr;  // [width][taps], or null: no convolution
+    const float* conv_w = nullptr;  // [taps][ring_ld], or null: no convolution
     float* ring = nullptr;          // of this sequence: [taps][ring_ld]
     int taps = 1, ring_ld = 0, pos0 = 0;
     uint8_t* img = nullptr;
@@ -33,17 +33,24 @@ struct LbGla {
     const float* a2b = nullptr;   // [heads*dim]
     float inv_tau = 1.f, qscale = 1.f;
     float* state = nullptr;       // [lane][heads][dim][vdim]
-    float* o = nullptr;           // [tokens, heads*vdim]
+    float* o = nullptr;           // [tokens, ldo]
+    int ldo = 0;
 };
 // one token of each of M sequences
 int lb_gla_step(loom_b200_ctx* ctx, const LbGla& p, const int* pos, int lane0, int M);
-// T tokens of one sequence whose state is `state` (lane 0 of it); alpha [T, heads*dim], chunk_state and chunk_decay as sized below
-constexpr int kGlaChunk = 128;
-static inline size_t lb_gla_chunk_state_elems(int T, int heads, int dim, int vdim) { return (size_t)lb_ceil_div(T, kGlaChunk / 2) * heads * dim * vdim; }
-static inline size_t lb_gla_chunk_decay_elems(int T, int heads, int dim) { return (size_t)lb_ceil_div(T, kGlaChunk / 2) * heads * dim; }
-int lb_gla_block(loom_b200_ctx* ctx, const LbGla& p, int T, int pos0, float* alpha, float* chunk_state, float* chunk_decay);
+// scratch of a block of T tokens in chunks of C = lb_gla_chunk(dim, rank)
+struct LbGlaBlock {
+    int C = 0;
+    float *qd = nullptr, *kd = nullptr;  // [T, heads*dim] queries decayed from the chunk's start, keys decayed to its end
+    float* decay = nullptr;              // [chunks, heads*dim] decay over a chunk
+    float* weights = nullptr;            // [chunks, heads, C, C]
+    float* states = nullptr;             // [chunks, heads, dim, vdim]
+};
+int lb_gla_chunk(int dim, int rank);
+// T tokens of one sequence whose state is `state` (lane 0 of it)
+int lb_gla_block(loom_b200_ctx* ctx, const LbGla& p, const LbGlaBlock& b, int T, int pos0);
 // image of (per-head rms of o) * head_w * silu(gate)
-int lb_gated_heads_image(loom_b200_ctx* ctx, int dtype, const float* o, const float* gate, int ldg, int T, int heads, int vdim, const float* head_w,
+int lb_gated_heads_image(loom_b200_ctx* ctx, int dtype, const float* o, int ldo, const float* gate, int ldg, int T, int heads, int vdim, const float* head_w,
                          float eps, int slices, uint8_t* img);
 // image of plain rows
 int lb_rows_image(loom_b200_ctx* ctx, int dtype, const float* x, int ldx, int T, int cols, int slices, uint8_t* img);
@@ -68,6 +75,19 @@ int lb_latent_absorb_q(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tok
 int lb_latent_attention(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tokens, const float* ql, float* ol);
 // out[token, heads*vdim] = W_uv[head] ol
 int lb_latent_absorb_v(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tokens, const float* ol, float* out, int ldo);
+
+// bf16, one token per sequence or a few tokens of one: every latent is read once for up to sixteen heads, the positions split over
+// `splits` CTAs whose results meet in front of the value rows.  part: [tokens, heads, splits, rank + 2]
+bool lb_latent_step_supported(const LbLatent& p);
+int lb_latent_step_splits(loom_b200_ctx* ctx, const LbLatent& p, int tokens);
+int lb_latent_step(loom_b200_ctx* ctx, const LbLatent& p, int tokens, const float* ql, float* part, int splits, float* out, int ldo);
+// bf16, a block of tokens on the tensor cores: keys and values of every position are expanded from the latents.  q_img and k_img hold
+// lb_latent_heads_bytes of T and pos0 + T rows, vt_img is an image of [heads*vdim] x positions (vt_slices K slices); the pads of
+// all three are zero.  out: token image of heads*vdim columns
+bool lb_latent_block_supported(const LbLatent& p);
+size_t lb_latent_heads_bytes(const LbLatent& p, int rows);
+int lb_latent_block(loom_b200_ctx* ctx, const LbLatent& p, int T, uint8_t* q_img, uint8_t* k_img, uint8_t* vt_img, int vt_slices, uint8_t* out,
+                    int out_slices);
 
 // ---- routing of a token block ------------------------------------------------------------------------------------
 struct LbRouteBlock {

@@ -18,7 +18,7 @@ bool is_bf16(const LbStack* st) { return st->d.dtype == LOOM_B200_DTYPE_BF16; }
 
 int hv_of(const loom_b200_layer_spec& s) { return s.heads * s.vdim; }
 
-LbGla gla_of(const LbLayer& l, const float* proj, int ldp, float* o, int lane) {
+LbGla gla_of(const LbLayer& l, const float* proj, int ldp, float* o, int ldo, int lane) {
     LbGla g;
     const loom_b200_layer_spec& s = l.s;
     g.proj = proj;
@@ -33,6 +33,7 @@ LbGla gla_of(const LbLayer& l, const float* proj, int ldp, float* o, int lane) {
     g.qscale = (float)(1.0 / std::sqrt((double)s.dim));
     g.state = l.gla_state + (size_t)lane * s.heads * s.dim * s.vdim;
     g.o = o;
+    g.ldo = ldo;
     return g;
 }
 
@@ -53,6 +54,53 @@ LbLatent latent_of(const LbStack* st, const LbLayer& l, const float* proj, int l
     p.lane_bytes = src.latent_lane;
     p.max_seq = st->d.max_seq_len;
     return p;
+}
+
+constexpr int kLatentStepTokens = 32;  // tokens of a portion that go through the step's attention kernels
+
+// attention of a few tokens in latent space, values applied: out [tokens, ldo]
+int latent_few(loom_b200_ctx* ctx, LbStack* st, int dt, const LbLatent& a, int tokens, float* ql, float* ol, float* part, float* out, int ldo) {
+    if (int rc = lb_latent_absorb_q(ctx, dt, a, tokens, ql)) return rc;
+    if (dt == LOOM_B200_DTYPE_BF16 && lb_latent_step_supported(a))
+        return lb_latent_step(ctx, a, tokens, ql, part, lb_latent_step_splits(ctx, a, tokens), out, ldo);
+    if (int rc = lb_latent_attention(ctx, dt, a, tokens, ql, ol)) return rc;
+    return lb_latent_absorb_v(ctx, dt, a, tokens, ol, out, ldo);
+}
+
+// floats of the split results of up to `tokens` tokens of any latent layer
+size_t latent_part_elems(loom_b200_ctx* ctx, LbStack* st, int tokens) {
+    size_t n = 0;
+    for (auto& l : st->layers) {
+        if (l.s.mixer != LOOM_B200_MIXER_LATENT || !is_bf16(st)) continue;
+        const LbLatent a = latent_of(st, l, nullptr, 0);
+        for (int t = 1; t <= tokens; ++t) n = std::max(n, (size_t)t * l.s.heads * lb_latent_step_splits(ctx, a, t) * (l.s.rank + 2));
+    }
+    return n;
+}
+
+// keys and transposed values of `rows` positions, expanded from the latents for a block
+int ensure_kv(loom_b200_ctx* ctx, LbStack* st, int rows) {
+    if ((size_t)rows <= st->kv_rows) return 0;
+    if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "stack scratch would grow while recording a graph");
+    LB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    if (st->pf_k) cudaFree(st->pf_k);
+    if (st->pf_v) cudaFree(st->pf_v);
+    st->pf_k = st->pf_v = nullptr;
+    st->kv_rows = 0;
+    const int n = lb_round_up(std::min(std::max(2 * rows, 1024), std::max(rows, st->d.max_seq_len)), kImgRows);
+    size_t k = 0, v = 0;
+    for (auto& l : st->layers) {
+        if (l.s.mixer != LOOM_B200_MIXER_LATENT) continue;
+        const LbLatent a = latent_of(st, l, nullptr, 0);
+        k = std::max(k, lb_latent_heads_bytes(a, n));
+        v = std::max(v, lb_img_bytes(hv_of(l.s), n, LOOM_B200_DTYPE_BF16));
+    }
+    LB_CUDA(ctx, cudaMalloc(&st->pf_k, k));
+    LB_CUDA(ctx, cudaMalloc(&st->pf_v, v));
+    LB_CUDA(ctx, cudaMemsetAsync(st->pf_k, 0, k, ctx->stream));
+    LB_CUDA(ctx, cudaMemsetAsync(st->pf_v, 0, v, ctx->stream));
+    st->kv_rows = n;
+    return 0;
 }
 
 int ensure_step_scratch(loom_b200_ctx* ctx, LbStack* st) {
@@ -89,6 +137,7 @@ int ensure_step_scratch(loom_b200_ctx* ctx, LbStack* st) {
     if (int rc = A(&st->ql, (size_t)M * hr * 4)) return rc;
     if (int rc = A(&st->ol, (size_t)M * hr * 4)) return rc;
     if (int rc = A(&st->rlog, (size_t)M * st->ldr * 4)) return rc;
+    if (int rc = A(&st->attn_part, latent_part_elems(ctx, st, M) * 4)) return rc;
     if (int rc = A(&st->pairs, (size_t)M * top * eff * (is_bf16(st) ? 2 : 4))) return rc;
     if (int rc = A(&st->list, sizeof(LbRouteList))) return rc;
     st->scratch_ready = true;
@@ -96,13 +145,13 @@ int ensure_step_scratch(loom_b200_ctx* ctx, LbStack* st) {
 }
 
 void free_block(LbStack* st) {
-    void* ptrs[] = {st->pf_tok, st->pf_x, st->pf_proj, st->pf_o, st->pf_alpha, st->pf_cs, st->pf_cd, st->pf_ql, st->pf_ol, st->pf_y, st->pf_rlog,
+    void* ptrs[] = {st->pf_tok, st->pf_x, st->pf_proj, st->pf_o, st->pf_qd, st->pf_kd, st->pf_cw, st->pf_part, st->pf_cs, st->pf_cd, st->pf_ql, st->pf_ol, st->pf_y, st->pf_rlog,
                     st->pf_score, st->pf_logits, st->pf_h, st->pf_io, st->pf_act, st->pf_gx, st->pf_ga, st->pf_idx, st->pf_slot, st->pf_count,
                     st->pf_offset, st->pf_bg, st->pf_nb, st->pf_rows, st->pf_qi, st->pf_k, st->pf_v};
     for (void* p : ptrs)
         if (p) cudaFree(p);
     st->pf_tok = nullptr;
-    st->pf_x = st->pf_proj = st->pf_o = st->pf_alpha = st->pf_cs = st->pf_cd = st->pf_ql = st->pf_ol = st->pf_y = st->pf_rlog = st->pf_score = st->pf_logits = nullptr;
+    st->pf_x = st->pf_proj = st->pf_o = st->pf_qd = st->pf_kd = st->pf_cw = st->pf_part = st->pf_cs = st->pf_cd = st->pf_ql = st->pf_ol = st->pf_y = st->pf_rlog = st->pf_score = st->pf_logits = nullptr;
     st->pf_h = st->pf_io = st->pf_act = st->pf_gx = st->pf_ga = st->pf_qi = st->pf_k = st->pf_v = nullptr;
     st->pf_idx = st->pf_slot = st->pf_count = st->pf_offset = st->pf_bg = st->pf_nb = st->pf_rows = nullptr;
     st->cap = 0;
@@ -159,7 +208,7 @@ int lb_stack_set_layer(loom_b200_ctx* ctx, LbStack* st, int layer, const loom_b2
     int in_rows = 0;
     if (s.mixer == LOOM_B200_MIXER_GLA) {
         LB_REQUIRE(ctx, s.tau > 0, "set_layer: layer %d: tau %g", layer, s.tau);
-        LB_REQUIRE(ctx, s.dim <= 512 && s.rank <= 4096, "set_layer: layer %d: %d key channels (at most 512), decay rank %d (at most 4096)", layer, s.dim, s.rank);
+        LB_REQUIRE(ctx, lb_gla_chunk(s.dim, s.rank) > 0, "set_layer: layer %d: %d key channels with decay rank %d", layer, s.dim, s.rank);
         LB_REQUIRE(ctx, w.mixer_norm && w.decay_w && w.decay_b, "set_layer: layer %d has no head norm or decay weights", layer);
         in_rows = 2 * HD + 2 * HV + s.rank;
     } else {
@@ -212,7 +261,10 @@ int lb_stack_set_layer(loom_b200_ctx* ctx, LbStack* st, int layer, const loom_b2
     const float scal[2] = {w.norm1, w.norm2};
     if (int rc = put(&l.scal, scal, 2)) return rc;
     if (w.conv_w) {
-        if (int rc = put(&l.conv_w, w.conv_w, (size_t)d.width * d.conv_taps)) return rc;
+        std::vector<float> t((size_t)d.conv_taps * st->ldx, 0.f);  // transposed: consecutive channels are consecutive in memory
+        for (int c = 0; c < d.width; ++c)
+            for (int j = 0; j < d.conv_taps; ++j) t[(size_t)j * st->ldx + c] = w.conv_w[(size_t)c * d.conv_taps + j];
+        if (int rc = put(&l.conv_w, t.data(), t.size())) return rc;
         if (int rc = zero(&l.conv_ring, (size_t)lanes * d.conv_taps * st->ldx * 4)) return rc;
     }
     if (s.mixer == LOOM_B200_MIXER_GLA) {
@@ -273,10 +325,10 @@ int lb_stack_step(loom_b200_ctx* ctx, LbStack* st, const int* tok, const int* po
         out.ldo = st->ldx;
         out.mult = mult;
         if (s.mixer == LOOM_B200_MIXER_GLA) {
-            LbGla g = gla_of(l, st->proj, st->ldp, st->o, 0);
+            LbGla g = gla_of(l, st->proj, st->ldp, st->o, st->ldo, 0);
             if (int rc = lb_gla_step(ctx, g, pos, lane0, M)) return rc;
             out.x = st->o;
-            out.ldx = hv_of(s);
+            out.ldx = st->ldo;
             out.gate = st->proj + 2 * s.heads * s.dim + hv_of(s);
             out.gate_ld = st->ldp;
             out.head_w = l.mixer_norm;
@@ -289,9 +341,7 @@ int lb_stack_step(loom_b200_ctx* ctx, LbStack* st, const int* tok, const int* po
             a.lane0 = lane0;
             if (s.kv_from < 0)
                 if (int rc = lb_latent_store(ctx, dt, a, st->proj + s.heads * s.dim, st->ldp, l.mixer_norm, eps, M)) return rc;
-            if (int rc = lb_latent_absorb_q(ctx, dt, a, M, st->ql)) return rc;
-            if (int rc = lb_latent_attention(ctx, dt, a, M, st->ql, st->ol)) return rc;
-            if (int rc = lb_latent_absorb_v(ctx, dt, a, M, st->ol, st->o, st->ldo)) return rc;
+            if (int rc = latent_few(ctx, st, dt, a, M, st->ql, st->ol, st->attn_part, st->o, st->ldo)) return rc;
             out.x = st->o;
             out.ldx = st->ldo;
             if (int rc = lb_dense_gemv(ctx, dt, LB_DPRO_PLAIN, LB_DEPI_RESID, out)) return rc;
@@ -363,17 +413,21 @@ int lb_stack_ensure_block(loom_b200_ctx* ctx, LbStack* st, int tokens) {
     LB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
     free_block(st);
     const int dt = st->d.dtype, T = lb_round_up(tokens, kImgRows), W = st->d.width;
-    size_t o = 0, io = 0, alpha = 0, cs = 0, cd = 0, hr = 0, act = 0, gx = 0, ga = 0, y = 0, rl = 0, pairs = 0, ex = 0, nb = 0;
+    size_t o = 0, io = 0, qd = 0, cs = 0, cd = 0, cw = 0, hr = 0, qi = 0, act = 0, gx = 0, ga = 0, y = 0, rl = 0, pairs = 0, ex = 0, nb = 0;
     for (auto& l : st->layers) {
         const loom_b200_layer_spec& s = l.s;
         o = std::max(o, (size_t)T * lb_round_up(hv_of(s), 8));
         io = std::max(io, lb_img_bytes(T, hv_of(s), dt));
         if (s.mixer == LOOM_B200_MIXER_GLA) {
-            alpha = std::max(alpha, (size_t)T * s.heads * s.dim);
-            cs = std::max(cs, lb_gla_chunk_state_elems(T, s.heads, s.dim, s.vdim));
-            cd = std::max(cd, lb_gla_chunk_decay_elems(T, s.heads, s.dim));
+            const size_t C = lb_gla_chunk(s.dim, s.rank), n = lb_ceil_div(T, (int)C);
+            qd = std::max(qd, (size_t)T * s.heads * s.dim);
+            cs = std::max(cs, n * s.heads * s.dim * s.vdim);
+            cd = std::max(cd, n * s.heads * s.dim);
+            cw = std::max(cw, n * s.heads * C * C);
         } else {
-            hr = std::max(hr, (size_t)T * s.heads * s.rank);
+            hr = std::max(hr, (size_t)std::min(T, kLatentStepTokens) * s.heads * s.rank);
+            LbLatent a = latent_of(st, l, nullptr, 0);
+            qi = std::max(qi, lb_latent_heads_bytes(a, T));
         }
         if (s.ffn == LOOM_B200_FFN_DENSE) act = std::max(act, lb_img_bytes(T, s.ff, dt));
         if (s.ffn == LOOM_B200_FFN_MOE) {
@@ -402,7 +456,11 @@ int lb_stack_ensure_block(loom_b200_ctx* ctx, LbStack* st, int tokens) {
     LB_A(pf_proj, (size_t)T * st->ldp * 4);
     LB_A(pf_o, o * 4);
     LB_A(pf_io, io);
-    LB_A(pf_alpha, alpha * 4);
+    LB_A(pf_qd, qd * 4);
+    LB_A(pf_kd, qd * 4);
+    LB_A(pf_cw, cw * 4);
+    LB_A(pf_part, latent_part_elems(ctx, st, std::min(T, kLatentStepTokens)) * 4);
+    if (is_bf16(st)) LB_A(pf_qi, qi);
     LB_A(pf_cs, cs * 4);
     LB_A(pf_cd, cd * 4);
     LB_A(pf_ql, hr * 4);
@@ -463,11 +521,17 @@ int lb_stack_block(loom_b200_ctx* ctx, LbStack* st, int T, int pos0, int lane) {
         g.ldo = st->ldp;
         if (int rc = lb_dense_gemm(ctx, dt, LB_DEPI_F32, g)) return rc;
 
-        const int hv = hv_of(s), oslices = l.w.out->slices;
+        const int hv = hv_of(s), ldo = lb_round_up(hv, 8), oslices = l.w.out->slices;
         if (s.mixer == LOOM_B200_MIXER_GLA) {
-            LbGla a = gla_of(l, st->pf_proj, st->ldp, st->pf_o, lane);
-            if (int rc = lb_gla_block(ctx, a, T, pos0, st->pf_alpha, st->pf_cs, st->pf_cd)) return rc;
-            if (int rc = lb_gated_heads_image(ctx, dt, st->pf_o, st->pf_proj + 2 * s.heads * s.dim + hv, st->ldp, T, s.heads, s.vdim, l.mixer_norm, eps,
+            LbGla a = gla_of(l, st->pf_proj, st->ldp, st->pf_o, ldo, lane);
+            LbGlaBlock b;
+            b.qd = st->pf_qd;
+            b.kd = st->pf_kd;
+            b.decay = st->pf_cd;
+            b.weights = st->pf_cw;
+            b.states = st->pf_cs;
+            if (int rc = lb_gla_block(ctx, a, b, T, pos0)) return rc;
+            if (int rc = lb_gated_heads_image(ctx, dt, st->pf_o, ldo, st->pf_proj + 2 * s.heads * s.dim + hv, st->ldp, T, s.heads, s.vdim, l.mixer_norm, eps,
                                               oslices, st->pf_io))
                 return rc;
         } else {
@@ -476,11 +540,20 @@ int lb_stack_block(loom_b200_ctx* ctx, LbStack* st, int T, int pos0, int lane) {
             a.lane0 = lane;
             if (s.kv_from < 0)
                 if (int rc = lb_latent_store(ctx, dt, a, st->pf_proj + s.heads * s.dim, st->ldp, l.mixer_norm, eps, T)) return rc;
-            const int ldo = lb_round_up(hv, 8);
-            if (int rc = lb_latent_absorb_q(ctx, dt, a, T, st->pf_ql)) return rc;
-            if (int rc = lb_latent_attention(ctx, dt, a, T, st->pf_ql, st->pf_ol)) return rc;
-            if (int rc = lb_latent_absorb_v(ctx, dt, a, T, st->pf_ol, st->pf_o, ldo)) return rc;
-            if (int rc = lb_rows_image(ctx, dt, st->pf_o, ldo, T, hv, oslices, st->pf_io)) return rc;
+            if (dt == LOOM_B200_DTYPE_BF16 && T > kLatentStepTokens && lb_latent_block_supported(a)) {
+                if (int rc = ensure_kv(ctx, st, pos0 + T)) return rc;
+                if (int rc = lb_latent_block(ctx, a, T, st->pf_qi, st->pf_k, st->pf_v, lb_ceil_div((int)st->kv_rows, 64), st->pf_io, oslices)) return rc;
+            } else {
+                // a few tokens at a time through the step's kernels, so that the scratch stays small
+                for (int t0 = 0; t0 < T; t0 += kLatentStepTokens) {
+                    LbLatent c = a;
+                    const int n = std::min(kLatentStepTokens, T - t0);
+                    c.q = a.q + (size_t)t0 * a.ldq;
+                    c.pos0 = pos0 + t0;
+                    if (int rc = latent_few(ctx, st, dt, c, n, st->pf_ql, st->pf_ol, st->pf_part, st->pf_o + (size_t)t0 * ldo, ldo)) return rc;
+                }
+                if (int rc = lb_rows_image(ctx, dt, st->pf_o, ldo, T, hv, oslices, st->pf_io)) return rc;
+            }
         }
         g = LbDenseGemm();
         g.x = st->pf_io;

@@ -39,7 +39,7 @@ struct LbStack {
     // scratch of a token block
     int cap = 0;
     int* pf_tok = nullptr;
-    float *pf_x = nullptr, *pf_proj = nullptr, *pf_o = nullptr, *pf_alpha = nullptr, *pf_cs = nullptr, *pf_cd = nullptr, *pf_ql = nullptr,
+    float *pf_x = nullptr, *pf_proj = nullptr, *pf_o = nullptr, *pf_qd = nullptr, *pf_kd = nullptr, *pf_cw = nullptr, *pf_part = nullptr, *pf_cs = nullptr, *pf_cd = nullptr, *pf_ql = nullptr,
           *pf_ol = nullptr, *pf_y = nullptr, *pf_rlog = nullptr, *pf_score = nullptr, *pf_logits = nullptr;
     uint8_t *pf_h = nullptr, *pf_io = nullptr, *pf_act = nullptr, *pf_gx = nullptr, *pf_ga = nullptr;
     uint8_t *pf_qi = nullptr, *pf_k = nullptr, *pf_v = nullptr;

@@ -105,9 +105,9 @@ def build_decoder(ctx, config: dict, weights, options: LoadOptions) -> "cabi.Dec
         dec.set_layer(i, s, w)
 
     table, code = weights.raw("embed", (d.vocab, W))
-    if dt == cabi.DTYPE_F32 or code == cabi.DTYPE_F32:
-        table = weights.f32("embed")
-        if dt == cabi.DTYPE_BF16:
-            table = cabi.to_bf16(table)
-    dec.set_stack_embeddings(ctx.to_device(np.ascontiguousarray(table)), weights.scalar("embed.norm"), matrix([("head", d.vocab)], W), weights.scalar("final.norm"))
+    if code != dt:
+        table = weights.f32("embed") if dt == cabi.DTYPE_F32 else cabi.to_bf16(table)
+    if not hasattr(table, "data_ptr"):  # (already on the device otherwise)
+        table = ctx.to_device(np.ascontiguousarray(table))
+    dec.set_stack_embeddings(table, weights.scalar("embed.norm"), matrix([("head", d.vocab)], W), weights.scalar("final.norm"))
     return dec
