@@ -418,6 +418,7 @@ void loom_b200_ctx_destroy(loom_b200_ctx* ctx) {
     if (ctx->head_scratch) cudaFree(ctx->head_scratch);
     if (ctx->gemm_scratch) cudaFree(ctx->gemm_scratch);
     if (ctx->quant_scratch) cudaFree(ctx->quant_scratch);
+    if (ctx->stage_scratch) cudaFree(ctx->stage_scratch);
     if (ctx->owns_stream) cudaStreamDestroy(ctx->stream);
     delete ctx;
 }

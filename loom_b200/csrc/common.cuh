@@ -63,6 +63,8 @@ struct loom_b200_ctx {
     int* status_host = nullptr;    // pinned mirror, refreshed by lb_sync_checked
     void* quant_scratch = nullptr;   // int8 row and absmax of the stand-alone GEMV prologue (wide inputs)
     size_t quant_scratch_bytes = 0;
+    void* stage_scratch = nullptr;   // input rows of the float GEMV for several sequences
+    size_t stage_scratch_bytes = 0;
     void* gemm_scratch = nullptr;    // int8 activations, amax and sums of the tensor-core GEMM path
     size_t gemm_scratch_bytes = 0;
     void* argmax_scratch = nullptr;  // per-CTA partial maxima of the greedy argmax

@@ -157,7 +157,7 @@ __device__ __forceinline__ void load_batch(GemvBatch<NB>& w, const uint8_t* stri
 
 // KW warps share a strip of 16 rows by K slices, 8/KW strips run side by side in a CTA.
 template <typename WT, int PRO, int EPI>
-__global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const LbDenseGemv p, int Mp, int KW, bool vec) {
+__global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const LbDenseGemv p, int Mp_launch, int KW, bool vec) {
     extern __shared__ __align__(16) uint8_t smem[];
     constexpr int C = LbElem<WT>::kChunk;
     constexpr bool kDual = EPI == LB_DEPI_GLU;
@@ -165,8 +165,11 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
     __shared__ float red[kGemvWarps][128];
     __shared__ float red2[kDual ? kGemvWarps : 1][128];
     __shared__ float s_stat[kGemvWarps];
-    __shared__ int s_pair[kMaxLanesPerPass];
+    __shared__ int s_pair[kMaxLanesPerPass], s_tok[kMaxLanesPerPass], s_n;
     __shared__ float s_w[kMaxLanesPerPass];
+    constexpr bool kStage = EPI == LB_DEPI_STAGE;
+    // columns of this CTA: every token; the token of a staging CTA; the tokens that chose this CTA's expert
+    int M = kStage ? 1 : p.M, Mp = kStage ? 1 : Mp_launch;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int SP = kGemvWarps / KW, kw = warp % KW, sp = warp / KW;
     const int strips = lb_ceil_div(p.rows, 16), chunks = p.slices * 8;
@@ -177,7 +180,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
     GemvBatch<NB> cur, cur2;
     int strip = (int)blockIdx.x * SP + sp;
     auto strip_ptr = [&](const uint8_t* base, int st) { return base + (size_t)(st >> 3) * p.slices * kImgBlock + (size_t)(st & 7) * 2048; };
-    constexpr bool kEarly = PRO != LB_DPRO_MOE && PRO != LB_DPRO_PAIRS;
+    constexpr bool kEarly = PRO != LB_DPRO_MOE && PRO != LB_DPRO_PAIRS && !kStage;
     if (kEarly && strip < strips) load_batch(cur, strip_ptr(w1, strip), kw, KW, p.slices, g, t);
     lb_pdl_launch_dependents();
     lb_pdl_wait();
@@ -243,25 +246,36 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
         const int e = s_idx[mine];
         w1 += (size_t)e * p.group_bytes;
         w2 += (size_t)e * p.group_bytes;
-        if (tid < p.M) {
-            int pr = -1;
-            for (int j = 0; j < p.top; ++j)
-                if (s_idx[tid * p.top + j] == e) pr = tid * p.top + j;
-            s_pair[tid] = pr;
-            s_w[tid] = pr >= 0 ? lb_sigmoidf(p.logits[(size_t)tid * p.ldl + e]) : 0.f;
+        if (tid == 0) {
+            int n = 0;
+            for (int q = 0; q < pairs; ++q)
+                if (s_idx[q] == e) {
+                    s_pair[n] = q;
+                    s_tok[n] = q / p.top;
+                    s_w[n] = lb_sigmoidf(p.logits[(size_t)(q / p.top) * p.ldl + e]);
+                    ++n;
+                }
+            s_n = n;
         }
         if (strip < strips) {
             load_batch(cur, strip_ptr(w1, strip), kw, KW, p.slices, g, t);
             load_batch(cur2, strip_ptr(w2, strip), kw, KW, p.slices, g, t);
         }
         __syncthreads();
+        M = s_n;
+        Mp = 1;
+        while (Mp < M) Mp *= 2;
     }
 
-    if (PRO != LB_DPRO_PAIRS) {
+    if (PRO == LB_DPRO_STAGED) {
+        for (int i = tid; i < chunks * Mp; i += kGemvThreads) xs[i] = p.staged[i];
+        __syncthreads();
+    } else if (PRO != LB_DPRO_PAIRS) {
         // ---- input rows: 8/Mp warps per token ----
         const int WPT = kGemvWarps / Mp, m = warp / WPT, wt = warp % WPT, lt = wt * 32 + lane, nt = WPT * 32;
-        const bool live = m < p.M;
-        const int src = live ? (p.row_idx ? p.row_idx[m] : m) : 0;
+        const bool live = m < M;
+        const int tok = !live ? 0 : kStage ? (int)blockIdx.x : PRO == LB_DPRO_MOE ? s_tok[m] : m;
+        const int src = p.row_idx ? p.row_idx[tok] : tok;
         const float* xr = p.x + (size_t)src * p.ldx;
         float rstd = 0.f, gain = 1.f;
         float* s_head = nullptr;
@@ -293,9 +307,9 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
                 }
             __syncthreads();
         }
-        const int seq = p.lane0 + m;
+        const int seq = p.lane0 + tok;
         int pos = 0;
-        if (PRO == LB_DPRO_CONV && live) pos = p.pos[m];
+        if (PRO == LB_DPRO_CONV && live) pos = p.pos[tok];
         for (int c = lt; c < chunks; c += nt) {
             float f[C];
             const int k0 = c * C;
@@ -311,7 +325,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
                 }
                 if (PRO == LB_DPRO_GATED) {
                     float gt[C];
-                    lb_load_cols<C>(p.gate + (size_t)m * p.gate_ld, k0, p.K, vec, gt);
+                    lb_load_cols<C>(p.gate + (size_t)tok * p.gate_ld, k0, p.K, vec, gt);
 #pragma unroll
                     for (int i = 0; i < C; ++i) {
                         const int k = k0 + i, h = k / p.head_dim;
@@ -336,7 +350,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
 #pragma unroll
                     for (int i = 0; i < C; ++i) {
                         a[i] = fmaf(w[i], f[i], a[i]);
-                        if (blockIdx.x == 0 && k0 + i < p.K) slot[i] = f[i];
+                        if ((kStage || blockIdx.x == 0) && k0 + i < p.K) slot[i] = f[i];
                         f[i] += a[i];
                     }
                 }
@@ -344,10 +358,16 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
 #pragma unroll
                 for (int i = 0; i < C; ++i) f[i] = 0.f;
             }
+            if (kStage) {
+                p.staged[(size_t)c * Mp_launch + tok] = lb_pack_chunk<WT>(f);
+                continue;
+            }
             xs[(size_t)c * Mp + m] = lb_pack_chunk<WT>(f);
         }
         __syncthreads();
     }
+
+    if (kStage) return;
 
     const int nact = PRO == LB_DPRO_PAIRS ? p.list->n : 1;
 
@@ -375,11 +395,11 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
                         const int sl = s + u * KW;
                         if (sl < p.slices) {
                             const uint4* x0 = xs + (size_t)(sl * 8 + t) * Mp;
-                            acc.step(now.a[u][0], now.b[u][0], x0, Mp, p.M, g);
-                            acc.step(now.a[u][1], now.b[u][1], x0 + 4 * Mp, Mp, p.M, g);
+                            acc.step(now.a[u][0], now.b[u][0], x0, Mp, M, g);
+                            acc.step(now.a[u][1], now.b[u][1], x0 + 4 * Mp, Mp, M, g);
                             if (kDual) {
-                                acc2.step(now2.a[u][0], now2.b[u][0], x0, Mp, p.M, g);
-                                acc2.step(now2.a[u][1], now2.b[u][1], x0 + 4 * Mp, Mp, p.M, g);
+                                acc2.step(now2.a[u][0], now2.b[u][0], x0, Mp, M, g);
+                                acc2.step(now2.a[u][1], now2.b[u][1], x0 + 4 * Mp, Mp, M, g);
                             }
                         }
                     }
@@ -418,7 +438,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
         for (int o = tid; o < SP * 128; o += kGemvThreads) {
             const int s = o >> 7, e = o & 127, r = e >> 3, m = e & 7;
             const int row = (strip - sp + s) * 16 + r;
-            if (m >= p.M || row >= p.rows) continue;
+            if (m >= M || row >= p.rows) continue;
             float v = 0.f, u = 0.f;
             for (int k = 0; k < KW; ++k) {
                 v += red[s * KW + k][e];
@@ -431,18 +451,17 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
             }
             if (EPI == LB_DEPI_GELU) p.out[(size_t)m * p.ldo + row] = lb_gelu_erff(v);
             if (EPI == LB_DEPI_GLU) {
-                const int pr = s_pair[m];
-                if (pr >= 0) {
-                    const float y = lb_clamped_glu(v, u, p.limit);
-                    reinterpret_cast<WT*>(p.out_pairs)[(size_t)pr * p.ldo + row] = (WT)y;
-                }
+                reinterpret_cast<WT*>(p.out_pairs)[(size_t)s_pair[m] * p.ldo + row] = (WT)lb_clamped_glu(v, u, p.limit);
             }
         }
     }
 }
 
+constexpr int kStageTokens = 3;  // from this many tokens on the input rows are made once, by a launch of their own
+
 template <typename WT, int PRO, int EPI>
-int gemv_launch(loom_b200_ctx* ctx, const LbDenseGemv& p) {
+int gemv_launch(loom_b200_ctx* ctx, const LbDenseGemv& pin) {
+    LbDenseGemv p = pin;
     LB_REQUIRE(ctx, p.M >= 1 && p.M <= kMaxLanesPerPass, "dense_gemv: %d tokens", p.M);
     int Mp = 1;
     while (Mp < p.M) Mp *= 2;
@@ -452,33 +471,59 @@ int gemv_launch(loom_b200_ctx* ctx, const LbDenseGemv& p) {
     // many strips per CTA: fewer warps per strip, so that a warp streams longer runs between two meetings of the sums
     while (KW > 1 && (long long)strips >= 6ll * (2 * kGemvWarps / KW) * cap) KW /= 2;
     const int SP = kGemvWarps / KW;
-    bool vec = lb_vec_rows(p.x, p.ldx);
+    bool vec = PRO == LB_DPRO_STAGED || PRO == LB_DPRO_PAIRS || lb_vec_rows(p.x, p.ldx);
     if (PRO == LB_DPRO_GATED) vec = vec && lb_vec_rows(p.gate, p.gate_ld);
     if (PRO == LB_DPRO_CONV) vec = vec && lb_vec_rows(p.conv_w, p.ring_ld) && lb_vec_rows(p.conv_ring, p.ring_ld);
-    size_t smem = PRO == LB_DPRO_PAIRS ? 0 : (size_t)p.slices * 8 * Mp * 16;
+    const size_t rows_smem = (size_t)p.slices * 8 * (EPI == LB_DEPI_STAGE ? 1 : Mp) * 16;
+    size_t smem = PRO == LB_DPRO_PAIRS || EPI == LB_DEPI_STAGE ? 0 : rows_smem;
     if (PRO == LB_DPRO_MOE) smem += (size_t)p.M * p.experts * 4 + (size_t)p.M * p.top * 4;
-    if (PRO == LB_DPRO_GATED) smem += (size_t)Mp * (p.K / p.head_dim) * 4;
+    if (PRO == LB_DPRO_GATED) smem = rows_smem + (size_t)Mp * (p.K / p.head_dim) * 4;
     if (smem > kGemvSmemX + 16 * 1024) return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "dense_gemv: %d tokens of %d columns need %zu B of shared memory", p.M, p.K, smem);
     if (smem > 48 * 1024) LB_BIG_SMEM(ctx, (lb_dense_gemv_kernel<WT, PRO, EPI>), kGemvSmemX + 16 * 1024);
-    int gx = lb_ceil_div(strips, SP);
-    const int gy = PRO == LB_DPRO_MOE ? p.M * p.top : 1;
-    if (gx > cap) gx = lb_ceil_div(gx, lb_ceil_div(gx, cap));  // equal numbers of strips per CTA
+    int gx = lb_ceil_div(strips, SP), gy = 1, share = cap;
+    if (EPI == LB_DEPI_STAGE) {
+        gx = share = p.M;
+    } else if (PRO == LB_DPRO_MOE) {
+        gy = p.M * p.top;
+        share = cap / (gy < p.experts ? gy : p.experts);
+        if (share < 1) share = 1;
+    }
+    if (gx > share) gx = lb_ceil_div(gx, lb_ceil_div(gx, share));  // equal numbers of strips per CTA
     LB_LAUNCH(ctx, (lb_dense_gemv_kernel<WT, PRO, EPI>), dim3(gx, gy), dim3(kGemvThreads), smem, p, Mp, KW, vec);
     return 0;
 }
 
+// a product whose input rows take some work: inside every CTA for one or two tokens, as a launch of their own for more
+template <typename WT, int PRO, int EPI>
+int gemv_rows(loom_b200_ctx* ctx, const LbDenseGemv& pin) {
+    if (pin.M < kStageTokens) return gemv_launch<WT, PRO, EPI>(ctx, pin);
+    LbDenseGemv p = pin;
+    const size_t bytes = (size_t)p.slices * 8 * kMaxLanesPerPass * 16;
+    if (bytes > ctx->stage_scratch_bytes) {
+        if (ctx->capturing) return lb_fail(ctx, LOOM_B200_ERR_INVALID, "the staging buffer of the GEMV would grow while recording a graph");
+        LB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+        if (ctx->stage_scratch) cudaFree(ctx->stage_scratch);
+        ctx->stage_scratch = nullptr;
+        ctx->stage_scratch_bytes = 0;
+        LB_CUDA(ctx, cudaMalloc(&ctx->stage_scratch, bytes));
+        ctx->stage_scratch_bytes = bytes;
+    }
+    p.staged = static_cast<uint4*>(ctx->stage_scratch);
+    if (int rc = gemv_launch<WT, PRO, LB_DEPI_STAGE>(ctx, p)) return rc;
+    return gemv_launch<WT, LB_DPRO_STAGED, EPI>(ctx, p);
+}
+
 template <typename WT>
 int gemv_dispatch(loom_b200_ctx* ctx, int pro, int epi, const LbDenseGemv& p) {
-#define LB_CASE(P, E) \
-    if (pro == P && epi == E) return gemv_launch<WT, P, E>(ctx, p)
-    LB_CASE(LB_DPRO_CONV, LB_DEPI_F32);
-    LB_CASE(LB_DPRO_NORM, LB_DEPI_F32);
-    LB_CASE(LB_DPRO_NORM, LB_DEPI_GELU);
-    LB_CASE(LB_DPRO_PLAIN, LB_DEPI_F32);
-    LB_CASE(LB_DPRO_PLAIN, LB_DEPI_RESID);
-    LB_CASE(LB_DPRO_GATED, LB_DEPI_RESID);
-    LB_CASE(LB_DPRO_MOE, LB_DEPI_GLU);
-    LB_CASE(LB_DPRO_PAIRS, LB_DEPI_RESID);
+#define LB_CASE(P, E, RUN) \
+    if (pro == P && epi == E) return RUN<WT, P, E>(ctx, p)
+    LB_CASE(LB_DPRO_CONV, LB_DEPI_F32, gemv_rows);
+    LB_CASE(LB_DPRO_NORM, LB_DEPI_F32, gemv_rows);
+    LB_CASE(LB_DPRO_NORM, LB_DEPI_GELU, gemv_rows);
+    LB_CASE(LB_DPRO_PLAIN, LB_DEPI_RESID, gemv_launch);
+    LB_CASE(LB_DPRO_GATED, LB_DEPI_RESID, gemv_rows);
+    LB_CASE(LB_DPRO_MOE, LB_DEPI_GLU, gemv_launch);
+    LB_CASE(LB_DPRO_PAIRS, LB_DEPI_RESID, gemv_launch);
 #undef LB_CASE
     return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "dense_gemv: prologue %d with epilogue %d is not built", pro, epi);
 }

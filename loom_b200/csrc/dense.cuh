@@ -148,6 +148,7 @@ enum LbDensePro : int {
     LB_DPRO_GATED = 3,  // per-head RMS norm with a weight, times silu of a gate row (output of gated linear attention)
     LB_DPRO_MOE = 4,    // routed experts: top-k of the router's logits, RMS norm, times the token's weight for the expert
     LB_DPRO_PAIRS = 5,  // routed experts, second product: one row per (token, choice), summed over the choices
+    LB_DPRO_STAGED = 6, // input rows already made by a launch of their own (several tokens; chosen by the launcher)
 };
 enum LbDenseEpi : int {
     LB_DEPI_F32 = 0,    // out [token, ldo] = acc
@@ -155,6 +156,7 @@ enum LbDenseEpi : int {
     LB_DEPI_GELU = 2,   // exact gelu (GEMV: float rows, GEMM: image)
     LB_DEPI_GLU = 3,    // clamped gated unit of two products (GEMV: rows of WT per pair, GEMM: image)
     LB_DEPI_IMG = 4,    // GEMM only: image
+    LB_DEPI_STAGE = 6,  // GEMV: only the prologue, a CTA per token, into `staged`
     LB_DEPI_HEADS = 5,  // GEMM only: per-head blocks [token block of 128][head][token/8][chunk][token%8][16 B]
 };
 
@@ -195,6 +197,7 @@ struct LbDenseGemv {
     int ldl = 0, experts = 0, top = 0;
     LbRouteList* list = nullptr;
     const uint8_t* pairs = nullptr;  // [M * top, ldp] rows of WT
+    uint4* staged = nullptr;         // [chunk][M rounded up to a power of two] input chunks, set by the launcher
     int ldp = 0;
     // output
     float* out = nullptr;

@@ -3,6 +3,8 @@
 #include "mixers.cuh"
 #include "umma.cuh"
 
+#include <cmath>
+
 namespace {
 
 __device__ __forceinline__ void mma_bf16(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
@@ -12,6 +14,12 @@ __device__ __forceinline__ void mma_bf16(float* d, uint32_t a0, uint32_t a1, uin
 }
 __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t* r, const void* p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(lb_smem_u32(p)));
+}
+// 2^x by the hardware's approximation (two units in the last place), results below 2^-126 as zero
+__device__ __forceinline__ float fast_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
 // value = hi + lo, both bf16: the pair carries sixteen bits of the float
 __device__ __forceinline__ void split_bf16(const float* f, uint4& hi, uint4& lo) {
@@ -260,9 +268,11 @@ __global__ void __launch_bounds__(256) lb_latent_value_kernel(const LbLatent p, 
     __syncthreads();
     for (int k = threadIdx.x; k < cols; k += blockDim.x) {
         float a = 0.f;
-        if (k < p.rank)
-            for (int s = 0; s < splits; ++s)
-                if (sw[s] > 0.f) a = fmaf(sw[s], base[(size_t)s * row + k], a);  // (a split without positions holds no sums)
+        if (k < p.rank) {
+            // (a split without positions has weight zero over whatever finite sums an earlier step left there)
+#pragma unroll 8
+            for (int s = 0; s < splits; ++s) a = fmaf(sw[s], base[(size_t)s * row + k], a);
+        }
         sm2[k] = a;
     }
     __syncthreads();
@@ -296,7 +306,7 @@ struct AttnParams {
     const uint8_t* vt;  // image of [heads*vdim rows] x positions
     int heads, dchunks, vdim, vslices;  // dchunks: 16-byte chunks of a query row (even); vslices: K slices of vt
     int T, pos0;
-    float scale_log2;   // score factor times log2(e)
+    float scale_log2;   // magnitude of the score factor times log2(e) (its sign is in the queries)
     uint8_t* out;       // token image of heads*vdim columns
     int out_slices;
     int* status;
@@ -364,7 +374,7 @@ __global__ void __launch_bounds__(kAtThreads, 2) lb_latent_block_kernel(const At
     float o[VC];
 #pragma unroll
     for (int c = 0; c < VC; ++c) o[c] = 0.f;
-    float mx = -INFINITY, sum = 0.f;
+    float mx = -3e38f, sum = 0.f;  // (finite: the factor may be zero)
     uint8_t* prow = sp + (size_t)(row >> 3) * 1024 + (row & 7) * 16;
     for (int j = 0; j < ntiles; ++j) {
         if (!lb_mbar_wait_bounded(&bar_s, (uint32_t)(j & 1), kTcWaitLimit)) failed = true;
@@ -380,28 +390,22 @@ __global__ void __launch_bounds__(kAtThreads, 2) lb_latent_block_kernel(const At
             for (int c = 0; c < kAtKeys; c += 16) lb_tmem_ld16(tmem + lanes + c, s + c);
             lb_tmem_wait_ld();
             const int vis = qpos - j * kAtKeys;  // keys 0..vis of the tile are visible
-            float m = mx;
             if (vis < kAtKeys - 1) {
 #pragma unroll
-                for (int c = 0; c < kAtKeys; ++c) {
-                    s[c] = c <= vis ? s[c] * p.scale_log2 : -INFINITY;
-                    m = fmaxf(m, s[c]);
-                }
-            } else {
-#pragma unroll
-                for (int c = 0; c < kAtKeys; ++c) {
-                    s[c] *= p.scale_log2;
-                    m = fmaxf(m, s[c]);
-                }
+                for (int c = 0; c < kAtKeys; ++c) s[c] = c <= vis ? s[c] : -INFINITY;
             }
-            f = exp2f(mx - m);
+            float m4[4] = {mx, -INFINITY, -INFINITY, -INFINITY};  // (the factor is not negative, so it may follow the maximum)
+#pragma unroll
+            for (int c = 0; c < kAtKeys; ++c) m4[c & 3] = fmaxf(m4[c & 3], s[c]);
+            const float m = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])), off = m * p.scale_log2;
+            f = fast_exp2(mx * p.scale_log2 - off);
             mx = m;
             float add = 0.f;
 #pragma unroll
             for (int c = 0; c < kAtKeys; c += 8) {
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
-                    s[c + e] = exp2f(s[c + e] - m);
+                    s[c + e] = fast_exp2(fmaf(s[c + e], p.scale_log2, -off));
                     add += s[c + e];
                 }
                 *reinterpret_cast<uint4*>(prow + (c >> 3) * 128) = lb_pack_chunk<__nv_bfloat16>(s + c);
@@ -468,7 +472,7 @@ __global__ void __launch_bounds__(kAtThreads, 2) lb_latent_block_kernel(const At
 }
 
 // float query rows -> per-head bf16 blocks
-__global__ void __launch_bounds__(256) lb_heads_image_kernel(const float* __restrict__ x, int ldx, int heads, int dim, int dchunks, uint8_t* __restrict__ img) {
+__global__ void __launch_bounds__(256) lb_heads_image_kernel(const float* __restrict__ x, int ldx, int heads, int dim, int dchunks, float sign, uint8_t* __restrict__ img) {
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const int t = blockIdx.x;
@@ -476,7 +480,7 @@ __global__ void __launch_bounds__(256) lb_heads_image_kernel(const float* __rest
         const int h = i / dchunks, c = i - h * dchunks;
         float f[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[e] = c * 8 + e < dim ? x[(size_t)t * ldx + h * dim + c * 8 + e] : 0.f;
+        for (int e = 0; e < 8; ++e) f[e] = c * 8 + e < dim ? sign * x[(size_t)t * ldx + h * dim + c * 8 + e] : 0.f;
         *reinterpret_cast<uint4*>(img + ((size_t)(t >> 7) * heads + h) * dchunks * 2048 + (size_t)((t & 127) >> 3) * dchunks * 128 + (size_t)c * 128 + (t & 7) * 16) =
             lb_pack_chunk<__nv_bfloat16>(f);
     }
@@ -530,14 +534,14 @@ int lb_latent_step(loom_b200_ctx* ctx, const LbLatent& p, int tokens, const floa
 
 int lb_latent_dchunks(int dim) { return lb_round_up(lb_ceil_div(dim, 8), 2); }
 
-bool lb_latent_block_supported(const LbLatent& p) { return p.dim % 8 == 0 && p.dim <= 256 && p.vdim % 8 == 0 && p.vdim <= 128; }
+bool lb_latent_block_supported(const LbLatent& p) { return p.dim % 8 == 0 && p.dim <= 256 && p.vdim % 8 == 0 && p.vdim <= 128 && p.scale != 0.f; }
 
 size_t lb_latent_heads_bytes(const LbLatent& p, int rows) { return (size_t)lb_ceil_div(rows, 128) * p.heads * lb_latent_dchunks(p.dim) * 2048; }
 
 int lb_latent_block(loom_b200_ctx* ctx, const LbLatent& p, int T, uint8_t* q_img, uint8_t* k_img, uint8_t* vt_img, int vt_slices, uint8_t* out, int out_slices) {
     const int ctx_rows = p.pos0 + T, dch = lb_latent_dchunks(p.dim);
     const uint8_t* cache = p.cache + (size_t)p.lane0 * p.lane_bytes;
-    LB_LAUNCH(ctx, lb_heads_image_kernel, dim3(T), dim3(256), 0, p.q, p.ldq, p.heads, p.dim, dch, q_img);
+    LB_LAUNCH(ctx, lb_heads_image_kernel, dim3(T), dim3(256), 0, p.q, p.ldq, p.heads, p.dim, dch, p.scale < 0.f ? -1.f : 1.f, q_img);
     // keys of every position, per head
     LbDenseGemm g;
     g.x = cache;
@@ -570,7 +574,7 @@ int lb_latent_block(loom_b200_ctx* ctx, const LbLatent& p, int T, uint8_t* q_img
     a.vslices = vt_slices;
     a.T = T;
     a.pos0 = p.pos0;
-    a.scale_log2 = p.scale * 1.4426950408889634f;
+    a.scale_log2 = fabsf(p.scale) * 1.4426950408889634f;
     a.out = out;
     a.out_slices = out_slices;
     a.status = ctx->status_dev;

@@ -143,37 +143,54 @@ __global__ void __launch_bounds__(256) lb_gated_heads_kernel(const float* __rest
 
 // ---- latent attention ---------------------------------------------------------------------------------------------
 
+// what a layer with a latent projection of its own adds to the cache: rms of the projected row times a weight
+struct LatentRow {
+    const float* raw;  // [tokens, ldr], or null
+    int ldr;
+    const float* weight;
+    float eps;
+};
+
 template <typename WT>
-__global__ void __launch_bounds__(256) lb_latent_store_kernel(const LbLatent p, const float* __restrict__ raw, int ldr, const float* __restrict__ w, float eps) {
+__device__ void latent_store_row(const LbLatent& p, const LatentRow& l, int t) {
     constexpr int C = LbElem<WT>::kChunk;
     __shared__ float red[8];
-    lb_pdl_launch_dependents();
-    lb_pdl_wait();
-    const int t = blockIdx.x;
     const int pos = p.pos ? p.pos[t] : p.pos0 + t, lane = p.pos ? p.lane0 + t : p.lane0;
     if (pos >= p.max_seq) return;
-    const float* row = raw + (size_t)t * ldr;
+    const float* row = l.raw + (size_t)t * l.ldr;
     float ss = 0.f;
     for (int k = threadIdx.x; k < p.rank; k += blockDim.x) ss = fmaf(row[k], row[k], ss);
     ss = lb_block_sumf(ss, red);
-    const float r = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)p.rank), eps)));
+    const float r = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)p.rank), l.eps)));
     uint8_t* img = p.cache + (size_t)lane * p.lane_bytes;
     for (int c = threadIdx.x; c < p.slices * 8; c += blockDim.x) {
         float f[C];
 #pragma unroll
-        for (int e = 0; e < C; ++e) f[e] = c * C + e < p.rank ? row[c * C + e] * r * w[c * C + e] : 0.f;
+        for (int e = 0; e < C; ++e) f[e] = c * C + e < p.rank ? row[c * C + e] * r * l.weight[c * C + e] : 0.f;
         *reinterpret_cast<uint4*>(img + lb_img_chunk(pos, c, p.slices)) = lb_pack_chunk<WT>(f);
     }
 }
 
-// CTA = (32 chunks of the latent, head, token): thread = (row % 8, chunk), the rows of the head in groups of eight
 template <typename WT>
-__global__ void __launch_bounds__(256) lb_absorb_q_kernel(const LbLatent p, float* __restrict__ ql) {
+__global__ void __launch_bounds__(256) lb_latent_store_kernel(const LbLatent p, const LatentRow l) {
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    latent_store_row<WT>(p, l, blockIdx.x);
+}
+
+// CTA = (32 chunks of the latent, head, token): thread = (row % 8, chunk), the rows of the head in groups of eight.  One CTA more
+// per token puts the token's latent into the cache.
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_absorb_q_kernel(const LbLatent p, const LatentRow l, float* __restrict__ ql) {
     extern __shared__ float sm[];
     constexpr int C = LbElem<WT>::kChunk;
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const int h = blockIdx.y, t = blockIdx.z;
+    if (h == p.heads) {
+        if (blockIdx.x == 0) latent_store_row<WT>(p, l, t);
+        return;
+    }
     const int r8 = threadIdx.x & 7, chunk = blockIdx.x * 32 + (threadIdx.x >> 3);
     float* sq = sm;  // [dim]
     for (int d = threadIdx.x; d < p.dim; d += blockDim.x) sq[d] = p.q[(size_t)t * p.ldq + h * p.dim + d] * p.scale;
@@ -445,14 +462,16 @@ int lb_gated_heads_image(loom_b200_ctx* ctx, int dtype, const float* o, int ldo,
 }
 
 int lb_latent_store(loom_b200_ctx* ctx, int dtype, const LbLatent& p, const float* raw, int ldr, const float* weight, float eps, int tokens) {
-    LB_TYPED(dtype, lb_latent_store_kernel<float>, lb_latent_store_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, p, raw, ldr, weight, eps);
+    const LatentRow l = {raw, ldr, weight, eps};
+    LB_TYPED(dtype, lb_latent_store_kernel<float>, lb_latent_store_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, p, l);
     return 0;
 }
 
-int lb_latent_absorb_q(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tokens, float* ql) {
+int lb_latent_absorb_q(loom_b200_ctx* ctx, int dtype, const LbLatent& p, const float* raw, int ldr, const float* weight, float eps, int tokens, float* ql) {
     LB_REQUIRE(ctx, p.dim <= 8192, "latent attention: query dimension %d", p.dim);
-    LB_TYPED(dtype, lb_absorb_q_kernel<float>, lb_absorb_q_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.slices * 8, 32), p.heads, tokens), dim3(256),
-             (size_t)p.dim * sizeof(float), p, ql);
+    const LatentRow l = {raw, ldr, weight, eps};
+    LB_TYPED(dtype, lb_absorb_q_kernel<float>, lb_absorb_q_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.slices * 8, 32), p.heads + (raw ? 1 : 0), tokens), dim3(256),
+             (size_t)p.dim * sizeof(float), p, l, ql);
     return 0;
 }
 

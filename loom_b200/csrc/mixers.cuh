@@ -69,8 +69,8 @@ struct LbLatent {
 };
 // latent rows: rms of raw * weight into the cache
 int lb_latent_store(loom_b200_ctx* ctx, int dtype, const LbLatent& p, const float* raw, int ldr, const float* weight, float eps, int tokens);
-// queries in latent space: ql[token, head, rank] = scale * W_uk[head]^T q
-int lb_latent_absorb_q(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tokens, float* ql);
+// queries in latent space: ql[token, head, rank] = scale * W_uk[head]^T q; with raw, the tokens' latents are stored by the same launch
+int lb_latent_absorb_q(loom_b200_ctx* ctx, int dtype, const LbLatent& p, const float* raw, int ldr, const float* weight, float eps, int tokens, float* ql);
 // attention over the latents: ol[token, head, rank] = sum_j softmax_j(ql . c_j) c_j
 int lb_latent_attention(loom_b200_ctx* ctx, int dtype, const LbLatent& p, int tokens, const float* ql, float* ol);
 // out[token, heads*vdim] = W_uv[head] ol

@@ -3,8 +3,8 @@
 // Step, per layer (M <= 8 sequences, one token each; every launch chained by programmatic dependent launch):
 //   gated linear attention   {norm + short convolution + input projections} -> {decay, state update, read-out}
 //                            -> {per-head norm, gate, output projection, residual}
-//   latent attention         {norm + short convolution + query / latent projections} -> {latent norm, cache} -> {queries into
-//                            latent space} -> {attention over the latents} -> {values} -> {output projection, residual}
+//   latent attention         {norm + short convolution + query / latent projections} -> {queries into latent space, latent
+//                            norm, cache} -> {attention over the latents} -> {values} -> {output projection, residual}
 //   feed-forward             dense {norm, up, gelu} -> {down, residual}; routed {norm, router} -> {choice, norm, gate / up,
 //                            clamped unit} -> {down of every chosen expert, sum, residual}
 #include "stack.cuh"
@@ -58,9 +58,11 @@ LbLatent latent_of(const LbStack* st, const LbLayer& l, const float* proj, int l
 
 constexpr int kLatentStepTokens = 32;  // tokens of a portion that go through the step's attention kernels
 
-// attention of a few tokens in latent space, values applied: out [tokens, ldo]
-int latent_few(loom_b200_ctx* ctx, LbStack* st, int dt, const LbLatent& a, int tokens, float* ql, float* ol, float* part, float* out, int ldo) {
-    if (int rc = lb_latent_absorb_q(ctx, dt, a, tokens, ql)) return rc;
+// attention of a few tokens in latent space, values applied: out [tokens, ldo].  raw: the latent projections that go into the cache
+// first (row stride of the queries), or null
+int latent_few(loom_b200_ctx* ctx, LbStack* st, int dt, const LbLatent& a, const float* raw, const float* norm, int tokens, float* ql, float* ol, float* part,
+               float* out, int ldo) {
+    if (int rc = lb_latent_absorb_q(ctx, dt, a, raw, a.ldq, norm, (float)st->d.norm_eps, tokens, ql)) return rc;
     if (dt == LOOM_B200_DTYPE_BF16 && lb_latent_step_supported(a))
         return lb_latent_step(ctx, a, tokens, ql, part, lb_latent_step_splits(ctx, a, tokens), out, ldo);
     if (int rc = lb_latent_attention(ctx, dt, a, tokens, ql, ol)) return rc;
@@ -339,9 +341,7 @@ int lb_stack_step(loom_b200_ctx* ctx, LbStack* st, const int* tok, const int* po
             LbLatent a = latent_of(st, l, st->proj, st->ldp);
             a.pos = pos;
             a.lane0 = lane0;
-            if (s.kv_from < 0)
-                if (int rc = lb_latent_store(ctx, dt, a, st->proj + s.heads * s.dim, st->ldp, l.mixer_norm, eps, M)) return rc;
-            if (int rc = latent_few(ctx, st, dt, a, M, st->ql, st->ol, st->attn_part, st->o, st->ldo)) return rc;
+            if (int rc = latent_few(ctx, st, dt, a, s.kv_from < 0 ? st->proj + s.heads * s.dim : nullptr, l.mixer_norm, M, st->ql, st->ol, st->attn_part, st->o, st->ldo)) return rc;
             out.x = st->o;
             out.ldx = st->ldo;
             if (int rc = lb_dense_gemv(ctx, dt, LB_DPRO_PLAIN, LB_DEPI_RESID, out)) return rc;
@@ -550,7 +550,7 @@ int lb_stack_block(loom_b200_ctx* ctx, LbStack* st, int T, int pos0, int lane) {
                     const int n = std::min(kLatentStepTokens, T - t0);
                     c.q = a.q + (size_t)t0 * a.ldq;
                     c.pos0 = pos0 + t0;
-                    if (int rc = latent_few(ctx, st, dt, c, n, st->pf_ql, st->pf_ol, st->pf_part, st->pf_o + (size_t)t0 * ldo, ldo)) return rc;
+                    if (int rc = latent_few(ctx, st, dt, c, nullptr, nullptr, n, st->pf_ql, st->pf_ol, st->pf_part, st->pf_o + (size_t)t0 * ldo, ldo)) return rc;
                 }
                 if (int rc = lb_rows_image(ctx, dt, st->pf_o, ldo, T, hv, oslices, st->pf_io)) return rc;
             }
