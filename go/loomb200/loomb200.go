@@ -394,6 +394,78 @@ func (dec *Decoder) ReadTokensBatch(batch, n int) ([]int32, error) {
 	return out, dec.ctx.check(rc)
 }
 
+// ---- float matrices and layer stacks: decoders whose layers are set one by one (no counterpart in poly) ----
+
+// Element types of a Matrix.
+const (
+	DTypeF32  = 0
+	DTypeBF16 = 1
+)
+
+// Matrix holds `groups` matrices of one shape as bf16 or float32 in the library's layout.
+type Matrix struct {
+	ctx *Context
+	m   *C.loom_b200_matrix
+}
+
+func (ctx *Context) NewMatrix(rows, cols, groups, dtype int) (*Matrix, error) {
+	m := &Matrix{ctx: ctx}
+	if err := ctx.check(C.loom_b200_matrix_create(ctx.c, C.int(rows), C.int(cols), C.int(groups), C.int(dtype), &m.m)); err != nil {
+		return nil, err
+	}
+	return m, nil
+}
+
+// PutF32 fills rows row0 ... of a group from row-major float32 values.
+func (m *Matrix) PutF32(group, row0, rows int, src []float32) error {
+	return m.ctx.check(C.loom_b200_matrix_put(m.ctx.c, m.m, C.int(group), C.int(row0), C.int(rows), unsafe.Pointer(&src[0]), DTypeF32, 0))
+}
+
+// PutBF16 does the same from bf16 bit patterns.
+func (m *Matrix) PutBF16(group, row0, rows int, src []uint16) error {
+	return m.ctx.check(C.loom_b200_matrix_put(m.ctx.c, m.m, C.int(group), C.int(row0), C.int(rows), unsafe.Pointer(&src[0]), DTypeBF16, 0))
+}
+
+func (m *Matrix) Free() {
+	if m.m != nil {
+		C.loom_b200_matrix_free(m.ctx.c, m.m)
+		m.m = nil
+	}
+}
+
+// StackDims, LayerSpec and LayerWeights are the C structures; LayerWeights borrows its matrices and copies its vectors.
+type StackDims = C.loom_b200_stack_dims
+type LayerSpec = C.loom_b200_layer_spec
+type LayerWeights = C.loom_b200_layer_weights
+
+// NewStackDecoder makes a decoder whose layers are set with SetLayer; Forward, Extend, Continue, Generate and the calls for
+// independent sequences work on it as on the ternary decoder.
+func (ctx *Context) NewStackDecoder(dims *StackDims) (*Decoder, error) {
+	dec := &Decoder{ctx: ctx}
+	if err := ctx.check(C.loom_b200_decoder_create_stack(ctx.c, dims, &dec.d)); err != nil {
+		return nil, err
+	}
+	return dec, nil
+}
+
+func (dec *Decoder) SetLayer(layer int, spec *LayerSpec, w *LayerWeights) error {
+	return dec.ctx.check(C.loom_b200_decoder_set_layer(dec.d, C.int(layer), spec, w))
+}
+
+// SetStackEmbeddings: table is a device address of [vocab, width] rows in the stack's dtype.
+func (dec *Decoder) SetStackEmbeddings(table uintptr, embedNorm float32, head *Matrix, finalNorm float32) error {
+	return dec.ctx.check(C.loom_b200_decoder_set_stack_embeddings(dec.d, unsafe.Pointer(table), C.float(embedNorm), head.m, C.float(finalNorm)))
+}
+
+// Extend appends tokens to the selected sequence; logits [len(want)*vocab] receives the rows after the tokens at those places.
+func (dec *Decoder) Extend(tokens, want []int32, logits []float32) error {
+	var w *C.int32_t
+	if len(want) > 0 {
+		w = (*C.int32_t)(unsafe.Pointer(&want[0]))
+	}
+	return dec.ctx.check(C.loom_b200_decoder_extend(dec.d, (*C.int32_t)(unsafe.Pointer(&tokens[0])), C.int(len(tokens)), w, C.int(len(want)), f32ptr(logits)))
+}
+
 func (dec *Decoder) Reset() error  { return dec.ctx.check(C.loom_b200_decoder_reset(dec.d)) }
 func (dec *Decoder) KVOffset() int { return int(C.loom_b200_decoder_kv_offset(dec.d)) }
 func (dec *Decoder) Close() {

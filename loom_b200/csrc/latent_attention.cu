@@ -318,7 +318,7 @@ __global__ void __launch_bounds__(kAtThreads, 2) lb_latent_block_kernel(const At
     __shared__ __align__(8) uint64_t bar_q, bar_k[2], bar_v[2], bar_s, bar_p, bar_o;
     __shared__ uint32_t tmem_base_s;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int nqb = lb_ceil_div(p.T, 128), qb = nqb - 1 - (int)blockIdx.x, h = blockIdx.y;  // the longest rows first
+    const int nqb = lb_ceil_div(p.T, 128), qb = nqb - 1 - (int)blockIdx.y, h = blockIdx.x;  // the longest rows of every head first
     const uint32_t qbytes = (uint32_t)p.dchunks * 2048, kbytes = (uint32_t)p.dchunks * 1024, vbytes = (uint32_t)p.vdim * 128;
     constexpr uint32_t kVStage = VC * 128;
     uint8_t *sq = sm, *sk = sq + qbytes, *sv = sk + 2 * kbytes, *sp = sv + 2 * kVStage;
@@ -440,13 +440,15 @@ __global__ void __launch_bounds__(kAtThreads, 2) lb_latent_block_kernel(const At
         if (tid == 0 && j + 2 < ntiles) load(j + 2);  // S_j and O_j are done: their stage is free
         __syncwarp();
         lb_tc_fence_after();
+        constexpr int VS = VC % 64 == 0 ? 64 : VC % 32 == 0 ? 32 : 16;  // columns per wait
 #pragma unroll
-        for (int c = 0; c < VC; c += 16) {
-            float v[16];
-            lb_tmem_ld16(tmem + lanes + kAtKeys + c, v);
+        for (int c = 0; c < VC; c += VS) {
+            float v[VS];
+#pragma unroll
+            for (int e = 0; e < VS; e += 16) lb_tmem_ld16(tmem + lanes + kAtKeys + c + e, v + e);
             lb_tmem_wait_ld();
 #pragma unroll
-            for (int e = 0; e < 16; ++e) o[c + e] = fmaf(o[c + e], f, v[e]);
+            for (int e = 0; e < VS; ++e) o[c + e] = fmaf(o[c + e], f, v[e]);
         }
     }
     if (failed) {
@@ -490,7 +492,7 @@ template <int VC>
 int launch_block(loom_b200_ctx* ctx, const AttnParams& p) {
     const size_t smem = (size_t)p.dchunks * (2048 + 2 * 1024) + 2 * VC * 128 + 16384;
     LB_BIG_SMEM(ctx, lb_latent_block_kernel<VC>, 220 * 1024);
-    LB_LAUNCH(ctx, lb_latent_block_kernel<VC>, dim3(lb_ceil_div(p.T, 128), p.heads), dim3(kAtThreads), smem, p);
+    LB_LAUNCH(ctx, lb_latent_block_kernel<VC>, dim3(p.heads, lb_ceil_div(p.T, 128)), dim3(kAtThreads), smem, p);
     return 0;
 }
 
