@@ -452,9 +452,10 @@ func (dec *Decoder) SetLayer(layer int, spec *LayerSpec, w *LayerWeights) error 
 	return dec.ctx.check(C.loom_b200_decoder_set_layer(dec.d, C.int(layer), spec, w))
 }
 
-// SetStackEmbeddings: table is a device address of [vocab, width] rows in the stack's dtype.
-func (dec *Decoder) SetStackEmbeddings(table uintptr, embedNorm float32, head *Matrix, finalNorm float32) error {
-	return dec.ctx.check(C.loom_b200_decoder_set_stack_embeddings(dec.d, unsafe.Pointer(table), C.float(embedNorm), head.m, C.float(finalNorm)))
+// SetStackEmbeddings: table is a device address of [vocab, width] rows in the stack's dtype, or 0 for the head's own rows;
+// finalNormW holds weights per column instead of finalNorm, or is nil.
+func (dec *Decoder) SetStackEmbeddings(table uintptr, embedNorm float32, head *Matrix, finalNorm float32, finalNormW []float32) error {
+	return dec.ctx.check(C.loom_b200_decoder_set_stack_embeddings(dec.d, unsafe.Pointer(table), C.float(embedNorm), head.m, C.float(finalNorm), f32ptr(finalNormW)))
 }
 
 // Extend appends tokens to the selected sequence; logits [len(want)*vocab] receives the rows after the tokens at those places.

@@ -403,9 +403,13 @@ void loom_b200_matrix_free(loom_b200_ctx* ctx, loom_b200_matrix* m);
 
 #define LOOM_B200_MIXER_GLA 0    /* gated linear attention, one decay per key channel */
 #define LOOM_B200_MIXER_LATENT 1 /* softmax attention over cached latents, no positions */
+#define LOOM_B200_MIXER_ATTENTION 2 /* softmax attention over cached keys and values of grouped heads */
+#define LOOM_B200_MIXER_DELTA 3  /* gated delta rule: one decay per head, short convolutions on q, k and v */
+#define LOOM_B200_MIXER_MLSTM 4  /* matrix memory with exponential gates, a normaliser and a running maximum */
 #define LOOM_B200_FFN_NONE 0
 #define LOOM_B200_FFN_DENSE 1    /* down(gelu(up h)), exact gelu */
 #define LOOM_B200_FFN_MOE 2      /* routed experts with the clamped gated unit; sigmoid scores, not renormalised, on the experts' input */
+#define LOOM_B200_FFN_GATED 3    /* down(silu(gate h) * (up h)) */
 
 typedef struct loom_b200_stack_dims {
     int num_layers, width, vocab;
@@ -413,7 +417,9 @@ typedef struct loom_b200_stack_dims {
     int dtype;             /* LOOM_B200_DTYPE_*: matrices, activations of the products and the latent cache */
     int conv_taps;         /* taps of the short convolution in front of a mixer (layers without weights for it have none) */
     double norm_eps;       /* every RMS norm: x / sqrt(mean(x^2) + eps) */
-    double residual_mult;  /* x += residual_mult * branch */
+    double residual_mult;  /* factor of a branch in the residual sum */
+    int post_norm;         /* 0: x <- x + residual_mult * branch(norm(x)); 1: x <- norm(residual_alpha * x + residual_mult * branch(x)) */
+    double residual_alpha; /* post_norm: factor of x in the sum */
 } loom_b200_stack_dims;
 
 typedef struct loom_b200_layer_spec {
@@ -427,28 +433,47 @@ typedef struct loom_b200_layer_spec {
     int ff;                /* inner size (of one expert) */
     int experts, top;
     double limit;          /* clamp of the gated unit */
+    int kv_heads;          /* attention, delta rule: heads of k (and of v in attention, of q in the delta rule); divides heads */
+    int chunk;             /* attention: position i sees j <= i with i / chunk == j / chunk; 0: every j <= i */
+    int buckets;           /* attention: rows of the distance bias, 0 for none */
+    double bias_max;       /* attention: distance from which on the last bucket is used */
+    int qk_norm;           /* attention: q and k divided by their root mean square, per head */
+    int sink;              /* attention: one added to the softmax's denominator (a score of 0 without a value) */
+    int head_gate;         /* attention: every head's output times the sigmoid of one projected number */
+    int conv;              /* delta rule: taps of the convolutions (the last belongs to the current token) */
+    double gate_cap;       /* matrix memory: gates pass cap * tanh(z / cap) */
 } loom_b200_layer_spec;
 
 /* Matrices are borrowed and must outlive the decoder; vectors are host float32 and are copied. */
 typedef struct loom_b200_layer_weights {
     const loom_b200_matrix* in;   /* GLA: rows q, k [heads*dim], v, gate [heads*vdim], decay input [rank]; latent: q [heads*dim] and,
-                                     unless kv_from is set, the latent projection [rank] */
+                                     unless kv_from is set, the latent projection [rank]; attention: q [heads*dim], k [kv_heads*dim],
+                                     v [kv_heads*vdim] and with head_gate the gate [heads]; delta rule: q, k [kv_heads*dim], v, gate
+                                     [heads*vdim], write strength, decay input [heads]; matrix memory: q, k [heads*dim], v, gate
+                                     [heads*vdim], input gate, forget gate [heads] */
     const loom_b200_matrix* out;  /* [width, heads*vdim] */
     const loom_b200_matrix *up_k, *up_v;          /* latent: [heads*dim, rank], [heads*vdim, rank] */
-    const float* mixer_norm;      /* GLA: [vdim] norm of every head's output; latent: [rank] norm of the latent */
+    const float* mixer_norm;      /* GLA, delta rule: [vdim] norm of every head's output; latent: [rank] norm of the latent; matrix
+                                     memory: [heads*vdim] */
     const float *decay_w, *decay_b;               /* GLA: [heads*dim, rank], [heads*dim] */
     const float* conv_w;          /* [width, conv_taps] or NULL */
     float norm1, norm2;           /* gains of the norms in front of the mixer and the feed-forward */
     const loom_b200_matrix *router;               /* [experts, width] */
-    const loom_b200_matrix *gate, *up, *down;     /* dense: up [ff, width], down [width, ff]; experts: one group each */
+    const loom_b200_matrix *gate, *up, *down;     /* dense: up [ff, width], down [width, ff]; gated: gate too; experts: one group each */
+    const float *norm1_w, *norm2_w;               /* [width] weights of the two norms instead of the gains, or NULL */
+    const float* rel;             /* attention: [buckets, heads] distance bias, added to the scaled score */
+    const float* conv_qkv;        /* delta rule: [2*kv_heads*dim + heads*vdim, conv] */
+    const float *a_log, *dt_bias; /* delta rule: [heads]; decay = exp(-exp(a_log) softplus(input + dt_bias)) */
+    const float *gate_b_i, *gate_b_f;             /* matrix memory: [heads] biases of the two gates */
 } loom_b200_layer_weights;
 
 int loom_b200_decoder_create_stack(loom_b200_ctx* ctx, const loom_b200_stack_dims* dims, loom_b200_decoder** out);
 /* after decoder_set_batch (if any): the states of every sequence are allocated here */
 int loom_b200_decoder_set_layer(loom_b200_decoder* dec, int layer, const loom_b200_layer_spec* spec, const loom_b200_layer_weights* weights);
-/* table: [vocab, width] in the stack's dtype, row-major device memory (borrowed); head [vocab, width] (borrowed) */
+/* table: [vocab, width] in the stack's dtype, row-major device memory (borrowed), or NULL: the rows of the head, not normed (tied);
+ * head [vocab, width] (borrowed); final_norm_w: [width] weights of the last norm instead of its gain, or NULL */
 int loom_b200_decoder_set_stack_embeddings(loom_b200_decoder* dec, const void* table_dev, float embed_norm, const loom_b200_matrix* head,
-                                           float final_norm);
+                                           float final_norm, const float* final_norm_w);
 /* Appends n tokens to the selected sequence from whatever state it is in (reset starts it anew) and returns the logits after
  * the tokens at places want[0..n_want) of this call (ascending), [n_want, vocab].  A prompt may be cut into calls anywhere.
  * Ternary decoders take it too, with want empty or the last place only. */

@@ -17,8 +17,8 @@ ACT_RELU, ACT_SILU, ACT_GELU, ACT_TANH, ACT_SIGMOID, ACT_LEAKY_RELU, ACT_RELU2, 
 
 DTYPE_F32, DTYPE_BF16 = 0, 1
 DTYPES = {"float32": DTYPE_F32, "bfloat16": DTYPE_BF16}
-MIXER_GLA, MIXER_LATENT = 0, 1
-FFN_NONE, FFN_DENSE, FFN_MOE = 0, 1, 2
+MIXER_GLA, MIXER_LATENT, MIXER_ATTENTION, MIXER_DELTA, MIXER_MLSTM = range(5)
+FFN_NONE, FFN_DENSE, FFN_MOE, FFN_GATED = range(4)
 
 ERR_INVALID, ERR_CUDA, ERR_UNSUPPORTED, ERR_NO_DEVICE, ERR_TIMEOUT, ERR_COMM = -1, -2, -3, -4, -5, -6
 
@@ -119,7 +119,7 @@ SIGNATURES = {
     "loom_b200_matrix_free": (None, [_vp, _vp]),
     "loom_b200_decoder_create_stack": (_i, [_vp, _vp, C.POINTER(_vp)]),
     "loom_b200_decoder_set_layer": (_i, [_vp, _i, _vp, _vp]),
-    "loom_b200_decoder_set_stack_embeddings": (_i, [_vp, _vp, _f, _vp, _f]),
+    "loom_b200_decoder_set_stack_embeddings": (_i, [_vp, _vp, _f, _vp, _f, _vp]),
     "loom_b200_decoder_extend": (_i, [_vp, _vp, _i, _vp, _i, _vp]),
     "loom_b200_tp_unique_id": (_i, [_vp]),
     "loom_b200_tp_init": (_i, [_vp, _i, _i, _vp]),
@@ -141,17 +141,19 @@ class DecoderDims(C.Structure):
 
 class StackDims(C.Structure):
     _fields_ = [("num_layers", _i), ("width", _i), ("vocab", _i), ("max_seq_len", _i), ("dtype", _i), ("conv_taps", _i), ("norm_eps", _d),
-                ("residual_mult", _d)]
+                ("residual_mult", _d), ("post_norm", _i), ("residual_alpha", _d)]
 
 
 class LayerSpec(C.Structure):
     _fields_ = [("mixer", _i), ("heads", _i), ("dim", _i), ("vdim", _i), ("rank", _i), ("kv_from", _i), ("tau", _d), ("scale", _d), ("ffn", _i),
-                ("ff", _i), ("experts", _i), ("top", _i), ("limit", _d)]
+                ("ff", _i), ("experts", _i), ("top", _i), ("limit", _d), ("kv_heads", _i), ("chunk", _i), ("buckets", _i), ("bias_max", _d),
+                ("qk_norm", _i), ("sink", _i), ("head_gate", _i), ("conv", _i), ("gate_cap", _d)]
 
 
 class LayerWeights(C.Structure):
     _fields_ = [("in_", _vp), ("out", _vp), ("up_k", _vp), ("up_v", _vp), ("mixer_norm", _vp), ("decay_w", _vp), ("decay_b", _vp), ("conv_w", _vp),
-                ("norm1", _f), ("norm2", _f), ("router", _vp), ("gate", _vp), ("up", _vp), ("down", _vp)]
+                ("norm1", _f), ("norm2", _f), ("router", _vp), ("gate", _vp), ("up", _vp), ("down", _vp),
+                ("norm1_w", _vp), ("norm2_w", _vp), ("rel", _vp), ("conv_qkv", _vp), ("a_log", _vp), ("dt_bias", _vp), ("gate_b_i", _vp), ("gate_b_f", _vp)]
 
 
 class GenMetrics(C.Structure):
@@ -557,11 +559,13 @@ class Decoder:
         self._keep = []
 
     @classmethod
-    def stack(cls, ctx: Context, layers, width, vocab, eps, residual_mult=1.0, conv_taps=0, dtype=DTYPE_BF16, max_seq_len=2048) -> "Decoder":
+    def stack(cls, ctx: Context, layers, width, vocab, eps, residual_mult=1.0, conv_taps=0, dtype=DTYPE_BF16, max_seq_len=2048,
+              residual_alpha=None) -> "Decoder":
+        """residual_alpha: norms after the sum, with this factor of the residual in it (None: norms in front of the branches)."""
         self = cls.__new__(cls)
         self.ctx, self.h, self._keep = ctx, None, []
         self.dims = DecoderDims(layers, width, 0, 0, 0, 0, vocab, eps, 0.0, ACT_LINEAR, max_seq_len)
-        d = StackDims(layers, width, vocab, max_seq_len, dtype, conv_taps, eps, residual_mult)
+        d = StackDims(layers, width, vocab, max_seq_len, dtype, conv_taps, eps, residual_mult, residual_alpha is not None, residual_alpha or 0.0)
         h = _vp()
         ctx._check(lib().loom_b200_decoder_create_stack(ctx.h, C.byref(d), C.byref(h)))
         self.h = h
@@ -584,10 +588,12 @@ class Decoder:
             setattr(w, "in_" if name == "in" else name, value)
         self.ctx._check(lib().loom_b200_decoder_set_layer(self.h, i, C.byref(s), C.byref(w)))
 
-    def set_stack_embeddings(self, table_dev, embed_norm: float, head: Matrix, final_norm: float):
-        """table_dev: [vocab, width] on the device in the stack's dtype."""
+    def set_stack_embeddings(self, table_dev, embed_norm: float, head: Matrix, final_norm):
+        """table_dev: [vocab, width] on the device in the stack's dtype, or None: the head's rows as they are; final_norm: one gain or a
+        vector of weights."""
         self._keep += [table_dev, head]
-        self.ctx._check(lib().loom_b200_decoder_set_stack_embeddings(self.h, _ptr(table_dev), float(embed_norm), head.h, float(final_norm)))
+        w = None if np.ndim(final_norm) == 0 else _f32(final_norm)
+        self.ctx._check(lib().loom_b200_decoder_set_stack_embeddings(self.h, _ptr(table_dev), float(embed_norm), head.h, float(final_norm) if w is None else 1.0, _hp(w)))
 
     def extend(self, tokens, want=()):
         """Appends tokens to the selected sequence; the logits [len(want), vocab] after the tokens at the places `want` (ascending)."""

@@ -631,7 +631,11 @@ int dec_step(loom_b200_decoder* dec, bool host_token) {
     const bool in_frame = !dec->fused_tail;  // without the fused tail the gather is the first launch of the frame
     if (dec->fused_tail && host_token && !dec->stack)  // (a stack's step starts with its own gather)
         if (int rc = lb_launch_embed(ctx, dec->emb, d.vocab, d.hidden, dec->cur_tok, 1, dec->x)) return rc;
-    if (dec->step_graph) return loom_b200_graph_launch(ctx, dec->step_graph);
+    if (dec->step_graph) {
+        dec->last_resid = dec->stack ? dec->stack->x : dec->x;
+        dec->last_resid_rows = 1;
+        return loom_b200_graph_launch(ctx, dec->step_graph);
+    }
     if (dec->tp_world > 1 && !ctx->opt_tp_graph) return dec_forward_chunk(dec, 1, dec->decode_splits, true, 0, false, in_frame, dec->cur_tok);
     if (int rc = dec_forward_chunk(dec, 1, dec->decode_splits, true, 0, false, in_frame, dec->cur_tok)) return rc;  // warm-up run, counts as the step
     // record the same step for all later tokens
@@ -822,11 +826,11 @@ int loom_b200_decoder_set_layer(loom_b200_decoder* dec, int layer, const loom_b2
 }
 
 int loom_b200_decoder_set_stack_embeddings(loom_b200_decoder* dec, const void* table_dev, float embed_norm, const loom_b200_matrix* head,
-                                           float final_norm) {
+                                           float final_norm, const float* final_norm_w) {
     if (!dec) return lb_fail(nullptr, LOOM_B200_ERR_INVALID, "decoder_set_stack_embeddings: decoder is NULL");
     loom_b200_ctx* ctx = dec->ctx;
     LB_REQUIRE(ctx, dec->stack, "decoder_set_stack_embeddings: not a layer stack");
-    LB_REQUIRE(ctx, table_dev && head, "decoder_set_stack_embeddings: NULL argument");
+    LB_REQUIRE(ctx, head, "decoder_set_stack_embeddings: NULL argument");
     LbStack* st = dec->stack;
     LB_REQUIRE(ctx, head->rows == st->d.vocab && head->cols == st->d.width && head->dtype == st->d.dtype && head->groups == 1,
                "decoder_set_stack_embeddings: head is %dx%d, expected %dx%d of the stack's dtype", head->rows, head->cols, st->d.vocab, st->d.width);
@@ -838,6 +842,10 @@ int loom_b200_decoder_set_stack_embeddings(loom_b200_decoder* dec, const void* t
     const float scal[2] = {embed_norm, final_norm};
     if (!st->scal) LB_CUDA(ctx, cudaMalloc(&st->scal, sizeof(scal)));
     LB_CUDA(ctx, cudaMemcpyAsync(st->scal, scal, sizeof(scal), cudaMemcpyHostToDevice, ctx->stream));
+    if (final_norm_w) {
+        if (!st->final_w) LB_CUDA(ctx, cudaMalloc(&st->final_w, (size_t)st->d.width * sizeof(float)));
+        LB_CUDA(ctx, cudaMemcpyAsync(st->final_w, final_norm_w, (size_t)st->d.width * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
+    }
     LB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
     return 0;
 }

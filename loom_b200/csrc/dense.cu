@@ -160,7 +160,7 @@ template <typename WT, int PRO, int EPI>
 __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const LbDenseGemv p, int Mp_launch, int KW, bool vec) {
     extern __shared__ __align__(16) uint8_t smem[];
     constexpr int C = LbElem<WT>::kChunk;
-    constexpr bool kDual = EPI == LB_DEPI_GLU;
+    constexpr bool kDual = EPI == LB_DEPI_GLU || EPI == LB_DEPI_SILU;
     constexpr int NB = kDual ? 1 : 2;
     __shared__ float red[kGemvWarps][128];
     __shared__ float red2[kDual ? kGemvWarps : 1][128];
@@ -181,7 +181,10 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
     int strip = (int)blockIdx.x * SP + sp;
     auto strip_ptr = [&](const uint8_t* base, int st) { return base + (size_t)(st >> 3) * p.slices * kImgBlock + (size_t)(st & 7) * 2048; };
     constexpr bool kEarly = PRO != LB_DPRO_MOE && PRO != LB_DPRO_PAIRS && !kStage;
-    if (kEarly && strip < strips) load_batch(cur, strip_ptr(w1, strip), kw, KW, p.slices, g, t);
+    if (kEarly && strip < strips) {
+        load_batch(cur, strip_ptr(w1, strip), kw, KW, p.slices, g, t);
+        if (kDual) load_batch(cur2, strip_ptr(w2, strip), kw, KW, p.slices, g, t);
+    }
     lb_pdl_launch_dependents();
     lb_pdl_wait();
 
@@ -290,7 +293,7 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
             float tot = 0.f;
             for (int i = 0; i < WPT; ++i) tot += s_stat[m * WPT + i];
             rstd = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(tot, (float)p.K), p.eps)));
-            gain = *p.gain;
+            if (p.gain) gain = *p.gain;
         }
         if (PRO == LB_DPRO_GATED) {
             heads = p.K / p.head_dim;
@@ -318,18 +321,30 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
                 if (PRO == LB_DPRO_NORM || PRO == LB_DPRO_CONV || PRO == LB_DPRO_MOE) {
 #pragma unroll
                     for (int i = 0; i < C; ++i) f[i] = f[i] * rstd * gain;
+                    if (p.gain_w) {
+                        float w[C];
+                        lb_load_cols<C>(p.gain_w, k0, p.K, vec, w);
+#pragma unroll
+                        for (int i = 0; i < C; ++i) f[i] *= w[i];
+                    }
+                    if (PRO == LB_DPRO_NORM && p.x_out && (kStage || blockIdx.x == 0)) {
+#pragma unroll
+                        for (int i = 0; i < C; ++i)
+                            if (k0 + i < p.K) p.x_out[(size_t)tok * p.ldx + k0 + i] = f[i];
+                    }
                 }
                 if (PRO == LB_DPRO_MOE) {
 #pragma unroll
                     for (int i = 0; i < C; ++i) f[i] *= s_w[m];
                 }
                 if (PRO == LB_DPRO_GATED) {
-                    float gt[C];
+                    float gt[C], hw[C];
                     lb_load_cols<C>(p.gate + (size_t)tok * p.gate_ld, k0, p.K, vec, gt);
+                    lb_load_cols<C>(p.head_w, k0, p.K, vec, hw);
 #pragma unroll
                     for (int i = 0; i < C; ++i) {
                         const int k = k0 + i, h = k / p.head_dim;
-                        if (k < p.K) f[i] = f[i] * s_head[h] * p.head_w[k - h * p.head_dim] * lb_siluf(gt[i]);
+                        if (k < p.K) f[i] = f[i] * s_head[h] * hw[i] * (p.gate_sigmoid ? lb_sigmoidf(gt[i]) : lb_siluf(gt[i]));
                     }
                 }
                 if (PRO == LB_DPRO_CONV) {
@@ -446,10 +461,11 @@ __global__ void __launch_bounds__(kGemvThreads, 2) lb_dense_gemv_kernel(const Lb
             }
             if (EPI == LB_DEPI_F32) p.out[(size_t)m * p.ldo + row] = v;
             if (EPI == LB_DEPI_RESID) {
-                float* y = p.out + (size_t)m * p.ldo + row;
-                *y = fmaf(p.mult, v, *y);
+                const size_t at = (size_t)m * p.ldo + row;
+                p.out[at] = fmaf(p.mult, v, p.res_mult * (p.res ? p.res : p.out)[at]);
             }
             if (EPI == LB_DEPI_GELU) p.out[(size_t)m * p.ldo + row] = lb_gelu_erff(v);
+            if (EPI == LB_DEPI_SILU) p.out[(size_t)m * p.ldo + row] = lb_siluf(v) * u;
             if (EPI == LB_DEPI_GLU) {
                 reinterpret_cast<WT*>(p.out_pairs)[(size_t)s_pair[m] * p.ldo + row] = (WT)lb_clamped_glu(v, u, p.limit);
             }
@@ -472,7 +488,8 @@ int gemv_launch(loom_b200_ctx* ctx, const LbDenseGemv& pin) {
     while (KW > 1 && (long long)strips >= 6ll * (2 * kGemvWarps / KW) * cap) KW /= 2;
     const int SP = kGemvWarps / KW;
     bool vec = PRO == LB_DPRO_STAGED || PRO == LB_DPRO_PAIRS || lb_vec_rows(p.x, p.ldx);
-    if (PRO == LB_DPRO_GATED) vec = vec && lb_vec_rows(p.gate, p.gate_ld);
+    if (PRO == LB_DPRO_GATED) vec = vec && lb_vec_rows(p.gate, p.gate_ld) && lb_vec_rows(p.head_w, 4);
+    if (p.gain_w) vec = vec && lb_vec_rows(p.gain_w, 4);
     if (PRO == LB_DPRO_CONV) vec = vec && lb_vec_rows(p.conv_w, p.ring_ld) && lb_vec_rows(p.conv_ring, p.ring_ld);
     const size_t rows_smem = (size_t)p.slices * 8 * (EPI == LB_DEPI_STAGE ? 1 : Mp) * 16;
     size_t smem = PRO == LB_DPRO_PAIRS || EPI == LB_DEPI_STAGE ? 0 : rows_smem;
@@ -520,6 +537,8 @@ int gemv_dispatch(loom_b200_ctx* ctx, int pro, int epi, const LbDenseGemv& p) {
     LB_CASE(LB_DPRO_CONV, LB_DEPI_F32, gemv_rows);
     LB_CASE(LB_DPRO_NORM, LB_DEPI_F32, gemv_rows);
     LB_CASE(LB_DPRO_NORM, LB_DEPI_GELU, gemv_rows);
+    LB_CASE(LB_DPRO_NORM, LB_DEPI_SILU, gemv_rows);
+    LB_CASE(LB_DPRO_PLAIN, LB_DEPI_F32, gemv_launch);
     LB_CASE(LB_DPRO_PLAIN, LB_DEPI_RESID, gemv_launch);
     LB_CASE(LB_DPRO_GATED, LB_DEPI_RESID, gemv_rows);
     LB_CASE(LB_DPRO_MOE, LB_DEPI_GLU, gemv_launch);
@@ -535,7 +554,7 @@ constexpr int kSimtTile = 64;
 template <typename WT, int EPI>
 __global__ void __launch_bounds__(256) lb_dense_gemm_simt_kernel(const LbDenseGemm p) {
     constexpr int C = LbElem<WT>::kChunk;
-    constexpr bool kDual = EPI == LB_DEPI_GLU;
+    constexpr bool kDual = EPI == LB_DEPI_GLU || EPI == LB_DEPI_SILU;
     __shared__ __align__(16) uint8_t sa[8192], sb[8192], sb2[kDual ? 8192 : 16];
     lb_pdl_launch_dependents();
     lb_pdl_wait();
@@ -594,7 +613,7 @@ __global__ void __launch_bounds__(256) lb_dense_gemm_simt_kernel(const LbDenseGe
             if (r >= p.ldo) continue;
             float* o = p.out + (size_t)tok * p.ldo + r;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) o[j] = EPI == LB_DEPI_F32 ? acc[i][j] : fmaf(p.mult, acc[i][j], o[j]);
+            for (int j = 0; j < 8; ++j) o[j] = EPI == LB_DEPI_F32 ? acc[i][j] : fmaf(p.mult, acc[i][j], p.res_mult * o[j]);
         } else {
             float f[8];
 #pragma unroll
@@ -602,6 +621,7 @@ __global__ void __launch_bounds__(256) lb_dense_gemm_simt_kernel(const LbDenseGe
                 f[j] = acc[i][j];
                 if (EPI == LB_DEPI_GELU) f[j] = lb_gelu_erff(acc[i][j]);
                 if (EPI == LB_DEPI_GLU) f[j] = lb_clamped_glu(acc[i][j], acc2[i][j], p.limit);
+                if (EPI == LB_DEPI_SILU) f[j] = lb_siluf(acc[i][j]) * acc2[i][j];
             }
             if (EPI == LB_DEPI_HEADS) {
                 if (r < p.rows) *reinterpret_cast<uint4*>(p.img + lb_heads_chunk(tok, r, p.heads, p.head_dim, p.head_chunks)) = lb_pack_chunk<__nv_bfloat16>(f);
@@ -627,6 +647,7 @@ int gemm_simt(loom_b200_ctx* ctx, int epi, const LbDenseGemm& p) {
     LB_CASE(LB_DEPI_RESID)
     LB_CASE(LB_DEPI_GELU)
     LB_CASE(LB_DEPI_GLU)
+    LB_CASE(LB_DEPI_SILU)
     LB_CASE(LB_DEPI_IMG)
     LB_CASE(LB_DEPI_HEADS)
 #undef LB_CASE

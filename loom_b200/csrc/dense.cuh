@@ -143,20 +143,21 @@ __device__ __forceinline__ float lb_log_sigmoidf(float z) { return fminf(z, 0.f)
 
 enum LbDensePro : int {
     LB_DPRO_PLAIN = 0,  // x [M, ldx] as it is
-    LB_DPRO_NORM = 1,   // RMS norm with one gain
+    LB_DPRO_NORM = 1,   // RMS norm with one gain or a weight per column; the normed row may be kept
     LB_DPRO_CONV = 2,   // RMS norm with one gain, then h + causal depthwise convolution of h over time
-    LB_DPRO_GATED = 3,  // per-head RMS norm with a weight, times silu of a gate row (output of gated linear attention)
+    LB_DPRO_GATED = 3,  // per-head RMS norm with a weight, times silu or sigmoid of a gate row (output of a recurrent mixer)
     LB_DPRO_MOE = 4,    // routed experts: top-k of the router's logits, RMS norm, times the token's weight for the expert
     LB_DPRO_PAIRS = 5,  // routed experts, second product: one row per (token, choice), summed over the choices
     LB_DPRO_STAGED = 6, // input rows already made by a launch of their own (several tokens; chosen by the launcher)
 };
 enum LbDenseEpi : int {
     LB_DEPI_F32 = 0,    // out [token, ldo] = acc
-    LB_DEPI_RESID = 1,  // out [token, ldo] += mult * acc
+    LB_DEPI_RESID = 1,  // out [token, ldo] = res_mult * res + mult * acc
     LB_DEPI_GELU = 2,   // exact gelu (GEMV: float rows, GEMM: image)
     LB_DEPI_GLU = 3,    // clamped gated unit of two products (GEMV: rows of WT per pair, GEMM: image)
     LB_DEPI_IMG = 4,    // GEMM only: image
     LB_DEPI_STAGE = 6,  // GEMV: only the prologue, a CTA per token, into `staged`
+    LB_DEPI_SILU = 7,   // silu of the first product times the second (GEMV: float rows, GEMM: image)
     LB_DEPI_HEADS = 5,  // GEMM only: per-head blocks [token block of 128][head][token/8][chunk][token%8][16 B]
 };
 
@@ -172,14 +173,16 @@ struct LbRouteList {
 
 struct LbDenseGemv {
     const uint8_t* w = nullptr;   // image
-    const uint8_t* w2 = nullptr;  // GLU: the second matrix
+    const uint8_t* w2 = nullptr;  // GLU, SILU: the second matrix
     size_t group_bytes = 0;       // routed: distance of two experts' images
     int rows = 0, K = 0, slices = 0, M = 0;
     // input
     const float* x = nullptr;
     int ldx = 0;
     const int* row_idx = nullptr;  // token m reads row row_idx[m] of x (null: m)
-    const float* gain = nullptr;   // one float
+    const float* gain = nullptr;   // one float, or null: 1
+    const float* gain_w = nullptr; // [K], or null: 1
+    float* x_out = nullptr;        // NORM: the normed rows [M, ldx], or null
     float eps = 0.f;
     // convolution: weights [taps][ring_ld], ring [lane][taps][ring_ld] of normed inputs (slot = position % taps)
     const float* conv_w = nullptr;
@@ -190,8 +193,9 @@ struct LbDenseGemv {
     // gated heads
     const float* gate = nullptr;  // [M, gate_ld]
     int gate_ld = 0;
-    const float* head_w = nullptr;
+    const float* head_w = nullptr;  // [K]
     int head_dim = 0;
+    bool gate_sigmoid = false;      // (silu otherwise)
     // routing
     const float* logits = nullptr;  // [M, ldl]
     int ldl = 0, experts = 0, top = 0;
@@ -203,7 +207,8 @@ struct LbDenseGemv {
     float* out = nullptr;
     uint8_t* out_pairs = nullptr;
     int ldo = 0;
-    float mult = 1.f, limit = 0.f;
+    const float* res = nullptr;  // RESID: [M, ldo], null: out itself
+    float mult = 1.f, res_mult = 1.f, limit = 0.f;
 };
 int lb_dense_gemv(loom_b200_ctx* ctx, int dtype, int pro, int epi, const LbDenseGemv& p);
 // tokens of one pass: what the input rows leave room for
@@ -214,7 +219,7 @@ int lb_dense_gemv_max_tokens(int K, int dtype);
 struct LbDenseGemm {
     const uint8_t* x = nullptr;  // token image
     const uint8_t* w = nullptr;
-    const uint8_t* w2 = nullptr;  // GLU
+    const uint8_t* w2 = nullptr;  // GLU, SILU
     size_t group_bytes = 0;
     int tokens = 0, rows = 0, slices = 0;
     // routed: the rows of x are grouped by expert in whole blocks of 128; *nblocks of them are in use
@@ -225,7 +230,7 @@ struct LbDenseGemm {
     uint8_t* img = nullptr;
     int ldo = 0, img_slices = 0;
     int heads = 0, head_dim = 0, head_chunks = 0;  // per-head blocks: head_dim % 8 == 0, head_chunks 16-byte chunks per row
-    float mult = 1.f, limit = 0.f;
+    float mult = 1.f, res_mult = 1.f, limit = 0.f;  // RESID: out = res_mult * out + mult * acc
     int* status = nullptr;
 };
 int lb_dense_gemm(loom_b200_ctx* ctx, int dtype, int epi, const LbDenseGemm& p);

@@ -91,7 +91,7 @@ __device__ __forceinline__ float warp_sum16(float* v, int lane) {
 }
 
 // CTA = (chunk, head): decays, the scaled queries and keys and the chunk's token-by-token weights
-__global__ void __launch_bounds__(kPrepThreads, 2) lb_gla_prep_kernel(const LbGla p, const LbGlaBlock b, int T) {
+__global__ void __launch_bounds__(kPrepThreads, 2) lb_gla_prep_kernel(const LbGla p, const LbChunks b, int T) {
     extern __shared__ __align__(16) float sm[];
     lb_pdl_launch_dependents();
     lb_pdl_wait();
@@ -288,42 +288,42 @@ __device__ __forceinline__ void tile_cols(float (*s)[kTileLd], const float* m, s
 }
 
 // what a chunk adds to the state: CTA = (64 channels x 64 value columns, head, chunk)
-__global__ void __launch_bounds__(kTileThreads) lb_gla_state_kernel(const LbGla p, const LbGlaBlock b, int T, int dtiles, bool vec) {
+__global__ void __launch_bounds__(kTileThreads) lb_chunk_state_kernel(const LbChunks b, int T, int dtiles, bool vec) {
     __shared__ __align__(16) float sa[kTileK][kTileLd], sb[kTileK][kTileLd];
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const int d0 = (blockIdx.x % dtiles) * kTile, v0 = (blockIdx.x / dtiles) * kTile, h = blockIdx.y, ch = blockIdx.z, tid = threadIdx.x;
-    const int HD = p.heads * p.dim, t0 = ch * b.C, n = min(b.C, T - t0), ty = tid >> 4, tx = tid & 15;
+    const int HD = b.heads * b.dim, t0 = ch * b.C, n = min(b.C, T - t0), ty = tid >> 4, tx = tid & 15;
     float acc[8][4] = {};
     for (int s0 = 0; s0 < n; s0 += kTileK) {
         __syncthreads();
-        tile_rows(sa, b.kd + (size_t)(t0 + s0) * HD + h * p.dim, HD, n - s0, d0, p.dim, vec);
-        tile_rows(sb, p.proj + (size_t)(t0 + s0) * p.ldp + 2 * HD + h * p.vdim, p.ldp, n - s0, v0, p.vdim, vec);
+        tile_rows(sa, b.kd + (size_t)(t0 + s0) * HD + h * b.dim, HD, n - s0, d0, b.dim, vec);
+        tile_rows(sb, b.v + (size_t)(t0 + s0) * b.ldv + h * b.vdim, b.ldv, n - s0, v0, b.vdim, vec);
         __syncthreads();
         tile_fma(sa, sb, ty, tx, acc);
     }
-    float* out = b.states + ((size_t)ch * p.heads + h) * p.dim * p.vdim;
+    float* out = b.states + ((size_t)ch * b.heads + h) * b.dim * b.vdim;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int d = d0 + ty * 8 + i, v = v0 + tx * 4;
-        if (d >= p.dim) continue;
-        if (vec && v + 4 <= p.vdim)
-            *reinterpret_cast<float4*>(out + (size_t)d * p.vdim + v) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+        if (d >= b.dim) continue;
+        if (vec && v + 4 <= b.vdim)
+            *reinterpret_cast<float4*>(out + (size_t)d * b.vdim + v) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
         else
 #pragma unroll
             for (int j = 0; j < 4; ++j)
-                if (v + j < p.vdim) out[(size_t)d * p.vdim + v + j] = acc[i][j];
+                if (v + j < b.vdim) out[(size_t)d * b.vdim + v + j] = acc[i][j];
     }
 }
 
 // what the chunks add -> the state in front of every chunk, in place; the last state becomes the sequence's
-__global__ void __launch_bounds__(256) lb_gla_scan_kernel(const LbGla p, const LbGlaBlock b, int chunks, int fresh) {
+__global__ void __launch_bounds__(256) lb_chunk_scan_kernel(const LbChunks b, int chunks, int fresh) {
     lb_pdl_launch_dependents();
     lb_pdl_wait();
-    const size_t all = (size_t)p.heads * p.dim * p.vdim, i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    const size_t all = (size_t)b.heads * b.dim * b.vdim, i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= all) return;
-    const size_t hd = i / p.vdim;
-    float s = fresh ? 0.f : p.state[i];
+    const size_t hd = i / b.vdim;
+    float s = fresh ? 0.f : b.state[i];
     constexpr int U = 8;
     for (int c0 = 0; c0 < chunks; c0 += U) {
         float add[U], dec[U];
@@ -331,7 +331,7 @@ __global__ void __launch_bounds__(256) lb_gla_scan_kernel(const LbGla p, const L
         for (int u = 0; u < U; ++u) {
             const int c = c0 + u;
             add[u] = c < chunks ? b.states[(size_t)c * all + i] : 0.f;
-            dec[u] = c < chunks ? b.decay[(size_t)c * p.heads * p.dim + hd] : 1.f;
+            dec[u] = c < chunks ? b.decay[(size_t)c * b.heads * b.dim + hd] : 1.f;
         }
 #pragma unroll
         for (int u = 0; u < U; ++u) {
@@ -339,30 +339,30 @@ __global__ void __launch_bounds__(256) lb_gla_scan_kernel(const LbGla p, const L
             s = fmaf(dec[u], s, add[u]);
         }
     }
-    p.state[i] = s;
+    b.state[i] = s;
 }
 
 // outputs: CTA = (64 value columns, head, chunk): (scaled queries | weights) times (state | values)
-__global__ void __launch_bounds__(kTileThreads) lb_gla_out_kernel(const LbGla p, const LbGlaBlock b, int T, bool vec) {
+__global__ void __launch_bounds__(kTileThreads) lb_chunk_out_kernel(const LbChunks b, int T, bool vec) {
     __shared__ __align__(16) float sa[kTileK][kTileLd], sb[kTileK][kTileLd];
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const int v0 = blockIdx.x * kTile, h = blockIdx.y, ch = blockIdx.z, tid = threadIdx.x, C = b.C;
-    const int HD = p.heads * p.dim, t0 = ch * C, n = min(C, T - t0), ty = tid >> 4, tx = tid & 15;
-    const float* S = b.states + ((size_t)ch * p.heads + h) * p.dim * p.vdim;
-    const float* A = b.weights + ((size_t)ch * p.heads + h) * C * C;
+    const int HD = b.heads * b.dim, t0 = ch * C, n = min(C, T - t0), ty = tid >> 4, tx = tid & 15;
+    const float* S = b.states + ((size_t)ch * b.heads + h) * b.dim * b.vdim;
+    const float* A = b.weights + ((size_t)ch * b.heads + h) * C * C;
     float acc[8][4] = {};
-    for (int k0 = 0; k0 < p.dim; k0 += kTileK) {
+    for (int k0 = 0; k0 < b.dim; k0 += kTileK) {
         __syncthreads();
-        tile_cols(sa, b.qd + (size_t)t0 * HD + h * p.dim, HD, n, k0, p.dim, vec);
-        tile_rows(sb, S + (size_t)k0 * p.vdim, p.vdim, p.dim - k0, v0, p.vdim, vec);
+        tile_cols(sa, b.qd + (size_t)t0 * HD + h * b.dim, HD, n, k0, b.dim, vec);
+        tile_rows(sb, S + (size_t)k0 * b.vdim, b.vdim, b.dim - k0, v0, b.vdim, vec);
         __syncthreads();
         tile_fma(sa, sb, ty, tx, acc);
     }
     for (int s0 = 0; s0 < n; s0 += kTileK) {
         __syncthreads();
         tile_cols(sa, A, C, n, s0, n, true);
-        tile_rows(sb, p.proj + (size_t)(t0 + s0) * p.ldp + 2 * HD + h * p.vdim, p.ldp, n - s0, v0, p.vdim, vec);
+        tile_rows(sb, b.v + (size_t)(t0 + s0) * b.ldv + h * b.vdim, b.ldv, n - s0, v0, b.vdim, vec);
         __syncthreads();
         tile_fma(sa, sb, ty, tx, acc);
     }
@@ -370,13 +370,13 @@ __global__ void __launch_bounds__(kTileThreads) lb_gla_out_kernel(const LbGla p,
     for (int i = 0; i < 8; ++i) {
         const int t = ty * 8 + i, v = v0 + tx * 4;
         if (t >= n) continue;
-        float* out = p.o + (size_t)(t0 + t) * p.ldo + h * p.vdim + v;
-        if (vec && v + 4 <= p.vdim)
+        float* out = b.o + (size_t)(t0 + t) * b.ldo + h * b.vdim + v;
+        if (vec && v + 4 <= b.vdim)
             *reinterpret_cast<float4*>(out) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
         else
 #pragma unroll
             for (int j = 0; j < 4; ++j)
-                if (v + j < p.vdim) out[j] = acc[i][j];
+                if (v + j < b.vdim) out[j] = acc[i][j];
     }
 }
 
@@ -400,18 +400,40 @@ int lb_gla_step(loom_b200_ctx* ctx, const LbGla& p, const int* pos, int lane0, i
     return 0;
 }
 
-int lb_gla_block(loom_b200_ctx* ctx, const LbGla& p, const LbGlaBlock& bin, int T, int pos0) {
-    LbGlaBlock b = bin;
+int lb_gla_block(loom_b200_ctx* ctx, const LbGla& p, const LbChunks& scratch, int T, int pos0) {
+    LbChunks b = scratch;
     b.C = lb_gla_chunk(p.dim, p.rank);
+    b.heads = p.heads;
+    b.dim = p.dim;
+    b.vdim = p.vdim;
+    b.v = p.proj + 2 * p.heads * p.dim;
+    b.ldv = p.ldp;
+    b.state = p.state;
+    b.o = p.o;
+    b.ldo = p.ldo;
     LB_REQUIRE(ctx, b.C > 0, "gla: %d key channels, decay rank %d", p.dim, p.rank);
-    const int chunks = lb_ceil_div(T, b.C), fresh = pos0 == 0 ? 1 : 0;
     LB_BIG_SMEM(ctx, lb_gla_prep_kernel, 200 * 1024);
-    LB_LAUNCH(ctx, lb_gla_prep_kernel, dim3(chunks, p.heads), dim3(kPrepThreads), prep_smem(b.C, p.dim, p.rank), p, b, T);
-    const bool vec = p.dim % 4 == 0 && p.vdim % 4 == 0 && p.ldp % 4 == 0 && p.ldo % 4 == 0;
-    const int dt = lb_ceil_div(p.dim, kTile), vt = lb_ceil_div(p.vdim, kTile);
-    LB_LAUNCH(ctx, lb_gla_state_kernel, dim3(dt * vt, p.heads, chunks), dim3(kTileThreads), 0, p, b, T, dt, vec);
-    const size_t all = (size_t)p.heads * p.dim * p.vdim;
-    LB_LAUNCH(ctx, lb_gla_scan_kernel, dim3((unsigned)((all + 255) / 256)), dim3(256), 0, p, b, chunks, fresh);
-    LB_LAUNCH(ctx, lb_gla_out_kernel, dim3(vt, p.heads, chunks), dim3(kTileThreads), 0, p, b, T, vec);
+    LB_LAUNCH(ctx, lb_gla_prep_kernel, dim3(lb_ceil_div(T, b.C), p.heads), dim3(kPrepThreads), prep_smem(b.C, p.dim, p.rank), p, b, T);
+    if (int rc = lb_chunk_states(ctx, b, T)) return rc;
+    if (int rc = lb_chunk_scan(ctx, b, T, pos0 == 0)) return rc;
+    return lb_chunk_out(ctx, b, T);
+}
+
+int lb_chunk_states(loom_b200_ctx* ctx, const LbChunks& c, int T) {
+    const bool vec = c.dim % 4 == 0 && c.vdim % 4 == 0 && lb_vec_rows(c.v, c.ldv);
+    const int dt = lb_ceil_div(c.dim, kTile), vt = lb_ceil_div(c.vdim, kTile);
+    LB_LAUNCH(ctx, lb_chunk_state_kernel, dim3(dt * vt, c.heads, lb_ceil_div(T, c.C)), dim3(kTileThreads), 0, c, T, dt, vec);
+    return 0;
+}
+
+int lb_chunk_scan(loom_b200_ctx* ctx, const LbChunks& c, int T, bool fresh) {
+    const size_t all = (size_t)c.heads * c.dim * c.vdim;
+    LB_LAUNCH(ctx, lb_chunk_scan_kernel, dim3((unsigned)((all + 255) / 256)), dim3(256), 0, c, lb_ceil_div(T, c.C), fresh ? 1 : 0);
+    return 0;
+}
+
+int lb_chunk_out(loom_b200_ctx* ctx, const LbChunks& c, int T) {
+    const bool vec = c.dim % 4 == 0 && c.vdim % 4 == 0 && lb_vec_rows(c.v, c.ldv) && lb_vec_rows(c.o, c.ldo);
+    LB_LAUNCH(ctx, lb_chunk_out_kernel, dim3(lb_ceil_div(c.vdim, kTile), c.heads, lb_ceil_div(T, c.C)), dim3(kTileThreads), 0, c, T, vec);
     return 0;
 }

@@ -31,7 +31,7 @@ struct Cfg {
 template <int NB, int EPI>
 __global__ void __launch_bounds__(kThreads, 1) lb_gemm_bf16_kernel(const LbDenseGemm p, int row_tiles) {
     using C = Cfg<NB>;
-    constexpr bool kDual = EPI == LB_DEPI_GLU;
+    constexpr bool kDual = EPI == LB_DEPI_GLU || EPI == LB_DEPI_SILU;
     extern __shared__ __align__(1024) uint8_t smem[];
     __shared__ __align__(8) uint64_t load_bar[C::kStages], empty_bar[C::kStages], acc_full[2], acc_empty[2];
     __shared__ uint32_t tmem_base_s;
@@ -165,14 +165,14 @@ __global__ void __launch_bounds__(kThreads, 1) lb_gemm_bf16_kernel(const LbDense
                             o[1] = make_float4(v8[4], v8[5], v8[6], v8[7]);
                         } else {
                             float4 x = o[0], y = o[1];
-                            x.x = fmaf(p.mult, v8[0], x.x);
-                            x.y = fmaf(p.mult, v8[1], x.y);
-                            x.z = fmaf(p.mult, v8[2], x.z);
-                            x.w = fmaf(p.mult, v8[3], x.w);
-                            y.x = fmaf(p.mult, v8[4], y.x);
-                            y.y = fmaf(p.mult, v8[5], y.y);
-                            y.z = fmaf(p.mult, v8[6], y.z);
-                            y.w = fmaf(p.mult, v8[7], y.w);
+                            x.x = fmaf(p.mult, v8[0], p.res_mult * x.x);
+                            x.y = fmaf(p.mult, v8[1], p.res_mult * x.y);
+                            x.z = fmaf(p.mult, v8[2], p.res_mult * x.z);
+                            x.w = fmaf(p.mult, v8[3], p.res_mult * x.w);
+                            y.x = fmaf(p.mult, v8[4], p.res_mult * y.x);
+                            y.y = fmaf(p.mult, v8[5], p.res_mult * y.y);
+                            y.z = fmaf(p.mult, v8[6], p.res_mult * y.z);
+                            y.w = fmaf(p.mult, v8[7], p.res_mult * y.w);
                             o[0] = x;
                             o[1] = y;
                         }
@@ -184,6 +184,7 @@ __global__ void __launch_bounds__(kThreads, 1) lb_gemm_bf16_kernel(const LbDense
                             f[j] = v8[j];
                             if (EPI == LB_DEPI_GELU) f[j] = lb_gelu_erff(v8[j]);
                             if (EPI == LB_DEPI_GLU) f[j] = lb_clamped_glu(v8[j], u8[j], p.limit);
+                            if (EPI == LB_DEPI_SILU) f[j] = lb_siluf(v8[j]) * u8[j];
                         }
                         if (EPI == LB_DEPI_HEADS)
                             *reinterpret_cast<uint4*>(p.img + lb_heads_chunk(tok, r, p.heads, p.head_dim, p.head_chunks)) = lb_pack_chunk<__nv_bfloat16>(f);
@@ -208,7 +209,7 @@ __global__ void __launch_bounds__(kThreads, 1) lb_gemm_bf16_kernel(const LbDense
 template <int NB, int EPI>
 int launch(loom_b200_ctx* ctx, const LbDenseGemm& p) {
     using C = Cfg<NB>;
-    const int per = EPI == LB_DEPI_GLU ? 1 : NB;
+    const int per = EPI == LB_DEPI_GLU || EPI == LB_DEPI_SILU ? 1 : NB;
     const int row_tiles = lb_ceil_div(lb_ceil_div(p.rows, kImgRows), per);
     const int blocks = p.nblocks ? p.max_blocks : lb_ceil_div(p.tokens, kImgRows);
     const int ntiles = row_tiles * blocks;
@@ -236,6 +237,7 @@ int lb_gemm_bf16_run(loom_b200_ctx* ctx, int epi, const LbDenseGemm& p) {
         case LB_DEPI_IMG: return launch_plain<LB_DEPI_IMG>(ctx, p);
         case LB_DEPI_HEADS: return launch_plain<LB_DEPI_HEADS>(ctx, p);
         case LB_DEPI_GLU: return launch<2, LB_DEPI_GLU>(ctx, p);
+        case LB_DEPI_SILU: return launch<2, LB_DEPI_SILU>(ctx, p);
     }
     return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "gemm_bf16: epilogue %d is not built", epi);
 }

@@ -1,7 +1,6 @@
 // latent_attention.cu -- attention over cached latents in bf16: a split kernel for single tokens that reads every latent once for
-// up to sixteen heads, and a tcgen05 kernel for token blocks over per-head keys and values expanded from the latents.
+// up to sixteen heads; token blocks expand per-head keys and values from the latents for the tensor-core kernel (attention_block.cu).
 #include "mixers.cuh"
-#include "umma.cuh"
 
 #include <cmath>
 
@@ -14,12 +13,6 @@ __device__ __forceinline__ void mma_bf16(float* d, uint32_t a0, uint32_t a1, uin
 }
 __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t* r, const void* p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(lb_smem_u32(p)));
-}
-// 2^x by the hardware's approximation (two units in the last place), results below 2^-126 as zero
-__device__ __forceinline__ float fast_exp2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
 }
 // value = hi + lo, both bf16: the pair carries sixteen bits of the float
 __device__ __forceinline__ void split_bf16(const float* f, uint4& hi, uint4& lo) {
@@ -291,187 +284,7 @@ __global__ void __launch_bounds__(256) lb_latent_value_kernel(const LbLatent p, 
     }
 }
 
-// ---- token blocks -------------------------------------------------------------------------------------------------
-//
-// CTA = (128 query tokens, head), two CTAs per SM: a query row per thread, one thread also issues the loads and the MMAs (a
-// fifth warp would cost every thread a fifth of its registers).  S = Q K^T of 64 keys and O_j = P V of the same keys are both
-// fresh TMEM accumulators; the running maximum, the sum and the output row live in the thread's registers, so nothing is ever
-// rescaled in tensor memory.  While the threads take in O_j, the tensor core is on S_(j+1) -- and on the other CTA's tiles.
-constexpr int kAtKeys = 64;
-constexpr int kAtThreads = 128;
-
-struct AttnParams {
-    const uint8_t* q;   // [token block of 128][head][row/8][chunk][row%8][16 B]
-    const uint8_t* k;   // the same of positions
-    const uint8_t* vt;  // image of [heads*vdim rows] x positions
-    int heads, dchunks, vdim, vslices;  // dchunks: 16-byte chunks of a query row (even); vslices: K slices of vt
-    int T, pos0;
-    float scale_log2;   // magnitude of the score factor times log2(e) (its sign is in the queries)
-    uint8_t* out;       // token image of heads*vdim columns
-    int out_slices;
-    int* status;
-};
-
-template <int VC>  // value columns, a multiple of sixteen
-__global__ void __launch_bounds__(kAtThreads, 2) lb_latent_block_kernel(const AttnParams p) {
-    extern __shared__ __align__(1024) uint8_t sm[];
-    __shared__ __align__(8) uint64_t bar_q, bar_k[2], bar_v[2], bar_s, bar_p, bar_o;
-    __shared__ uint32_t tmem_base_s;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int nqb = lb_ceil_div(p.T, 128), qb = nqb - 1 - (int)blockIdx.y, h = blockIdx.x;  // the longest rows of every head first
-    const uint32_t qbytes = (uint32_t)p.dchunks * 2048, kbytes = (uint32_t)p.dchunks * 1024, vbytes = (uint32_t)p.vdim * 128;
-    constexpr uint32_t kVStage = VC * 128;
-    uint8_t *sq = sm, *sk = sq + qbytes, *sv = sk + 2 * kbytes, *sp = sv + 2 * kVStage;
-    constexpr uint32_t kTmem = VC + kAtKeys <= 64 ? 64 : VC + kAtKeys <= 128 ? 128 : 256;
-    constexpr uint32_t id_s = lb_idesc_bf16(128, kAtKeys, false), id_o = lb_idesc_bf16(128, VC, false);
-    const int last = min(p.T, qb * 128 + 128) - 1;  // last query row of the block
-    const int ntiles = (p.pos0 + last) / kAtKeys + 1;
-    if (tid == 0) {
-        uint64_t* one[] = {&bar_q, &bar_k[0], &bar_k[1], &bar_v[0], &bar_v[1], &bar_s, &bar_o};
-        for (auto* b : one) lb_mbar_init(b, 1);
-        lb_mbar_init(&bar_p, kAtThreads);
-        lb_fence_mbar_init();
-    }
-    if (warp == 0) lb_tmem_alloc(&tmem_base_s, kTmem);
-    lb_tc_fence_before();
-    __syncthreads();
-    lb_tc_fence_after();
-    const uint32_t tmem = tmem_base_s;
-    lb_pdl_launch_dependents();
-    lb_pdl_wait();
-
-    const uint32_t a_q = lb_smem_u32(sq), a_k = lb_smem_u32(sk), a_v = lb_smem_u32(sv), a_p = lb_smem_u32(sp), sbo_d = (uint32_t)p.dchunks * 128;
-    auto load = [&](int j) {
-        const int s = j & 1;
-        lb_mbar_expect_tx(&bar_k[s], kbytes);
-        lb_bulk_g2s(sk + s * kbytes, p.k + ((size_t)(j >> 1) * p.heads + h) * p.dchunks * 2048 + (size_t)(j & 1) * kbytes, kbytes, &bar_k[s]);
-        lb_mbar_expect_tx(&bar_v[s], vbytes);
-        for (int r = h * p.vdim, end = r + p.vdim; r < end;) {  // the head's rows, block of 128 rows by block
-            const int n = min(end, (r & ~127) + 128) - r;
-            lb_bulk_g2s(sv + s * kVStage + (uint32_t)(r - h * p.vdim) * 128, p.vt + ((size_t)(r >> 7) * p.vslices + j) * kImgBlock + (size_t)((r & 127) >> 3) * 1024,
-                        (uint32_t)n * 128, &bar_v[s]);
-            r += n;
-        }
-    };
-    auto scores = [&](int j) {
-        for (int k = 0; k < p.dchunks / 2; ++k)
-            lb_mma_f16(tmem, lb_smem_desc(a_q + k * 256, 128, sbo_d), lb_smem_desc(a_k + (j & 1) * kbytes + k * 256, 128, sbo_d), id_s, k > 0 ? 1u : 0u);
-        lb_mma_commit(&bar_s);
-    };
-    bool failed = false;
-    if (tid == 0) {
-        lb_mbar_expect_tx(&bar_q, qbytes);
-        lb_bulk_g2s(sq, p.q + ((size_t)qb * p.heads + h) * qbytes, qbytes, &bar_q);
-        load(0);
-        if (ntiles > 1) load(1);
-        failed = !lb_mbar_wait_bounded(&bar_q, 0, kTcWaitLimit) || !lb_mbar_wait_bounded(&bar_k[0], 0, kTcWaitLimit);
-        if (!failed) scores(0);
-    }
-    __syncwarp();
-
-    const int row = warp * 32 + lane, tok = qb * 128 + row, qpos = p.pos0 + tok;
-    const uint32_t lanes = (uint32_t)(warp * 32) << 16;
-    float o[VC];
-#pragma unroll
-    for (int c = 0; c < VC; ++c) o[c] = 0.f;
-    float mx = -3e38f, sum = 0.f;  // (finite: the factor may be zero)
-    uint8_t* prow = sp + (size_t)(row >> 3) * 1024 + (row & 7) * 16;
-    for (int j = 0; j < ntiles; ++j) {
-        if (!lb_mbar_wait_bounded(&bar_s, (uint32_t)(j & 1), kTcWaitLimit)) failed = true;
-        if (__any_sync(0xffffffffu, failed)) {  // a warp leaves together; the others' waits run out
-            failed = true;
-            break;
-        }
-        lb_tc_fence_after();
-        float f;
-        {
-            float s[kAtKeys];
-#pragma unroll
-            for (int c = 0; c < kAtKeys; c += 16) lb_tmem_ld16(tmem + lanes + c, s + c);
-            lb_tmem_wait_ld();
-            const int vis = qpos - j * kAtKeys;  // keys 0..vis of the tile are visible
-            if (vis < kAtKeys - 1) {
-#pragma unroll
-                for (int c = 0; c < kAtKeys; ++c) s[c] = c <= vis ? s[c] : -INFINITY;
-            }
-            float m4[4] = {mx, -INFINITY, -INFINITY, -INFINITY};  // (the factor is not negative, so it may follow the maximum)
-#pragma unroll
-            for (int c = 0; c < kAtKeys; ++c) m4[c & 3] = fmaxf(m4[c & 3], s[c]);
-            const float m = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])), off = m * p.scale_log2;
-            f = fast_exp2(mx * p.scale_log2 - off);
-            mx = m;
-            float add = 0.f;
-#pragma unroll
-            for (int c = 0; c < kAtKeys; c += 8) {
-#pragma unroll
-                for (int e = 0; e < 8; ++e) {
-                    s[c + e] = fast_exp2(fmaf(s[c + e], p.scale_log2, -off));
-                    add += s[c + e];
-                }
-                *reinterpret_cast<uint4*>(prow + (c >> 3) * 128) = lb_pack_chunk<__nv_bfloat16>(s + c);
-            }
-            sum = fmaf(sum, f, add);
-        }
-        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-        lb_tc_fence_before();
-        lb_mbar_arrive(&bar_p);
-        if (tid == 0) {  // every row's weights are in shared memory, S_j and O_(j-1) have left tensor memory
-            if (!lb_mbar_wait_bounded(&bar_p, (uint32_t)(j & 1), kTcWaitLimit) || !lb_mbar_wait_bounded(&bar_v[j & 1], (uint32_t)((j >> 1) & 1), kTcWaitLimit)) {
-                failed = true;
-            } else {
-                lb_tc_fence_after();
-                for (int k = 0; k < kAtKeys / 16; ++k)
-                    lb_mma_f16(tmem + kAtKeys, lb_smem_desc(a_p + k * 256, 128, 1024), lb_smem_desc(a_v + (j & 1) * kVStage + k * 256, 128, 1024), id_o, k > 0 ? 1u : 0u);
-                lb_mma_commit(&bar_o);
-                if (j + 1 < ntiles) {
-                    if (lb_mbar_wait_bounded(&bar_k[(j + 1) & 1], (uint32_t)(((j + 1) >> 1) & 1), kTcWaitLimit))
-                        scores(j + 1);
-                    else
-                        failed = true;
-                }
-            }
-        }
-        __syncwarp();
-        if (!lb_mbar_wait_bounded(&bar_o, (uint32_t)(j & 1), kTcWaitLimit)) failed = true;
-        if (__any_sync(0xffffffffu, failed)) {
-            failed = true;
-            break;
-        }
-        if (tid == 0 && j + 2 < ntiles) load(j + 2);  // S_j and O_j are done: their stage is free
-        __syncwarp();
-        lb_tc_fence_after();
-        constexpr int VS = VC % 64 == 0 ? 64 : VC % 32 == 0 ? 32 : 16;  // columns per wait
-#pragma unroll
-        for (int c = 0; c < VC; c += VS) {
-            float v[VS];
-#pragma unroll
-            for (int e = 0; e < VS; e += 16) lb_tmem_ld16(tmem + lanes + kAtKeys + c + e, v + e);
-            lb_tmem_wait_ld();
-#pragma unroll
-            for (int e = 0; e < VS; ++e) o[c + e] = fmaf(o[c + e], f, v[e]);
-        }
-    }
-    if (failed) {
-        if (lane == 0) atomicExch(p.status, 3);
-    } else if (tok < p.T) {
-        const float r = __fdiv_rn(1.f, sum);
-#pragma unroll
-        for (int c = 0; c < VC; c += 8) {
-            if (c < p.vdim) {
-                float v[8];
-#pragma unroll
-                for (int e = 0; e < 8; ++e) v[e] = o[c + e] * r;
-                lb_img_store8<__nv_bfloat16>(p.out, tok, h * p.vdim + c, p.out_slices, v);
-            }
-        }
-    }
-    lb_tc_fence_before();
-    __syncthreads();
-    if (warp == 0) {
-        lb_tc_fence_after();
-        lb_tmem_dealloc(tmem, kTmem);
-    }
-}
+// ---- token blocks: queries, expanded keys and transposed values for attention_block.cu -----------------------------------
 
 // float query rows -> per-head bf16 blocks
 __global__ void __launch_bounds__(256) lb_heads_image_kernel(const float* __restrict__ x, int ldx, int heads, int dim, int dchunks, float sign, uint8_t* __restrict__ img) {
@@ -486,14 +299,6 @@ __global__ void __launch_bounds__(256) lb_heads_image_kernel(const float* __rest
         *reinterpret_cast<uint4*>(img + ((size_t)(t >> 7) * heads + h) * dchunks * 2048 + (size_t)((t & 127) >> 3) * dchunks * 128 + (size_t)c * 128 + (t & 7) * 16) =
             lb_pack_chunk<__nv_bfloat16>(f);
     }
-}
-
-template <int VC>
-int launch_block(loom_b200_ctx* ctx, const AttnParams& p) {
-    const size_t smem = (size_t)p.dchunks * (2048 + 2 * 1024) + 2 * VC * 128 + 16384;
-    LB_BIG_SMEM(ctx, lb_latent_block_kernel<VC>, 220 * 1024);
-    LB_LAUNCH(ctx, lb_latent_block_kernel<VC>, dim3(p.heads, lb_ceil_div(p.T, 128)), dim3(kAtThreads), smem, p);
-    return 0;
 }
 
 template <int CPW>
@@ -566,23 +371,18 @@ int lb_latent_block(loom_b200_ctx* ctx, const LbLatent& p, int T, uint8_t* q_img
     g.img = vt_img;
     g.img_slices = vt_slices;
     if (int rc = lb_dense_gemm(ctx, LOOM_B200_DTYPE_BF16, LB_DEPI_IMG, g)) return rc;
-    AttnParams a;
+    LbAttnBlock a;
     a.q = q_img;
     a.k = k_img;
     a.vt = vt_img;
-    a.heads = p.heads;
+    a.heads = a.kv_heads = p.heads;
     a.dchunks = dch;
-    a.vdim = p.vdim;
+    a.vdim = a.vrows = p.vdim;
     a.vslices = vt_slices;
     a.T = T;
     a.pos0 = p.pos0;
     a.scale_log2 = fabsf(p.scale) * 1.4426950408889634f;
     a.out = out;
     a.out_slices = out_slices;
-    a.status = ctx->status_dev;
-    if (p.vdim <= 16) return launch_block<16>(ctx, a);
-    if (p.vdim <= 32) return launch_block<32>(ctx, a);
-    if (p.vdim <= 64) return launch_block<64>(ctx, a);
-    if (p.vdim <= 96) return launch_block<96>(ctx, a);
-    return launch_block<128>(ctx, a);
+    return lb_attn_block(ctx, a);
 }

@@ -25,6 +25,23 @@ __global__ void __launch_bounds__(256) lb_embed_norm_kernel(const WT* __restrict
     for (int k = threadIdx.x; k < width; k += blockDim.x) out[k] = ok ? (float)row[k] * r : 0.f;
 }
 
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_embed_image_kernel(const uint8_t* __restrict__ img, int slices, int vocab, int width, const int* tok, float* __restrict__ x, int ldx) {
+    constexpr int C = LbElem<WT>::kChunk;
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = tok[blockIdx.x];
+    const bool ok = t >= 0 && t < vocab;
+    float* out = x + (size_t)blockIdx.x * ldx;
+    for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
+        float f[C];
+        lb_unpack_chunk<WT>(*reinterpret_cast<const uint4*>(img + lb_img_chunk(ok ? t : 0, c, slices)), f);
+#pragma unroll
+        for (int e = 0; e < C; ++e)
+            if (c * C + e < width) out[c * C + e] = ok ? f[e] : 0.f;
+    }
+}
+
 constexpr int kNormTokens = 8;  // tokens of a CTA
 constexpr int kMaxTaps = 16;
 
@@ -44,7 +61,7 @@ __global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p,
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * kNormTokens, t1 = min(p.T, t0 + kNormTokens);
     const int back = p.conv_w ? p.taps - 1 : 0;
-    const float gain = *p.gain;
+    const float gain = p.gain ? *p.gain : 1.f;
     for (int i = warp; i < t1 - t0 + back; i += 8) {
         const int t = t0 - back + i;
         if (t < 0) continue;
@@ -61,6 +78,17 @@ __global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p,
         lb_load_cols<C>(p.x + (size_t)src * p.ldx, k0, p.width, vec, f);
 #pragma unroll
         for (int e = 0; e < C; ++e) f[e] *= s_r[tt + back];
+        if (p.gain_w) {
+            float w[C];
+            lb_load_cols<C>(p.gain_w, k0, p.width, vec, w);
+#pragma unroll
+            for (int e = 0; e < C; ++e) f[e] *= w[e];
+        }
+        if (p.rows) {
+#pragma unroll
+            for (int e = 0; e < C; ++e)
+                if (k0 + e < p.width) p.rows[(size_t)t * p.ldx + k0 + e] = f[e];
+        }
         if (p.conv_w && k0 < p.width) {
             float a[C], w[C], h[C];
 #pragma unroll
@@ -82,7 +110,7 @@ __global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p,
 #pragma unroll
             for (int e = 0; e < C; ++e) f[e] += a[e];
         }
-        *reinterpret_cast<uint4*>(p.img + lb_img_chunk(t, c, p.slices)) = lb_pack_chunk<WT>(f);
+        if (p.img) *reinterpret_cast<uint4*>(p.img + lb_img_chunk(t, c, p.slices)) = lb_pack_chunk<WT>(f);
     }
 }
 
@@ -116,7 +144,8 @@ __global__ void __launch_bounds__(256) lb_rows_image_kernel(const float* __restr
 
 template <typename WT>
 __global__ void __launch_bounds__(256) lb_gated_heads_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, bool vec, int heads, int vdim,
-                                                             const float* __restrict__ w, float eps, int slices, uint8_t* __restrict__ img) {
+                                                             const float* __restrict__ w, bool gate_sigmoid, const float* __restrict__ scale, float eps, int slices,
+                                                             uint8_t* __restrict__ img) {
     extern __shared__ float s_r[];
     constexpr int C = LbElem<WT>::kChunk;
     lb_pdl_launch_dependents();
@@ -124,18 +153,25 @@ __global__ void __launch_bounds__(256) lb_gated_heads_kernel(const float* __rest
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, HV = heads * vdim;
     const float* row = o + (size_t)t * ldo;
     for (int h = warp; h < heads; h += 8) {
-        const float r = row_rstd(row + (size_t)h * vdim, vdim, eps, lane);
-        if (lane == 0) s_r[h] = r;
+        float ss = 0.f;
+        const float by = scale ? scale[(size_t)t * heads + h] : 1.f;
+        for (int k = lane; k < vdim; k += 32) {
+            const float v = row[(size_t)h * vdim + k] * by;
+            ss = fmaf(v, v, ss);
+        }
+        ss = lb_warp_sumf(ss);
+        if (lane == 0) s_r[h] = by * __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)vdim), eps)));
     }
     __syncthreads();
     for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
-        float f[C], g[C];
+        float f[C], g[C], hw[C];
         lb_load_cols<C>(row, c * C, HV, vec, f);
         lb_load_cols<C>(gate + (size_t)t * ldg, c * C, HV, vec, g);
+        lb_load_cols<C>(w, c * C, HV, vec, hw);
 #pragma unroll
         for (int e = 0; e < C; ++e) {
             const int k = c * C + e, h = k / vdim;
-            f[e] = k < HV ? f[e] * s_r[h] * w[k - h * vdim] * lb_siluf(g[e]) : 0.f;
+            f[e] = k < HV ? f[e] * s_r[h] * hw[e] * (gate_sigmoid ? lb_sigmoidf(g[e]) : lb_siluf(g[e])) : 0.f;
         }
         *reinterpret_cast<uint4*>(img + lb_img_chunk(t, c, slices)) = lb_pack_chunk<WT>(f);
     }
@@ -436,10 +472,15 @@ int lb_embed_norm(loom_b200_ctx* ctx, int dtype, const void* table, int vocab, i
     return 0;
 }
 
+int lb_embed_image(loom_b200_ctx* ctx, int dtype, const uint8_t* img, int slices, int vocab, int width, const int* tok, int n, float* x, int ldx) {
+    LB_TYPED(dtype, lb_embed_image_kernel<float>, lb_embed_image_kernel<__nv_bfloat16>, dim3(n), dim3(256), 0, img, slices, vocab, width, tok, x, ldx);
+    return 0;
+}
+
 int lb_norm_block(loom_b200_ctx* ctx, int dtype, const LbNormBlock& p) {
     LB_REQUIRE(ctx, p.taps >= 1 && p.taps <= kMaxTaps, "norm_block: %d taps (1..%d)", p.taps, kMaxTaps);
     LB_TYPED(dtype, lb_norm_block_kernel<float>, lb_norm_block_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.T, kNormTokens)), dim3(256), 0, p,
-             lb_vec_rows(p.x, p.ldx) && (!p.conv_w || (lb_vec_rows(p.conv_w, p.ring_ld) && lb_vec_rows(p.ring, p.ring_ld))));
+             lb_vec_rows(p.x, p.ldx) && (!p.gain_w || lb_vec_rows(p.gain_w, 4)) && (!p.conv_w || (lb_vec_rows(p.conv_w, p.ring_ld) && lb_vec_rows(p.ring, p.ring_ld))));
     return 0;
 }
 
@@ -455,9 +496,9 @@ int lb_rows_image(loom_b200_ctx* ctx, int dtype, const float* x, int ldx, int T,
 }
 
 int lb_gated_heads_image(loom_b200_ctx* ctx, int dtype, const float* o, int ldo, const float* gate, int ldg, int T, int heads, int vdim, const float* head_w,
-                         float eps, int slices, uint8_t* img) {
+                         bool gate_sigmoid, const float* scale, float eps, int slices, uint8_t* img) {
     LB_TYPED(dtype, lb_gated_heads_kernel<float>, lb_gated_heads_kernel<__nv_bfloat16>, dim3(T), dim3(256), (size_t)heads * sizeof(float), o, ldo, gate, ldg,
-             lb_vec_rows(o, ldo) && lb_vec_rows(gate, ldg), heads, vdim, head_w, eps, slices, img);
+             lb_vec_rows(o, ldo) && lb_vec_rows(gate, ldg) && lb_vec_rows(head_w, 4), heads, vdim, head_w, gate_sigmoid, scale, eps, slices, img);
     return 0;
 }
 

@@ -1,0 +1,401 @@
+// softmax_attention.cu -- softmax attention over cached keys and values of grouped heads, with any of: unit-variance queries and
+// keys, a learned bias by distance, chunks, a sink, a gate per head.  Storing a block of tokens, the step of one token per sequence
+// (any precision), and the block's operands for the tensor-core kernel (attention_block.cu).
+#include "mixers.cuh"
+
+#include <cmath>
+
+namespace {
+
+constexpr int kTile = 64;  // positions of a tile: half of a block of keys; one K slice (two in 32-bit) of the transposed values
+constexpr int kStepThreads = 256;
+
+__host__ __device__ inline int vrows_of(int vdim) { return lb_round_up(vdim, 8); }
+
+// 1 / root mean square of a head's row (a warp)
+__device__ __forceinline__ float head_rstd(const float* row, int n, float eps, int lane) {
+    float ss = 0.f;
+    for (int d = lane; d < n; d += 32) ss = fmaf(row[d], row[d], ss);
+    ss = lb_warp_sumf(ss);
+    return __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)n), eps)));
+}
+
+// byte offset of 16-byte chunk c of a position's row of kv head g
+__device__ __forceinline__ size_t key_chunk(int row, int g, int kv_heads, int kchunks, int c) {
+    return ((size_t)(row >> 7) * kv_heads + g) * kchunks * 2048 + (size_t)((row & 127) >> 3) * kchunks * 128 + (size_t)c * 128 + (size_t)(row & 7) * 16;
+}
+template <typename WT>
+__device__ __forceinline__ size_t value_at(int g, int v, int vrows, int row, int slices) {  // one element
+    constexpr int C = LbElem<WT>::kChunk;
+    return lb_img_chunk(g * vrows + v, row / C, slices) + (size_t)(row % C) * sizeof(WT);
+}
+
+// A CTA takes the tokens of eight aligned positions: a warp per token for queries and keys, then a thread per value row.
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_attention_store_kernel(const LbAttention p, int T, int kchunks, int qchunks, uint8_t* __restrict__ q_img, bool vec) {
+    constexpr int C = LbElem<WT>::kChunk;
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, first = (p.pos0 & ~7) + (int)blockIdx.x * 8;
+    const int QD = p.heads * p.dim, KD = p.kv_heads * p.dim, vrows = vrows_of(p.vdim);
+    uint8_t *kc = p.k + (size_t)p.lane0 * p.k_lane, *vc = p.vt + (size_t)p.lane0 * p.vt_lane;
+    const int pos = first + warp, t = pos - p.pos0;
+    if (t >= 0 && t < T) {
+        const float* row = p.proj + (size_t)t * p.ldp;
+        const int r = pos % p.ring;
+        for (int i = q_img ? 0 : p.heads; i < p.heads + p.kv_heads; ++i) {
+            const bool key = i >= p.heads;
+            const int h = key ? i - p.heads : i, chunks = key ? kchunks : qchunks;
+            const float* x = row + (key ? QD + h * p.dim : h * p.dim);
+            const float by = p.qk_norm ? head_rstd(x, p.dim, p.eps, lane) : 1.f;
+            if (key) {
+                for (int c = lane; c < chunks; c += 32) {
+                    float f[C];
+                    lb_load_cols<C>(x, c * C, p.dim, vec, f);
+#pragma unroll
+                    for (int e = 0; e < C; ++e) f[e] *= by;
+                    *reinterpret_cast<uint4*>(kc + key_chunk(r, h, p.kv_heads, kchunks, c)) = lb_pack_chunk<WT>(f);
+                }
+            } else {
+                for (int c = lane; c < chunks; c += 32) {
+                    float f[8];
+                    lb_load_cols<8>(x, c * 8, p.dim, vec, f);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) f[e] *= by;
+                    *reinterpret_cast<uint4*>(q_img + key_chunk(t, h, p.heads, chunks, c)) = lb_pack_chunk<__nv_bfloat16>(f);
+                }
+            }
+        }
+    }
+    const int t0 = first - p.pos0, r0 = first % p.ring;
+    for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += 256) {
+        const int g = i / p.vdim, v = i - g * p.vdim;
+        float f[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = t0 + e >= 0 && t0 + e < T ? p.proj[(size_t)(t0 + e) * p.ldp + QD + KD + i] : 0.f;
+        if (t0 >= 0 && t0 + 8 <= T) {
+#pragma unroll
+            for (int e = 0; e < 8; e += C) *reinterpret_cast<uint4*>(vc + lb_img_chunk(g * vrows + v, (r0 + e) / C, p.slices)) = lb_pack_chunk<WT>(f + e);
+        } else {  // the eight positions hold tokens of other calls too
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+                if (t0 + e >= 0 && t0 + e < T) *reinterpret_cast<WT*>(vc + value_at<WT>(g, v, vrows, r0 + e, p.slices)) = (WT)f[e];
+        }
+    }
+}
+
+// One token per sequence: CTA = (split of the visible positions, HB query heads of a kv head, token).  Tiles of 64 positions: four
+// threads per key for the scores, a warp per head for the running softmax, then four threads per value row and K slice for the
+// weighted sum.  The split with the newest position takes its key and value from the projections and puts them into the cache.
+// The last CTA of a (token, heads) to arrive merges the splits; nothing waits.
+template <typename WT, int HB>
+__global__ void __launch_bounds__(kStepThreads) lb_attention_step_kernel(const LbAttention p, int kchunks, int splits, float* __restrict__ part, unsigned* __restrict__ count,
+                                                                         float* __restrict__ out, int ldo) {
+    extern __shared__ __align__(16) uint8_t sm[];
+    constexpr int C = LbElem<WT>::kChunk, S = LbElem<WT>::kSlice, KS = kTile / S;  // KS: K slices of a tile
+    __shared__ __align__(16) float s_w[HB][kTile];
+    __shared__ float s_max[HB], s_sum[HB], s_fac[HB], s_new[HB], s_rq[HB], s_rk;
+    __shared__ bool s_last;
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int per = p.heads / p.kv_heads, nb = lb_ceil_div(per, HB), split = blockIdx.x, g = blockIdx.y / nb, hb = blockIdx.y % nb, m = blockIdx.z;
+    const int h0 = g * per + hb * HB, nh = min(HB, per - hb * HB);
+    const int pos = p.pos ? p.pos[m] : p.pos0 + m, seq = p.pos ? p.lane0 + m : p.lane0;
+    const int low = p.chunk ? pos - pos % p.chunk : 0, tile_lo = low / kTile, ntiles = pos / kTile - tile_lo + 1;
+    const int active = min(splits, ntiles);
+    if (split >= active) return;
+    const int j0 = tile_lo + (int)((long long)ntiles * split / active), j1 = tile_lo + (int)((long long)ntiles * (split + 1) / active);
+    const bool newest = p.pos && split == active - 1;  // (otherwise every position is in the cache)
+    const int vrows = vrows_of(p.vdim), QD = p.heads * p.dim, KD = p.kv_heads * p.dim, kcols = kchunks * C;
+    float *sq = reinterpret_cast<float*>(sm), *so = sq + HB * kcols;              // queries [HB][kcols]; sums [HB][vrows]
+    uint4* skey = reinterpret_cast<uint4*>(so + HB * vrows);                      // the newest key's chunks
+    float* sval = reinterpret_cast<float*>(skey + kchunks);                       // the newest value
+    const float* row = p.proj + (size_t)m * p.ldp;
+    uint8_t *kc = p.k + (size_t)seq * p.k_lane, *vc = p.vt + (size_t)seq * p.vt_lane;
+    for (int i = warp; i <= nh; i += 8) {
+        const float* x = i < nh ? row + (h0 + i) * p.dim : row + QD + g * p.dim;
+        const float by = p.qk_norm ? head_rstd(x, p.dim, p.eps, lane) : 1.f;
+        if (lane == 0) (i < nh ? s_rq[i] : s_rk) = by;
+    }
+    if (tid < HB) {
+        s_max[tid] = p.sink && split == 0 ? 0.f : -INFINITY;
+        s_sum[tid] = p.sink && split == 0 ? 1.f : 0.f;
+    }
+    for (int i = tid; i < HB * vrows; i += kStepThreads) so[i] = 0.f;
+    __syncthreads();
+    for (int i = tid; i < HB * kcols; i += kStepThreads) {
+        const int h = i / kcols, d = i - h * kcols;
+        sq[i] = h < nh && d < p.dim ? row[(h0 + h) * p.dim + d] * s_rq[h] : 0.f;
+    }
+    if (newest) {
+        const int r = pos % p.ring;
+        for (int c = tid; c < kchunks; c += kStepThreads) {
+            float f[C];
+            lb_load_cols<C>(row + QD + g * p.dim, c * C, p.dim, false, f);
+#pragma unroll
+            for (int e = 0; e < C; ++e) f[e] *= s_rk;
+            const uint4 w = lb_pack_chunk<WT>(f);
+            skey[c] = w;
+            if (hb == 0) *reinterpret_cast<uint4*>(kc + key_chunk(r, g, p.kv_heads, kchunks, c)) = w;
+        }
+        for (int v = tid; v < p.vdim; v += kStepThreads) {
+            const WT w = (WT)row[QD + KD + g * p.vdim + v];
+            sval[v] = (float)w;
+            if (hb == 0) *reinterpret_cast<WT*>(vc + value_at<WT>(g, v, vrows, r, p.slices)) = w;
+        }
+    }
+    __syncthreads();
+    const int kg = (warp << 3) | (lane >> 2), kt = lane & 3;  // key of the tile, quarter of its chunks
+    for (int j = j0; j < j1; ++j) {
+        const int base = j * kTile, rbase = base % p.ring;
+        // ---- scores ----
+        {
+            const int key = base + kg;
+            float a[HB];
+#pragma unroll
+            for (int h = 0; h < HB; ++h) a[h] = 0.f;
+            if (key >= low && key <= pos) {
+                const uint8_t* src = kc + key_chunk(rbase + kg, g, p.kv_heads, kchunks, 0);
+                const bool fresh = newest && key == pos;
+#pragma unroll 4
+                for (int c = kt; c < kchunks; c += 4) {
+                    float f[C];
+                    lb_unpack_chunk<WT>(fresh ? skey[c] : *reinterpret_cast<const uint4*>(src + (size_t)c * 128), f);
+#pragma unroll
+                    for (int h = 0; h < HB; ++h)
+#pragma unroll
+                        for (int e = 0; e < C; e += 4) {
+                            const float4 q = *reinterpret_cast<const float4*>(sq + h * kcols + c * C + e);
+                            a[h] = fmaf(f[e], q.x, fmaf(f[e + 1], q.y, fmaf(f[e + 2], q.z, fmaf(f[e + 3], q.w, a[h]))));
+                        }
+                }
+            }
+            const float* bias = p.bias + kBiasFront + min(max(pos - key, 0), p.bias_len - 1);
+#pragma unroll
+            for (int h = 0; h < HB; ++h) {
+                a[h] += __shfl_xor_sync(0xffffffffu, a[h], 1);
+                a[h] += __shfl_xor_sync(0xffffffffu, a[h], 2);
+                if (kt == 0) {
+                    float s = -INFINITY;
+                    if (h < nh && key >= low && key <= pos) s = fmaf(a[h], p.scale, p.bias ? bias[(size_t)(h0 + h) * p.bias_ld] : 0.f);
+                    s_w[h][kg] = s;
+                }
+            }
+        }
+        __syncthreads();
+        // ---- running softmax: a warp per head, two positions per lane (every tile has a visible position) ----
+        for (int h = warp; h < nh; h += 8) {
+            const float x0 = s_w[h][lane], x1 = s_w[h][lane + 32], old = s_max[h];
+            const float mx = fmaxf(old, lb_warp_max(fmaxf(x0, x1)));
+            const float w0 = expf(x0 - mx), w1 = expf(x1 - mx), sum = lb_warp_sumf(w0 + w1);
+            const int at = newest && pos >= base && pos < base + kTile ? pos - base : -1;  // its value is not in the cache yet
+            s_w[h][lane] = lane == at ? 0.f : w0;
+            s_w[h][lane + 32] = lane + 32 == at ? 0.f : w1;
+            if (at >= 0 && lane == (at & 31)) s_new[h] = at < 32 ? w0 : w1;
+            if (lane == 0) {
+                const float f = expf(old - mx);
+                s_max[h] = mx;
+                s_sum[h] = fmaf(s_sum[h], f, sum);
+                s_fac[h] = f;
+            }
+        }
+        __syncthreads();
+        // ---- weighted sum: lane (row of eight, chunk quarter) ----
+        const bool with_new = newest && pos >= base && pos < base + kTile;
+        for (int vg = warp; vg < vrows / 8; vg += 8) {
+            const int v = vg * 8 + (lane >> 2), irow = g * vrows + v;
+            uint4 w[2 * KS];
+#pragma unroll
+            for (int x = 0; x < 2 * KS; ++x) {
+                const int c = kt + 4 * x;
+                w[x] = *reinterpret_cast<const uint4*>(vc + lb_img_chunk(irow, rbase / C + c, p.slices));
+            }
+            float a[HB];
+#pragma unroll
+            for (int h = 0; h < HB; ++h) a[h] = 0.f;
+#pragma unroll
+            for (int x = 0; x < 2 * KS; ++x) {
+                const int c = kt + 4 * x;
+                float f[C];
+                lb_unpack_chunk<WT>(w[x], f);
+#pragma unroll
+                for (int h = 0; h < HB; ++h)
+#pragma unroll
+                    for (int e = 0; e < C; e += 4) {
+                        const float4 s = *reinterpret_cast<const float4*>(&s_w[h][c * C + e]);
+                        a[h] = fmaf(f[e], s.x, fmaf(f[e + 1], s.y, fmaf(f[e + 2], s.z, fmaf(f[e + 3], s.w, a[h]))));
+                    }
+            }
+#pragma unroll
+            for (int h = 0; h < HB; ++h) {
+                a[h] += __shfl_xor_sync(0xffffffffu, a[h], 1);
+                a[h] += __shfl_xor_sync(0xffffffffu, a[h], 2);
+                if (kt == 0 && h < nh) {
+                    if (with_new && v < p.vdim) a[h] = fmaf(s_new[h], sval[v], a[h]);
+                    so[h * vrows + v] = fmaf(so[h * vrows + v], s_fac[h], a[h]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    const float* gate = row + QD + KD + p.kv_heads * p.vdim;
+    float* o = out + (size_t)m * ldo;
+    if (active == 1) {
+        for (int i = tid; i < nh * p.vdim; i += kStepThreads) {
+            const int h = i / p.vdim, v = i - h * p.vdim;
+            const float r = __fdiv_rn(so[h * vrows + v], s_sum[h]);
+            o[(h0 + h) * p.vdim + v] = p.head_gate ? r * lb_sigmoidf(gate[h0 + h]) : r;
+        }
+        return;
+    }
+    // ---- partial sums [token][kv head and block][split][HB][vdim + 2], merged by the last to arrive ----
+    const int prow = p.vdim + 2, group = m * gridDim.y + blockIdx.y;
+    float* mine = part + ((size_t)group * splits + split) * HB * prow;
+    for (int i = tid; i < nh * p.vdim; i += kStepThreads) {
+        const int h = i / p.vdim, v = i - h * p.vdim;
+        mine[h * prow + v] = so[h * vrows + v];
+    }
+    if (tid < nh) {
+        mine[tid * prow + p.vdim] = s_max[tid];
+        mine[tid * prow + p.vdim + 1] = s_sum[tid];
+    }
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) {
+        s_last = atomicAdd(count + group, 1u) == (unsigned)active - 1;
+        if (s_last) count[group] = 0;
+    }
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+    const float* all = part + (size_t)group * splits * HB * prow;
+    float* sw = sq;  // [HB][64] share of every split
+    for (int h = warp; h < nh; h += 8) {
+        float mx = -INFINITY, den = 0.f;
+        for (int s = lane; s < active; s += 32) mx = fmaxf(mx, __ldcg(all + ((size_t)s * HB + h) * prow + p.vdim));
+        mx = lb_warp_max(mx);
+        for (int s = lane; s < active; s += 32) {
+            const float w = expf(__ldcg(all + ((size_t)s * HB + h) * prow + p.vdim) - mx);
+            sw[h * 64 + s] = w;
+            den = fmaf(w, __ldcg(all + ((size_t)s * HB + h) * prow + p.vdim + 1), den);
+        }
+        den = lb_warp_sumf(den);
+        float r = __fdiv_rn(1.f, den);
+        if (p.head_gate) r *= lb_sigmoidf(gate[h0 + h]);
+        __syncwarp();
+        for (int s = lane; s < active; s += 32) sw[h * 64 + s] *= r;
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * p.vdim; i += kStepThreads) {
+        const int h = i / p.vdim, v = i - h * p.vdim;
+        float a = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < active; ++s) a = fmaf(sw[h * 64 + s], __ldcg(all + ((size_t)s * HB + h) * prow + v), a);
+        o[(h0 + h) * p.vdim + v] = a;
+    }
+}
+
+// query heads of a CTA of the step
+int heads_block(const LbAttention& p) {
+    const int per = p.heads / p.kv_heads;
+    return per >= 8 ? 8 : per > 2 ? 4 : per;
+}
+int groups_of(const LbAttention& p) { return p.kv_heads * lb_ceil_div(p.heads / p.kv_heads, heads_block(p)); }
+
+size_t step_smem(const LbAttention& p, int HB, int kchunks, int C) {
+    const size_t front = (size_t)HB * kchunks * C < (size_t)HB * 64 ? (size_t)HB * 64 : (size_t)HB * kchunks * C;  // (the merge uses 64 a head)
+    return (front + (size_t)HB * vrows_of(p.vdim)) * sizeof(float) + (size_t)kchunks * 16 + (size_t)p.vdim * sizeof(float);
+}
+constexpr size_t kStepSmem = 200 * 1024;
+
+template <typename WT, int HB>
+int launch_step(loom_b200_ctx* ctx, const LbAttention& p, int tokens, int kchunks, float* part, unsigned* count, float* out, int ldo) {
+    const size_t smem = step_smem(p, HB, kchunks, LbElem<WT>::kChunk);
+    LB_REQUIRE(ctx, smem <= kStepSmem, "attention: head dimensions %d and %d", p.dim, p.vdim);
+    if (smem > 40 * 1024) LB_BIG_SMEM(ctx, (lb_attention_step_kernel<WT, HB>), kStepSmem);
+    const int splits = lb_attention_splits(ctx, p, tokens);
+    LB_LAUNCH(ctx, (lb_attention_step_kernel<WT, HB>), dim3(splits, groups_of(p), tokens), dim3(kStepThreads), smem, p, kchunks, splits, part, count, out, ldo);
+    return 0;
+}
+
+template <typename WT>
+int step_heads(loom_b200_ctx* ctx, const LbAttention& p, int tokens, int kchunks, float* part, unsigned* count, float* out, int ldo) {
+    switch (heads_block(p)) {
+        case 1: return launch_step<WT, 1>(ctx, p, tokens, kchunks, part, count, out, ldo);
+        case 2: return launch_step<WT, 2>(ctx, p, tokens, kchunks, part, count, out, ldo);
+        case 4: return launch_step<WT, 4>(ctx, p, tokens, kchunks, part, count, out, ldo);
+    }
+    return launch_step<WT, 8>(ctx, p, tokens, kchunks, part, count, out, ldo);
+}
+
+}  // namespace
+
+int lb_attention_kchunks(int dim, int dtype) { return lb_round_up(lb_ceil_div(dim, dtype == LOOM_B200_DTYPE_BF16 ? 8 : 4), 2); }
+
+size_t lb_attention_k_bytes(int kv_heads, int dim, int ring, int dtype) { return (size_t)(ring / 128) * kv_heads * lb_attention_kchunks(dim, dtype) * 2048; }
+
+size_t lb_attention_vt_bytes(int kv_heads, int vdim, int ring, int dtype) { return lb_img_bytes(kv_heads * vrows_of(vdim), ring, dtype); }
+
+size_t lb_attention_q_bytes(const LbAttention& p, int rows) { return (size_t)lb_ceil_div(rows, 128) * p.heads * lb_attention_kchunks(p.dim, LOOM_B200_DTYPE_BF16) * 2048; }
+
+int lb_attention_store(loom_b200_ctx* ctx, int dtype, const LbAttention& p, int T, uint8_t* q_img) {
+    const int kch = lb_attention_kchunks(p.dim, dtype), qch = lb_attention_kchunks(p.dim, LOOM_B200_DTYPE_BF16);
+    const dim3 grid((p.pos0 + T - 1) / 8 - p.pos0 / 8 + 1);
+    const bool vec = p.dim % 4 == 0 && lb_vec_rows(p.proj, p.ldp);
+    if (dtype == LOOM_B200_DTYPE_BF16)
+        LB_LAUNCH(ctx, lb_attention_store_kernel<__nv_bfloat16>, grid, dim3(256), 0, p, T, kch, qch, q_img, vec);
+    else
+        LB_LAUNCH(ctx, lb_attention_store_kernel<float>, grid, dim3(256), 0, p, T, kch, qch, nullptr, vec);
+    return 0;
+}
+
+int lb_attention_splits(loom_b200_ctx* ctx, const LbAttention& p, int tokens) {
+    int s = lb_ceil_div(4 * ctx->sm_count, groups_of(p) * tokens);
+    const int tiles = (p.chunk && p.chunk < p.ring ? p.chunk : p.ring) / kTile + 2;  // a chunk may begin and end inside a tile
+    if (s > tiles) s = tiles;
+    if (s > 64) s = 64;
+    return s < 1 ? 1 : s;
+}
+
+size_t lb_attention_part_elems(loom_b200_ctx* ctx, const LbAttention& p, int tokens) {
+    return (size_t)tokens * groups_of(p) * lb_attention_splits(ctx, p, tokens) * heads_block(p) * (p.vdim + 2);
+}
+
+size_t lb_attention_counters(const LbAttention& p, int tokens) { return (size_t)tokens * groups_of(p); }
+
+int lb_attention_step(loom_b200_ctx* ctx, int dtype, const LbAttention& p, int tokens, float* part, unsigned* count, float* out, int ldo) {
+    const int kch = lb_attention_kchunks(p.dim, dtype);
+    LB_REQUIRE(ctx, tokens > 0 && tokens <= 65535, "attention: %d tokens", tokens);
+    return dtype == LOOM_B200_DTYPE_BF16 ? step_heads<__nv_bfloat16>(ctx, p, tokens, kch, part, count, out, ldo) : step_heads<float>(ctx, p, tokens, kch, part, count, out, ldo);
+}
+
+bool lb_attention_block_supported(const LbAttention& p) { return p.dim <= 256 && p.vdim <= 128; }
+
+int lb_attention_block(loom_b200_ctx* ctx, const LbAttention& p, int T, const uint8_t* q_img, uint8_t* out, int out_slices) {
+    LbAttnBlock a;
+    a.q = q_img;
+    a.k = p.k + (size_t)p.lane0 * p.k_lane;
+    a.vt = p.vt + (size_t)p.lane0 * p.vt_lane;
+    a.heads = p.heads;
+    a.kv_heads = p.kv_heads;
+    a.dchunks = lb_attention_kchunks(p.dim, LOOM_B200_DTYPE_BF16);
+    a.vdim = p.vdim;
+    a.vrows = vrows_of(p.vdim);
+    a.vslices = p.slices;
+    a.T = T;
+    a.pos0 = p.pos0;
+    a.scale_log2 = p.scale * 1.4426950408889634f;
+    a.out = out;
+    a.out_slices = out_slices;
+    a.general = true;
+    a.chunk = p.chunk;
+    a.ring = p.ring;
+    a.bias = p.bias_log2;
+    a.bias_len = p.bias_len;
+    a.bias_ld = p.bias_ld;
+    a.sink = p.sink;
+    a.gate = p.head_gate ? p.proj + (size_t)p.heads * p.dim + (size_t)p.kv_heads * (p.dim + p.vdim) : nullptr;
+    a.ldg = p.ldp;
+    return lb_attn_block(ctx, a);
+}

@@ -48,4 +48,17 @@ def load(ctx, path: str, dtype: str = "bfloat16", max_seq_len: int = 2048, batch
     return build(ctx, read_config(path), Checkpoint(path), LoadOptions(cabi.DTYPES[dtype], max_seq_len, batch))
 
 
-from . import zitupel  # noqa: E402,F401
+def matrix(ctx, weights, dtype: int, parts: list, cols: int) -> "cabi.Matrix":
+    """A matrix out of a checkpoint: parts [(tensor, rows)] are stacked; a list of such lists gives one group each."""
+    groups = parts if isinstance(parts[0], list) else [parts]
+    m = cabi.Matrix(ctx, sum(r for _, r in groups[0]), cols, len(groups), dtype)
+    for g, rows in enumerate(groups):
+        at = 0
+        for name, n in rows:
+            a, code = weights.raw(name, (n, cols))
+            m.put(a, code, row0=at, group=g)
+            at += n
+    return m
+
+
+from . import donodra, zitupel  # noqa: E402,F401

@@ -12,6 +12,7 @@ import numpy as np
 
 from .. import cabi
 from . import LoadOptions, register
+from . import matrix as stacked
 
 
 @dataclasses.dataclass
@@ -71,16 +72,7 @@ def build_decoder(ctx, config: dict, weights, options: LoadOptions) -> "cabi.Dec
     dec.set_batch(options.batch)
 
     def matrix(parts, cols):
-        """parts: [(tensor, rows)] stacked, or a list of such lists, one per group."""
-        groups = parts if isinstance(parts[0], list) else [parts]
-        m = cabi.Matrix(ctx, sum(r for _, r in groups[0]), cols, len(groups), dt)
-        for g, rows in enumerate(groups):
-            at = 0
-            for name, n in rows:
-                a, code = weights.raw(name, (n, cols))
-                m.put(a, code, row0=at, group=g)
-                at += n
-        return m
+        return stacked(ctx, weights, dt, parts, cols)
 
     for i, layer in enumerate(layers):
         s, p = layer.spec, "l%d." % i
