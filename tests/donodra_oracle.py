@@ -37,7 +37,7 @@ def chunked_biased_attention(q, k, v, scale, rel, far, chunk):
         lo = i // chunk * chunk
         for h in range(heads):
             g = h // per
-            s = np.array([q[i, h] @ k[j, g] * scale + bias[i - j, h] for j in range(lo, i + 1)])
+            s = k[lo:i + 1, g] @ q[i, h] * scale + bias[i - np.arange(lo, i + 1), h]
             m = max(s.max(), 0.0)
             p = np.exp(s - m)
             out[i, h] = (p / (np.exp(-m) + p.sum())) @ v[lo:i + 1, g]
