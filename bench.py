@@ -777,12 +777,14 @@ def batch_mode(args):
     return 0
 
 
-# Layer stacks (`--mode stack`): a Zitupel of each size beside a ternary decoder of the same width, depth, vocabulary and -- for the
-# dense size -- feed-forward.  Every fourth layer is latent attention, and every second of those reads the latents of the one before.
+# Layer stacks (`--mode stack`).  `--design zitupel`: a Zitupel of each size beside a ternary decoder of the same width, depth,
+# vocabulary and -- for the dense size -- feed-forward.  Every fourth layer is latent attention, and every second of those reads the
+# latents of the one before.  `--design donodra`: a Donodra (attention, delta rule, attention, matrix memory) beside a Zitupel of the
+# same width, depth, vocabulary, recurrent heads and feed-forward parameters.
 STACK_SHAPES = {
-    "2b": dict(layers=8, width=2560, vocab=128256, gla=(10, 128, 256, 16), latent=(20, 128, 128, 512), ff=6912, experts=0, top=0,
+    "2b": dict(layers=8, width=2560, vocab=128256, gla=(10, 128, 256, 16), latent=(20, 128, 128, 512), ff=6912, experts=0, top=0, attention=(20, 5, 128, 128),
                ternary=dict(heads=20, kv_heads=5, inter=6912)),
-    "8b": dict(layers=8, width=4096, vocab=128256, gla=(16, 128, 256, 16), latent=(32, 128, 128, 512), ff=14336, experts=0, top=0,
+    "8b": dict(layers=8, width=4096, vocab=128256, gla=(16, 128, 256, 16), latent=(32, 128, 128, 512), ff=14336, experts=0, top=0, attention=(32, 8, 128, 128),
                ternary=dict(heads=32, kv_heads=8, inter=14336)),
     "8b-moe": dict(layers=8, width=4096, vocab=128256, gla=(16, 128, 256, 16), latent=(32, 128, 128, 512), ff=1792, experts=32, top=4,
                    ternary=dict(heads=32, kv_heads=8, inter=7168)),  # the experts a token goes through add up to inter
@@ -810,6 +812,18 @@ def stack_config(sh):
             "vocab": sh["vocab"], "width": sh["width"]}
 
 
+def donodra_config(sh):
+    """Chunks as long as those of real models, so a prompt of a few thousand tokens sees all of itself."""
+    h, g, dim, vdim = sh["attention"]
+    rh, rdim, rvdim, _ = sh["gla"]
+    attention = ("attention", {"heads": h, "kv_heads": g, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "bias_max": 128, "mask": {"size": 8192}})
+    delta = ("delta", {"heads": rh, "kv_heads": rh, "dim": rdim, "vdim": rvdim, "conv": 4})
+    mlstm = ("mlstm", {"heads": rh, "dim": rdim, "vdim": rvdim, "gate_cap": 15.0})
+    order = [attention, delta, attention, mlstm]
+    return {"architecture": "Donodra", "layers": [{"type": order[i % 4][0], "mixer": order[i % 4][1], "mlp": {"kind": "dense", "ff": sh["ff"]}} for i in range(sh["layers"])],
+            "norm": {"eps": 1e-5}, "postln_alpha": 2.0, "vocab": sh["vocab"], "width": sh["width"]}
+
+
 class RandomWeights:
     """Seeded random tensors under a checkpoint's interface, made on the device as they are asked for."""
 
@@ -830,7 +844,7 @@ class RandomWeights:
 
     def f32(self, name, shape):
         t = self.torch.randn(*shape, device=self.dev, generator=self.g, dtype=self.torch.float32) * 0.1
-        return (t + (1.0 if name.endswith("norm") else 3.0 if name.endswith(".b") else 0.0)).cpu().numpy()
+        return (t + (1.0 if ".norm" in name else 3.0 if name.endswith(".b") else 0.0)).cpu().numpy()
 
     def scalar(self, name):
         return 1.0
@@ -870,8 +884,8 @@ def stack_measure(torch, ctx, dec, vocab, prompt_len, steps, warmup, batch, reps
 
 
 def stack_mode(args):
-    """A layer stack and a ternary decoder of equal size, one after the other on one GPU: prompt tok/s and greedy decode tok/s for
-    one and for `--batch` sequences.  The value is the stack's batch-1 decode rate."""
+    """A layer stack and the closest other model of equal size, one after the other on one GPU: prompt tok/s and greedy decode tok/s
+    for one and for `--batch` sequences.  The value is the stack's batch-1 decode rate."""
     import torch
 
     import loom_b200
@@ -884,19 +898,27 @@ def stack_mode(args):
         sh["layers"] = args.layers
     if args.vocab != SHAPE["vocab"]:
         sh["vocab"] = args.vocab
+    donodra = args.design == "donodra"
+    if donodra and sh["experts"]:
+        raise SystemExit("--design donodra has no routed experts: choose --stack-shape 2b or 8b")
+    kinds = ("donodra", "zitupel") if donodra else ("stack", "ternary")
     msl = args.prompt + warm + steps * reps + 8
     clocks = ClockSampler(0)
     clocks.start()
     out, launches = {}, 0
     for batch in sorted({1, args.batch}):
-        for kind in ("stack", "ternary"):
+        for kind in kinds:
             if args.only and kind != args.only:
                 continue
             ctx = loom_b200.Context(0)
             apply_opts(ctx, args)
-            if kind == "stack":
-                dec = models.build(ctx, stack_config(sh), RandomWeights(torch, dev, {"a1": (sh["gla"][3], sh["width"])}, args.seed),
-                                   models.LoadOptions(cabi.DTYPES[args.dtype], msl, batch))
+            if kind != "ternary":
+                if kind == "donodra":
+                    cfg = donodra_config(sh)
+                else:  # (beside a gated feed-forward: as many parameters in two matrices as in three)
+                    cfg = stack_config(dict(sh, ff=sh["ff"] * 3 // 2) if donodra else sh)
+                sizes = {"a1": (sh["gla"][3], sh["width"]), "rel": (32, sh.get("attention", (0,))[0])}
+                dec = models.build(ctx, cfg, RandomWeights(torch, dev, sizes, args.seed), models.LoadOptions(cabi.DTYPES[args.dtype], msl, batch))
                 keep = None
             else:
                 t = sh["ternary"]
@@ -911,8 +933,9 @@ def stack_mode(args):
             del dec, keep
             ctx.close()
             torch.cuda.empty_cache()
-    first = out.get("stack", out.get("ternary"))["batch1"]
-    print(json.dumps({"metric": "decode tok/s (Zitupel, %s-shape layers, bs=1) beside a ternary decoder of equal size" % args.stack_shape,
+    first = out.get(kinds[0], out.get(kinds[1]))["batch1"]
+    names = ("Donodra", "a Zitupel") if donodra else ("Zitupel", "a ternary decoder")
+    print(json.dumps({"metric": "decode tok/s (%s, %s-shape layers, bs=1) beside %s of equal size" % (names[0], args.stack_shape, names[1]),
                       "value": first["decode_tok_per_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warm, "ms_per_step": first["step_ms"],
                       "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": args.dtype, "data": "synthetic",
                       "config": {"shape": args.stack_shape, "layers": sh["layers"], "width": sh["width"], "prompt": args.prompt, "vocab": sh["vocab"],
@@ -941,10 +964,11 @@ def main():
     ap.add_argument("--tp-exchange", default="peer", choices=["peer", "nccl"],
                     help="tp mode: how the row-parallel projections exchange their partial results")
     ap.add_argument("--tokens", type=int, default=512)
-    ap.add_argument("--stack-shape", default="2b", choices=sorted(STACK_SHAPES), help="stack mode: a layer stack and a ternary decoder of equal size")
+    ap.add_argument("--stack-shape", default="2b", choices=sorted(STACK_SHAPES), help="stack mode: the size of the layers")
+    ap.add_argument("--design", default="zitupel", choices=["zitupel", "donodra"], help="stack mode: Zitupel beside a ternary decoder, or Donodra beside Zitupel")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="stack mode: element type of the stack")
     ap.add_argument("--reps", type=int, default=5, help="stack mode: repetitions of a timed region (the median counts)")
-    ap.add_argument("--only", default="", choices=["", "stack", "ternary"], help="stack mode: one of the two models (profiling)")
+    ap.add_argument("--only", default="", choices=["", "stack", "ternary", "donodra", "zitupel"], help="stack mode: one of the two models (profiling)")
     ap.add_argument("--no-tp-section", action="store_true", help="multi-GPU runs: skip the tensor-parallel decode after the replica measurement")
     args = ap.parse_args()
     if args.mode == "gemm":
