@@ -4,7 +4,7 @@
 //
 // A block of tokens is cut into chunks of C.  With G_t the product of the decays inside a chunk and S the state in front of it,
 //   u_t + sum_(s < t) L_ts u_s = beta_t v_t - beta_t G_t S^T k_t,   L_ts = beta_t (G_t / G_s) k_t.k_s
-// so forward substitution with L on the columns of (beta v | beta G k) gives u = Wv - Wk S without knowing S, and
+// so (I + L)^-1 times (beta v | beta G k) gives u = Wv - Wk S without knowing S, and
 //   o_t   = (G_t q_t - sum_s A_ts wk_s)^T S + sum_s A_ts wv_s,   A_ts = (G_t / G_s) q_t.k_s, s <= t
 //   S_end = (G_C - Kd^T Wk) S + Kd^T Wv,                         Kd_s = (G_C / G_s) k_s
 // Only the last line runs chunk after chunk.  Ratios of decays come from differences of their logarithms (no exponent is ever
@@ -122,43 +122,66 @@ __global__ void __launch_bounds__(256) lb_delta_step_kernel(const LbDelta p, con
 
 constexpr int kRows = 8;  // tokens of a CTA
 
-// convolution, activation and norms of the block's tokens, their gates: a warp per (head of q, k or v; token)
+// columns c .. c + 3 of a row of n
+template <bool VEC>
+__device__ __forceinline__ void store4(float* row, int c, int n, const float* f) {
+    if (VEC && c + 4 <= n) {
+        *reinterpret_cast<float4*>(row + c) = make_float4(f[0], f[1], f[2], f[3]);
+    } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+            if (c + e < n) row[c + e] = f[e];
+    }
+}
+
+// Convolution, activation and norms of the block's tokens, their gates: a warp per (head of q, k or v; token), four channels per
+// lane and pass.
+template <bool VEC>
 __global__ void __launch_bounds__(256) lb_delta_tokens_kernel(const LbDelta p, const LbDeltaBlock b, int T, int pos0) {
     lb_pdl_launch_dependents();
     lb_pdl_wait();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t0 = blockIdx.x * kRows, rows = min(kRows, T - t0);
-    const int nch = lb_delta_channels(p), slots = 2 * p.kv_heads + p.heads, back = p.taps - 1;
-    for (int i = warp; i < slots * kRows; i += 8) {
-        const int slot = i / kRows, t = t0 + i % kRows;
-        if (t >= T) continue;
-        const bool value = slot >= 2 * p.kv_heads;
-        const int n = value ? p.vdim : p.dim, c0 = value ? 2 * p.kv_heads * p.dim + (slot - 2 * p.kv_heads) * p.vdim : slot * p.dim;
-        float* out = b.qkv + (size_t)t * nch + c0;
-        const float *x = p.proj + c0, *w = p.conv_w + c0;
-        float ss = 0.f;
-        for (int c = lane; c < n; c += 32) {
-            float a = 0.f;
-#pragma unroll 4
-            for (int j = 0; j <= back; ++j) {
-                const int ts = t - back + j;
-                if (pos0 + ts < 0) continue;
-                const float y = ts >= 0 ? x[(size_t)ts * p.ldp + c] : p.ring[(size_t)((pos0 + ts) % p.taps) * nch + c0 + c];
-                a = fmaf(w[(size_t)j * nch + c], y, a);
-            }
-            a = lb_siluf(a);
-            out[c] = a;
-            ss = fmaf(a, a, ss);
-        }
-        if (value) continue;
-        ss = lb_warp_sumf(ss);
-        const float r = __fdiv_rn(slot < p.kv_heads ? p.qscale : 1.f, sqrtf(ss + kUnitEps));
-        for (int c = lane; c < n; c += 32) out[c] *= r;  // (a thread reads back what it wrote)
-    }
-    for (int i = threadIdx.x; i < rows * p.heads; i += 256) {
-        const int t = t0 + i / p.heads, h = i % p.heads;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, slots = 2 * p.kv_heads + p.heads, nch = lb_delta_channels(p), back = p.taps - 1;
+    const int t = blockIdx.x * kRows + warp, slot = blockIdx.y;
+    if (t >= T) return;
+    if (slot == slots) {  // the last row of CTAs makes the gates
         const float* row = p.proj + (size_t)t * p.ldp;
-        b.beta[(size_t)t * p.heads + h] = write_strength(p, row, h);
-        b.logg[(size_t)t * p.heads + h] = log_gate(p, row, h);
+        for (int h = lane; h < p.heads; h += 32) {
+            b.beta[(size_t)t * p.heads + h] = write_strength(p, row, h);
+            b.logg[(size_t)t * p.heads + h] = log_gate(p, row, h);
+        }
+        return;
+    }
+    const bool value = slot >= 2 * p.kv_heads;
+    const int n = value ? p.vdim : p.dim, c0 = value ? 2 * p.kv_heads * p.dim + (slot - 2 * p.kv_heads) * p.vdim : slot * p.dim;
+    float* out = b.qkv + (size_t)t * nch + c0;
+    float ss = 0.f;
+    for (int c = lane * 4; c < n; c += 128) {
+        float a[4] = {0.f, 0.f, 0.f, 0.f}, w[4], y[4];
+#pragma unroll 4
+        for (int j = 0; j <= back; ++j) {
+            const int ts = t - back + j;
+            if (pos0 + ts < 0) continue;
+            lb_load_cols<4>(p.conv_w + (size_t)j * nch + c0, c, n, VEC, w);
+            lb_load_cols<4>(ts >= 0 ? p.proj + (size_t)ts * p.ldp + c0 : p.ring + (size_t)((pos0 + ts) % p.taps) * nch + c0, c, n, VEC, y);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) a[e] = fmaf(w[e], y[e], a[e]);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            a[e] = lb_siluf(a[e]);  // (zero behind the last channel)
+            ss = fmaf(a[e], a[e], ss);
+        }
+        store4<VEC>(out, c, n, a);
+    }
+    if (value) return;
+    ss = lb_warp_sumf(ss);
+    const float r = __fdiv_rn(slot < p.kv_heads ? p.qscale : 1.f, sqrtf(ss + kUnitEps));
+    for (int c = lane * 4; c < n; c += 128) {  // (a thread reads back what it wrote)
+        float a[4];
+        lb_load_cols<4>(out, c, n, VEC, a);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[e] *= r;
+        store4<VEC>(out, c, n, a);
     }
 }
 
@@ -173,38 +196,133 @@ __global__ void __launch_bounds__(256) lb_delta_commit_kernel(const LbDelta p, i
 
 __host__ __device__ inline int lead(int dim) { return lb_round_up(dim, 4) + 4; }
 
+// acc[i][e] += sum over s of m[ty + 16 i][s] x[s][col + e] for a lower triangular m (its upper blocks are never read)
+template <int NI>
+__device__ __forceinline__ void tri_mul(const float* m, int ldm, const float* x, int ldx, int ty, int col, float (*acc)[4]) {
+#pragma unroll
+    for (int sb = 0; sb < NI; ++sb)
+#pragma unroll
+        for (int s = sb * 16; s < sb * 16 + 16; s += 4) {
+            float4 w[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float4*>(x + (s + e) * ldx + col);
+#pragma unroll
+            for (int i = sb; i < NI; ++i) {
+                const float4 a = *reinterpret_cast<const float4*>(m + (ty + 16 * i) * ldm + s);
+                const float av[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    acc[i][0] = fmaf(av[e], w[e].x, acc[i][0]);
+                    acc[i][1] = fmaf(av[e], w[e].y, acc[i][1]);
+                    acc[i][2] = fmaf(av[e], w[e].z, acc[i][2]);
+                    acc[i][3] = fmaf(av[e], w[e].w, acc[i][3]);
+                }
+            }
+        }
+}
+
+// (I + L)^-1 in place of the strictly lower triangular L [C][ld]: blocks of sixteen by substitution, a thread per column, then pairs of
+// blocks of 16 and of 32: the lower left block of the inverse is -T22 L21 T11.  x: C/2 * C/2 floats
+template <int C>
+__device__ __forceinline__ void invert(float* l, int ld, float* x, int tid) {
+    const int blk = tid >> 4, j = tid & 15;
+    float c[16];
+    if (blk < C / 16) {
+        const float* b = l + (blk * 16) * ld + blk * 16;
+#pragma unroll
+        for (int t = 0; t < 16; ++t) {
+            float a = t == j ? 1.f : 0.f;
+#pragma unroll
+            for (int s = 0; s < t; ++s) a = fmaf(-b[t * ld + s], c[s], a);
+            c[t] = a;
+        }
+    }
+    __syncthreads();
+    if (blk < C / 16)
+#pragma unroll
+        for (int t = 0; t < 16; ++t) l[(blk * 16 + t) * ld + blk * 16 + j] = c[t];
+    __syncthreads();
+#pragma unroll
+    for (int n = 16; n < C; n *= 2) {
+        for (int i = tid; i < C / (2 * n) * n * n; i += 256) {  // X = L21 T11
+            const int q = i / (n * n), r = i / n % n, k = i % n;
+            const float *l21 = l + (2 * q * n + n + r) * ld + 2 * q * n, *t11 = l + 2 * q * n * ld + 2 * q * n + k;
+            float a = 0.f;
+            for (int e = 0; e < n; ++e) a = fmaf(l21[e], t11[e * ld], a);  // (T11 is zero above its diagonal)
+            x[i] = a;
+        }
+        __syncthreads();
+        for (int i = tid; i < C / (2 * n) * n * n; i += 256) {
+            const int q = i / (n * n), r = i / n % n, k = i % n;
+            const float* t22 = l + (2 * q * n + n + r) * ld + 2 * q * n + n;
+            float a = 0.f;
+            for (int e = 0; e < n; ++e) a = fmaf(-t22[e], x[q * n * n + e * n + k], a);
+            l[(2 * q * n + n + r) * ld + 2 * q * n + k] = a;
+        }
+        __syncthreads();
+    }
+}
+
+constexpr int kValueCols = 64;                 // value columns of a pass
+constexpr int kValueLd = kValueCols + 4;
+
 // CTA = (chunk, head): L and A, the substitution, and the operands of the products over chunks
 template <int C>
-__global__ void __launch_bounds__(256, 2) lb_delta_prep_kernel(const LbDelta p, const LbDeltaBlock b, int T) {
+__global__ void __launch_bounds__(256, 2) lb_delta_prep_kernel(const LbDelta p, const LbDeltaBlock b, int T, bool vec) {
     extern __shared__ __align__(16) float sm[];
     __shared__ double s_log[C];
-    __shared__ float s_beta[C], s_g[C];
+    __shared__ float s_beta[C], s_g[C], s_end[C];
     constexpr int NI = C / 16, LC = C + 4;
-    const int ch = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, dim = p.dim, LD = lead(dim);
+    const int ch = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, ty = tid >> 4, tx = tid & 15, dim = p.dim, LD = lead(dim), D4 = lb_round_up(dim, 4) / 4;
     const int hk = h / (p.heads / p.kv_heads), nch = lb_delta_channels(p), QK = p.kv_heads * dim, t0 = ch * C, n = min(C, T - t0);
-    float *sq = sm, *sk = sq + C * LD, *sl = sk + C * LD, *sa = sl + C * LC;
+    float *sk = sm, *sl = sk + C * LD, *sa = sl + C * LC, *sq = sa + C * LC;  // sq: also value columns [C][kValueLd], and scratch of the inversion
     lb_pdl_launch_dependents();
     lb_pdl_wait();
-    for (int i = tid; i < C * LD; i += 256) {
-        const int t = i / LD, d = i - t * LD;
-        const bool ok = t < n && d < dim;
-        const float* row = b.qkv + (size_t)(t0 + t) * nch + hk * dim + d;
-        sq[i] = ok ? row[0] : 0.f;
-        sk[i] = ok ? row[QK] : 0.f;
+    for (int i = tid; i < C * D4; i += 256) {
+        const int t = i / D4, d = (i - t * D4) * 4;
+        float q[4] = {0.f, 0.f, 0.f, 0.f}, k[4] = {0.f, 0.f, 0.f, 0.f};
+        if (t < n) {
+            const float* row = b.qkv + (size_t)(t0 + t) * nch + hk * dim;
+            lb_load_cols<4>(row, d, dim, vec, q);
+            lb_load_cols<4>(row + QK, d, dim, vec, k);
+        }
+        *reinterpret_cast<float4*>(sq + t * LD + d) = make_float4(q[0], q[1], q[2], q[3]);
+        *reinterpret_cast<float4*>(sk + t * LD + d) = make_float4(k[0], k[1], k[2], k[3]);
     }
     if (tid < C) {
         s_beta[tid] = tid < n ? b.beta[(size_t)(t0 + tid) * p.heads + h] : 0.f;
         s_log[tid] = tid < n ? (double)b.logg[(size_t)(t0 + tid) * p.heads + h] : 0.0;
     }
     __syncthreads();
-    if (tid == 0)
-        for (int t = 1; t < C; ++t) s_log[t] += s_log[t - 1];
+    if (tid < 32) {  // running sums: C / 32 tokens per lane, then over the lanes
+        constexpr int PER = C < 32 ? 1 : C / 32;
+        double v[PER], run = 0.0;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int t = tid * PER + i;
+            run += t < C ? s_log[t] : 0.0;
+            v[i] = run;
+        }
+        double before = run;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double up = __shfl_up_sync(0xffffffffu, before, o);
+            if (tid >= o) before += up;
+        }
+        before -= run;
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+            if (tid * PER + i < C) s_log[tid * PER + i] = before + v[i];
+    }
     __syncthreads();
-    if (tid < C) s_g[tid] = expf((float)s_log[tid]);
+    if (tid < C) {
+        s_g[tid] = expf((float)s_log[tid]);
+        s_end[tid] = expf((float)(s_log[C - 1] - s_log[tid]));
+    }
     {
-        const int ty = tid >> 4, tx = tid & 15;
         float qk[NI][NI] = {}, kk[NI][NI] = {};
-        for (int d = 0; d < dim; d += 4) {  // (columns dim .. LD are zero)
+#pragma unroll 2
+        for (int d = 0; d < dim; d += 4) {  // (columns dim .. are zero)
             float4 q[NI], a[NI], k[NI];
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
@@ -233,103 +351,110 @@ __global__ void __launch_bounds__(256, 2) lb_delta_prep_kernel(const LbDelta p, 
                     if (s < t) l = s_beta[t] * r * kk[i][j];
                 }
                 sl[t * LC + s] = l;
-                sa[t * LC + s] = w;
+                sa[t * LC + s] = -w;
                 A[t * C + s] = w;
             }
     }
     __syncthreads();
     if (tid == 0) b.c.decay[(size_t)ch * p.heads + h] = s_g[C - 1];
-    for (int i = tid; i < n * dim; i += 256) {
-        const int t = i / dim, d = i - t * dim;
-        b.c.kd[((size_t)(t0 + t) * p.heads + h) * dim + d] = sk[t * LD + d] * expf((float)(s_log[C - 1] - s_log[t]));
-    }
-    __syncthreads();
-    // a thread per column of (beta v | beta G k); the solved key columns replace the keys
-    for (int col = tid; col < p.vdim + dim; col += 256) {
-        const bool value = col < p.vdim;
-        const int d = col - p.vdim;
-        float w[C];
-#pragma unroll
-        for (int t = 0; t < C; ++t) {
-            if (value)
-                w[t] = t < n ? b.qkv[(size_t)(t0 + t) * nch + 2 * QK + h * p.vdim + col] * s_beta[t] : 0.f;
+    // keys decayed to the chunk's end; the keys in shared memory become beta G k, and queries go out of the way of the inversion
+    for (int i = tid; i < C * D4; i += 256) {
+        const int t = i / D4, d = (i - t * D4) * 4;
+        const float4 k = *reinterpret_cast<const float4*>(sk + t * LD + d);
+        const float e = s_end[t], g = s_beta[t] * s_g[t], f[4] = {k.x * e, k.y * e, k.z * e, k.w * e};
+        if (t < n) {
+            float* out = b.c.kd + ((size_t)(t0 + t) * p.heads + h) * dim;
+            if (vec)
+                store4<true>(out, d, dim, f);
             else
-                w[t] = sk[t * LD + d] * (s_beta[t] * s_g[t]);
+                store4<false>(out, d, dim, f);
         }
-#pragma unroll
-        for (int t = 1; t < C; ++t) {
-            float a0 = 0.f, a1 = 0.f;
-#pragma unroll
-            for (int s = 0; s < t; s += 4) {
-                const float4 l = *reinterpret_cast<const float4*>(sl + t * LC + s);
-                a0 = fmaf(l.x, w[s], a0);
-                if (s + 1 < t) a1 = fmaf(l.y, w[s + 1], a1);
-                if (s + 2 < t) a0 = fmaf(l.z, w[s + 2], a0);
-                if (s + 3 < t) a1 = fmaf(l.w, w[s + 3], a1);
-            }
-            w[t] -= a0 + a1;
-        }
-#pragma unroll
-        for (int t = 0; t < C; ++t) {
-            if (value) {
-                if (t < n) b.wv[(size_t)(t0 + t) * p.heads * p.vdim + h * p.vdim + col] = w[t];
-            } else {
-                sk[t * LD + d] = w[t];
-                if (t < n) b.wk[((size_t)(t0 + t) * p.heads + h) * dim + d] = w[t];
-            }
-        }
+        *reinterpret_cast<float4*>(sk + t * LD + d) = make_float4(k.x * g, k.y * g, k.z * g, k.w * g);
     }
-    __syncthreads();
-    const int ty = tid >> 4, tx = tid & 15;
-    for (int d = tx * 4; d < dim; d += 64) {
-        float acc[NI][4];
+    invert<C>(sl, LC, sq + C * (LD > kValueLd ? LD : kValueLd), tid);
+    for (int d = tx * 4, d0 = 0; d0 < dim; d += 64, d0 += 64) {  // Wk, in place of the keys, and the queries against the state
+        float acc[NI][4] = {};
+        if (d < dim) tri_mul<NI>(sl, LC, sk, LD, ty, d, acc);
+        __syncthreads();
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
             const int t = ty + 16 * i;
-            const float4 q = *reinterpret_cast<const float4*>(sq + t * LD + d);
-            acc[i][0] = s_g[t] * q.x;
-            acc[i][1] = s_g[t] * q.y;
-            acc[i][2] = s_g[t] * q.z;
-            acc[i][3] = s_g[t] * q.w;
+            if (d >= dim) continue;
+            *reinterpret_cast<float4*>(sk + t * LD + d) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+            if (t >= n) continue;
+            float* out = b.wk + ((size_t)(t0 + t) * p.heads + h) * dim;
+            if (vec)
+                store4<true>(out, d, dim, acc[i]);
+            else
+                store4<false>(out, d, dim, acc[i]);
         }
+        __syncthreads();
 #pragma unroll
-        for (int sb = 0; sb < NI; ++sb)
-#pragma unroll
-            for (int s = sb * 16; s < sb * 16 + 16; s += 4) {
-                float4 w[4];
-#pragma unroll
-                for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float4*>(sk + (s + e) * LD + d);
-#pragma unroll
-                for (int i = sb; i < NI; ++i) {
-                    const float4 a = *reinterpret_cast<const float4*>(sa + (ty + 16 * i) * LC + s);
-                    const float av[4] = {a.x, a.y, a.z, a.w};
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        acc[i][0] = fmaf(-av[e], w[e].x, acc[i][0]);
-                        acc[i][1] = fmaf(-av[e], w[e].y, acc[i][1]);
-                        acc[i][2] = fmaf(-av[e], w[e].z, acc[i][2]);
-                        acc[i][3] = fmaf(-av[e], w[e].w, acc[i][3]);
-                    }
-                }
-            }
+        for (int i = 0; i < NI; ++i) {
+            const float4 q = *reinterpret_cast<const float4*>(sq + (ty + 16 * i) * LD + (d < dim ? d : 0));
+            const float g = s_g[ty + 16 * i];
+            acc[i][0] = g * q.x;
+            acc[i][1] = g * q.y;
+            acc[i][2] = g * q.z;
+            acc[i][3] = g * q.w;
+        }
+        if (d >= dim) continue;
+        tri_mul<NI>(sa, LC, sk, LD, ty, d, acc);  // (sa holds -A)
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
             const int t = ty + 16 * i;
             if (t >= n) continue;
-            float* out = b.c.qd + ((size_t)(t0 + t) * p.heads + h) * dim + d;
+            float* out = b.c.qd + ((size_t)(t0 + t) * p.heads + h) * dim;
+            if (vec)
+                store4<true>(out, d, dim, acc[i]);
+            else
+                store4<false>(out, d, dim, acc[i]);
+        }
+    }
+    const float* v = b.qkv + (size_t)t0 * nch + 2 * QK + h * p.vdim;
+    float f[NI][4];
+    auto read = [&](int v0) {
 #pragma unroll
-            for (int e = 0; e < 4; ++e)
-                if (d + e < dim) out[e] = acc[i][e];
+        for (int i = 0; i < NI; ++i) {
+            const int t = ty + 16 * i;
+            if (t < n)
+                lb_load_cols<4>(v + (size_t)t * nch, v0 + tx * 4, p.vdim, vec, f[i]);
+            else
+                f[i][0] = f[i][1] = f[i][2] = f[i][3] = 0.f;
+        }
+    };
+    read(0);
+    for (int v0 = 0; v0 < p.vdim; v0 += kValueCols) {
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int t = ty + 16 * i;
+            const float x = s_beta[t];
+            *reinterpret_cast<float4*>(sq + t * kValueLd + tx * 4) = make_float4(f[i][0] * x, f[i][1] * x, f[i][2] * x, f[i][3] * x);
+        }
+        __syncthreads();
+        if (v0 + kValueCols < p.vdim) read(v0 + kValueCols);
+        float acc[NI][4] = {};
+        tri_mul<NI>(sl, LC, sq, kValueLd, ty, tx * 4, acc);
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int t = ty + 16 * i;
+            if (t >= n) continue;
+            float* out = b.wv + ((size_t)(t0 + t) * p.heads + h) * p.vdim;
+            if (vec)
+                store4<true>(out, v0 + tx * 4, p.vdim, acc[i]);
+            else
+                store4<false>(out, v0 + tx * 4, p.vdim, acc[i]);
         }
     }
 }
 
-// ---- the states in front of the chunks, one after the other: CTA = (16 value columns, head) ------------------------------
+// ---- the states in front of the chunks, one after the other: CTA = (a few value columns, head) ---------------------------
 //
 // S <- G S + N - M S with M = Kd^T Wk (dim x dim) and N = Kd^T Wv.  Panels of rows of M and the columns of N travel while the panel
-// before is worked on; the old and the new state are in shared memory.
-constexpr int kScanCols = 16;
-constexpr size_t kScanSmem = 200 * 1024;
+// before is worked on; the old and the new state are in shared memory.  Two halves of the threads split the sum over the old state's
+// rows; a thread has 4 x 4 of the panel's results, its rows a quarter of the panel apart (neighbouring threads, neighbouring rows).
+constexpr size_t kScanSmem = 224 * 1024;
 
 __device__ __forceinline__ void copy_async(float* dst, const float* src, bool wide) {
     if (wide)
@@ -338,123 +463,141 @@ __device__ __forceinline__ void copy_async(float* dst, const float* src, bool wi
         asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(lb_smem_u32(dst)), "l"(src) : "memory");
 }
 
-size_t scan_smem(int dim, int panel) { return ((size_t)2 * panel * lead(dim) + (size_t)4 * lb_round_up(dim, 4) * kScanCols) * sizeof(float); }
-int scan_panel(int dim) {
-    int p = 128;
-    while (p > 16 && p / 2 >= dim) p /= 2;
-    while (p > 8 && scan_smem(dim, p) > kScanSmem) p /= 2;
-    return scan_smem(dim, p) <= kScanSmem ? p : 0;
+size_t scan_smem(int dim, int panel, int cols) {
+    return ((size_t)2 * panel * lead(dim) + (size_t)4 * lb_round_up(dim, 4) * cols + (size_t)panel * cols) * sizeof(float);
+}
+struct ScanShape {
+    int panel, cols;
+};
+// as few columns as keep every SM busy once, in panels as high as fit; panel 0: does not fit
+ScanShape scan_shape(int dim, int vdim, int heads, int sms) {
+    const int per_head = sms / heads > 1 ? sms / heads : 1;
+    int cols = lb_round_up(lb_ceil_div(vdim, per_head), 4);
+    if (cols > 32) cols = 32;
+    int want = 128;
+    while (want > 16 && want / 2 >= dim) want /= 2;
+    for (; cols >= 4; cols -= 4) {
+        int panel = want;
+        while (panel > 8 && scan_smem(dim, panel, cols) > kScanSmem) panel /= 2;
+        if (scan_smem(dim, panel, cols) > kScanSmem) continue;
+        if (panel >= 32 || panel == want || cols == 4) return {panel, cols};
+    }
+    return {0, 0};
 }
 
-__global__ void __launch_bounds__(256) lb_delta_scan_kernel(const LbDeltaBlock b, int chunks, int panel, int fresh, bool wide_m, bool wide_n) {
+__global__ void __launch_bounds__(512) lb_delta_scan_kernel(const LbDeltaBlock b, int chunks, int panel, int cols, int fresh, bool wide_m, bool wide_n) {
     extern __shared__ __align__(16) float sm[];
     const LbChunks& c = b.c;
-    const int dim = c.dim, vdim = c.vdim, LD = lead(dim), DP = lb_round_up(dim, 4), tid = threadIdx.x, h = blockIdx.y, v0 = blockIdx.x * kScanCols;
-    float *sM = sm, *sN = sM + 2 * panel * LD, *sS = sN + 2 * DP * kScanCols;
-    const int panels = lb_ceil_div(dim, panel), steps = chunks * panels, cols = min(kScanCols, vdim - v0);
-    for (int i = tid; i < 2 * panel * LD + 4 * DP * kScanCols; i += 256) sm[i] = 0.f;
+    const int dim = c.dim, vdim = c.vdim, LD = lead(dim), DP = lb_round_up(dim, 4), tid = threadIdx.x, nt = blockDim.x, h = blockIdx.y, v0 = blockIdx.x * cols;
+    float *sM = sm, *sN = sM + 2 * panel * LD, *sS = sN + 2 * DP * cols, *red = sS + 2 * DP * cols;
+    const int panels = lb_ceil_div(dim, panel), steps = chunks * panels, live = min(cols, vdim - v0);
+    for (int i = tid; i < 2 * panel * LD + (4 * DP + panel) * cols; i += nt) sm[i] = 0.f;
     __syncthreads();
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     float* S0 = c.state + (size_t)h * dim * vdim + v0;
     if (!fresh)
-        for (int i = tid; i < dim * kScanCols; i += 256) {
-            const int d = i / kScanCols, v = i % kScanCols;
-            if (v < cols) sS[i] = S0[(size_t)d * vdim + v];
+        for (int i = tid; i < dim * cols; i += nt) {
+            const int d = i / cols, v = i % cols;
+            if (v < live) sS[i] = S0[(size_t)d * vdim + v];
         }
+    const int qm = wide_m ? 4 : 1, per = dim / qm, qn = wide_n ? 4 : 1, pn = live / qn;
     auto fetch = [&](int step) {
         const int cc = step / panels, d0 = (step - cc * panels) * panel, rows = min(panel, dim - d0);
         const float* M = b.mix + (((size_t)cc * c.heads + h) * dim + d0) * dim;
         float* dst = sM + (step & 1) * panel * LD;
-        const int q = wide_m ? 4 : 1, per = dim / q;
-        for (int i = tid; i < rows * per; i += 256) {
-            const int r = i / per, e = (i - r * per) * q;
+        for (int i = tid; i < rows * per; i += nt) {
+            const int r = i / per, e = (i - r * per) * qm;
             copy_async(dst + r * LD + e, M + (size_t)r * dim + e, wide_m);
         }
         if (d0 == 0) {
             const float* N = c.states + ((size_t)cc * c.heads + h) * dim * vdim + v0;
-            float* to = sN + (cc & 1) * DP * kScanCols;
-            const int qn = wide_n ? 4 : 1, pn = cols / qn;
-            for (int i = tid; i < dim * pn; i += 256) {
+            float* to = sN + (cc & 1) * DP * cols;
+            for (int i = tid; i < dim * pn; i += nt) {
                 const int d = i / pn, v = (i - d * pn) * qn;
-                copy_async(to + d * kScanCols + v, N + (size_t)d * vdim + v, wide_n);
+                copy_async(to + d * cols + v, N + (size_t)d * vdim + v, wide_n);
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
+    const int RG = panel / 4, CG = cols / 4, items = RG * CG, half = tid / items, item = tid - half * items, rg = item / CG, v = (item - rg * CG) * 4;
+    const int split = DP / 8 * 4, e0 = half == 0 ? 0 : split, e1 = half == 0 ? split : DP;
     fetch(0);
     for (int step = 0; step < steps; ++step) {
-        const int cc = step / panels, d0 = (step - cc * panels) * panel, rows = min(panel, dim - d0);
+        const int cc = step / panels, d0 = (step - cc * panels) * panel;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // the panel is here, and everyone is done with the other buffer
         if (step + 1 < steps) fetch(step + 1);
-        const float *S = sS + (cc & 1) * DP * kScanCols, *N = sN + (cc & 1) * DP * kScanCols, *M = sM + (step & 1) * panel * LD;
-        float* next = sS + ((cc + 1) & 1) * DP * kScanCols;
-        const float g = c.decay[(size_t)cc * c.heads + h];
-        float* out = c.states + ((size_t)cc * c.heads + h) * dim * vdim + v0;
-        for (int i = tid; i < (panel / 2) * 4; i += 256) {
-            const int r = (i >> 2) * 2, v = (i & 3) * 4;
-            if (r >= rows) continue;
-            const float *m0 = M + r * LD, *m1 = m0 + LD;  // (a row behind the last one holds finite leftovers and is not stored)
-            float a0[4] = {}, a1[4] = {};
-#pragma unroll 4
-            for (int e = 0; e < DP; e += 4) {
-                const float4 x = *reinterpret_cast<const float4*>(m0 + e), y = *reinterpret_cast<const float4*>(m1 + e);
-                const float xv[4] = {x.x, x.y, x.z, x.w}, yv[4] = {y.x, y.y, y.z, y.w};
+        const float *S = sS + (cc & 1) * DP * cols, *N = sN + (cc & 1) * DP * cols, *M = sM + (step & 1) * panel * LD + rg * LD;
+        float acc[4][4] = {};
+        if (half < 2) {
+#pragma unroll 2
+            for (int e = e0; e < e1; e += 4) {  // (rows behind the panel's last one hold finite leftovers and are not stored)
+                float4 m[4], s[4];
 #pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    const float4 s = *reinterpret_cast<const float4*>(S + (e + k) * kScanCols + v);
-                    a0[0] = fmaf(xv[k], s.x, a0[0]);
-                    a0[1] = fmaf(xv[k], s.y, a0[1]);
-                    a0[2] = fmaf(xv[k], s.z, a0[2]);
-                    a0[3] = fmaf(xv[k], s.w, a0[3]);
-                    a1[0] = fmaf(yv[k], s.x, a1[0]);
-                    a1[1] = fmaf(yv[k], s.y, a1[1]);
-                    a1[2] = fmaf(yv[k], s.z, a1[2]);
-                    a1[3] = fmaf(yv[k], s.w, a1[3]);
-                }
-            }
+                for (int i = 0; i < 4; ++i) m[i] = *reinterpret_cast<const float4*>(M + i * RG * LD + e);
 #pragma unroll
-            for (int rr = 0; rr < 2; ++rr) {
-                const int d = d0 + r + rr;
-                if (r + rr >= rows) continue;
-                float old[4];
+                for (int k = 0; k < 4; ++k) s[k] = *reinterpret_cast<const float4*>(S + (e + k) * cols + v);
 #pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    old[k] = S[d * kScanCols + v + k];
-                    next[d * kScanCols + v + k] = fmaf(g, old[k], N[d * kScanCols + v + k] - (rr ? a1[k] : a0[k]));
-                }
-                if (wide_n && v + 4 <= cols) {
-                    *reinterpret_cast<float4*>(out + (size_t)d * vdim + v) = make_float4(old[0], old[1], old[2], old[3]);
-                } else {
+                for (int i = 0; i < 4; ++i) {
+                    const float mv[4] = {m[i].x, m[i].y, m[i].z, m[i].w};
 #pragma unroll
-                    for (int k = 0; k < 4; ++k)
-                        if (v + k < cols) out[(size_t)d * vdim + v + k] = old[k];
+                    for (int k = 0; k < 4; ++k) {
+                        acc[i][0] = fmaf(mv[k], s[k].x, acc[i][0]);
+                        acc[i][1] = fmaf(mv[k], s[k].y, acc[i][1]);
+                        acc[i][2] = fmaf(mv[k], s[k].z, acc[i][2]);
+                        acc[i][3] = fmaf(mv[k], s[k].w, acc[i][3]);
+                    }
                 }
             }
         }
+        if (half == 1)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + (rg + i * RG) * cols + v) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+        __syncthreads();
+        if (half != 0) continue;
+        const float g = c.decay[(size_t)cc * c.heads + h];
+        float* next = sS + ((cc + 1) & 1) * DP * cols;
+        float* out = c.states + ((size_t)cc * c.heads + h) * dim * vdim + v0;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int r = rg + i * RG, d = d0 + r;
+            if (d >= dim) continue;
+            const float4 x = *reinterpret_cast<const float4*>(red + r * cols + v), old = *reinterpret_cast<const float4*>(S + d * cols + v),
+                         add = *reinterpret_cast<const float4*>(N + d * cols + v);
+            *reinterpret_cast<float4*>(next + d * cols + v) = make_float4(fmaf(g, old.x, add.x - (acc[i][0] + x.x)), fmaf(g, old.y, add.y - (acc[i][1] + x.y)),
+                                                                          fmaf(g, old.z, add.z - (acc[i][2] + x.z)), fmaf(g, old.w, add.w - (acc[i][3] + x.w)));
+            const float o[4] = {old.x, old.y, old.z, old.w};
+            if (wide_n)
+                store4<true>(out + (size_t)d * vdim, v, live, o);
+            else
+                store4<false>(out + (size_t)d * vdim, v, live, o);
+        }
     }
     __syncthreads();
-    const float* last = sS + (chunks & 1) * DP * kScanCols;
-    for (int i = tid; i < dim * kScanCols; i += 256) {
-        const int d = i / kScanCols, v = i % kScanCols;
-        if (v < cols) S0[(size_t)d * vdim + v] = last[i];
+    const float* last = sS + (chunks & 1) * DP * cols;
+    for (int i = tid; i < dim * cols; i += nt) {
+        const int d = i / cols, x = i % cols;
+        if (x < live) S0[(size_t)d * vdim + x] = last[i];
     }
 }
 
-size_t prep_smem(int C, int dim) { return ((size_t)2 * C * lead(dim) + (size_t)2 * C * (C + 4)) * sizeof(float); }
+size_t prep_smem(int C, int dim) {
+    const size_t q = lead(dim) > kValueLd ? lead(dim) : kValueLd;
+    return ((size_t)C * lead(dim) + (size_t)C * q + (size_t)2 * C * (C + 4) + (size_t)C * C / 4) * sizeof(float);
+}
 
 template <int C>
-int launch_prep(loom_b200_ctx* ctx, const LbDelta& p, const LbDeltaBlock& b, int T) {
+int launch_prep(loom_b200_ctx* ctx, const LbDelta& p, const LbDeltaBlock& b, int T, bool vec) {
     LB_BIG_SMEM(ctx, lb_delta_prep_kernel<C>, 200 * 1024);
-    LB_LAUNCH(ctx, lb_delta_prep_kernel<C>, dim3(lb_ceil_div(T, C), p.heads), dim3(256), prep_smem(C, p.dim), p, b, T);
+    LB_LAUNCH(ctx, lb_delta_prep_kernel<C>, dim3(lb_ceil_div(T, C), p.heads), dim3(256), prep_smem(C, p.dim), p, b, T, vec);
     return 0;
 }
 
 }  // namespace
 
 int lb_delta_chunk(int dim) {
-    if (!scan_panel(dim)) return 0;
+    if (!scan_shape(dim, 4, 1, 148).panel) return 0;
     for (int C = 64; C >= 16; C /= 2)
         if (prep_smem(C, dim) <= 200 * 1024) return C;
     return 0;
@@ -480,9 +623,14 @@ int lb_delta_block(loom_b200_ctx* ctx, const LbDelta& p, const LbDeltaBlock& bin
     b.c.o = p.o;
     b.c.ldo = p.ldo;
     const int chunks = lb_ceil_div(T, b.c.C);
-    LB_LAUNCH(ctx, lb_delta_tokens_kernel, dim3(lb_ceil_div(T, kRows)), dim3(256), 0, p, b, T, pos0);
+    const bool vec = p.dim % 4 == 0 && p.vdim % 4 == 0 && lb_vec_rows(p.proj, p.ldp);
+    const dim3 tokens(lb_ceil_div(T, kRows), 2 * p.kv_heads + p.heads + 1);
+    if (vec)
+        LB_LAUNCH(ctx, lb_delta_tokens_kernel<true>, tokens, dim3(256), 0, p, b, T, pos0);
+    else
+        LB_LAUNCH(ctx, lb_delta_tokens_kernel<false>, tokens, dim3(256), 0, p, b, T, pos0);
     if (p.taps > 1) LB_LAUNCH(ctx, lb_delta_commit_kernel, dim3(lb_ceil_div(lb_delta_channels(p), 256), p.taps - 1), dim3(256), 0, p, T, pos0);
-    int rc = b.c.C == 64 ? launch_prep<64>(ctx, p, b, T) : b.c.C == 32 ? launch_prep<32>(ctx, p, b, T) : launch_prep<16>(ctx, p, b, T);
+    int rc = b.c.C == 64 ? launch_prep<64>(ctx, p, b, T, vec) : b.c.C == 32 ? launch_prep<32>(ctx, p, b, T, vec) : launch_prep<16>(ctx, p, b, T, vec);
     if (rc) return rc;
     if ((rc = lb_chunk_states(ctx, b.c, T))) return rc;
     LbChunks m = b.c;  // what a chunk takes out of the state
@@ -491,9 +639,10 @@ int lb_delta_block(loom_b200_ctx* ctx, const LbDelta& p, const LbDeltaBlock& bin
     m.ldv = p.heads * p.dim;
     m.states = b.mix;
     if ((rc = lb_chunk_states(ctx, m, T))) return rc;
-    const int panel = scan_panel(p.dim);
+    const ScanShape sh = scan_shape(p.dim, p.vdim, p.heads, ctx->sm_count);
+    const int threads = lb_round_up(2 * (sh.panel / 4) * (sh.cols / 4), 32);
     LB_BIG_SMEM(ctx, lb_delta_scan_kernel, kScanSmem);
-    LB_LAUNCH(ctx, lb_delta_scan_kernel, dim3(lb_ceil_div(p.vdim, kScanCols), p.heads), dim3(256), scan_smem(p.dim, panel), b, chunks, panel, pos0 == 0 ? 1 : 0,
-              p.dim % 4 == 0, p.vdim % 4 == 0);
+    LB_LAUNCH(ctx, lb_delta_scan_kernel, dim3(lb_ceil_div(p.vdim, sh.cols), p.heads), dim3(threads), scan_smem(p.dim, sh.panel, sh.cols), b, chunks, sh.panel, sh.cols,
+              pos0 == 0 ? 1 : 0, p.dim % 4 == 0, p.vdim % 4 == 0);
     return lb_chunk_out(ctx, b.c, T);
 }

@@ -92,40 +92,52 @@ struct Run {
 };
 __device__ __forceinline__ Run join(const Run& a, const Run& b) { return {a.F + b.F, fmaxf((float)(a.M + b.F), b.M)}; }
 
+// log gates of every token, [heads][T]
+__global__ void __launch_bounds__(256) lb_memory_gates_kernel(const LbMemory p, const LbMemoryBlock b, int T) {
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int i = blockIdx.x * 256 + threadIdx.x;
+    if (i >= T * p.heads) return;
+    const int t = i / p.heads, h = i - t * p.heads;
+    float gi, gf;
+    gates(p, p.proj + (size_t)t * p.ldp, h, gi, gf);
+    b.gate_i[(size_t)h * T + t] = gi;
+    b.gate_f[(size_t)h * T + t] = gf;
+}
+
 // CTA = (chunk, head): maxima, weights, and the operands of the products over chunks
 template <int C>
-__global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p, const LbMemoryBlock b, int T, int pos0) {
+__global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p, const LbMemoryBlock b, int T, int pos0, bool vec) {
     extern __shared__ __align__(16) float sm[];
     __shared__ Run s_run[8];
     __shared__ double s_F[C];
-    __shared__ float s_i[C], s_f[C], s_m[C], s_keep[C], s_m0;
+    __shared__ float s_i[C], s_f[C], s_m[C], s_keep[C], s_end[C], s_m0;
     constexpr int NI = C / 16, LC = C + 4;
     const int ch = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, dim = p.dim, LD = lead(dim);
-    const int HD = p.heads * dim, t0 = ch * C, n = min(C, T - t0);
+    const int HD = p.heads * dim, t0 = ch * C, n = min(C, T - t0), D4 = lb_round_up(dim, 4) / 4;
     float *sq = sm, *sk = sq + C * LD, *sa = sk + C * LD;
     lb_pdl_launch_dependents();
     lb_pdl_wait();
-    for (int i = tid; i < C * LD; i += 256) {
-        const int t = i / LD, d = i - t * LD;
-        const bool ok = t < n && d < dim;
-        const float* row = p.proj + (size_t)(t0 + t) * p.ldp + h * dim + d;
-        sq[i] = ok ? row[0] * p.qscale : 0.f;
-        sk[i] = ok ? row[HD] : 0.f;
+    const float *gi = b.gate_i + (size_t)h * T, *gf = b.gate_f + (size_t)h * T;
+    for (int i = tid; i < C * D4; i += 256) {
+        const int t = i / D4, d = (i - t * D4) * 4;
+        float q[4] = {0.f, 0.f, 0.f, 0.f}, k[4] = {0.f, 0.f, 0.f, 0.f};
+        if (t < n) {
+            const float* row = p.proj + (size_t)(t0 + t) * p.ldp + h * dim;
+            lb_load_cols<4>(row, d, dim, vec, q);
+            lb_load_cols<4>(row + HD, d, dim, vec, k);
+        }
+        *reinterpret_cast<float4*>(sq + t * LD + d) = make_float4(q[0] * p.qscale, q[1] * p.qscale, q[2] * p.qscale, q[3] * p.qscale);
+        *reinterpret_cast<float4*>(sk + t * LD + d) = make_float4(k[0], k[1], k[2], k[3]);
     }
     if (tid < C) {
-        float gi = -INFINITY, gf = 0.f;
-        if (tid < n) gates(p, p.proj + (size_t)(t0 + tid) * p.ldp, h, gi, gf);
-        s_i[tid] = gi;
-        s_f[tid] = gf;
+        s_i[tid] = tid < n ? gi[t0 + tid] : -INFINITY;
+        s_f[tid] = tid < n ? gf[t0 + tid] : 0.f;
     }
     {
         const int per = lb_ceil_div(t0, 256);
         Run r = {0.0, -INFINITY};
-        for (int t = tid * per; t < min(t0, (tid + 1) * per); ++t) {
-            float gi, gf;
-            gates(p, p.proj + (size_t)t * p.ldp, h, gi, gf);
-            r = join(r, {(double)gf, gi});
-        }
+        for (int t = tid * per; t < min(t0, (tid + 1) * per); ++t) r = join(r, {(double)gf[t], gi[t]});
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const Run right = {__shfl_down_sync(0xffffffffu, r.F, o), __shfl_down_sync(0xffffffffu, r.M, o)};
@@ -151,6 +163,7 @@ __global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p
     __syncthreads();
     if (tid < C) {
         s_keep[tid] = expf((float)(s_F[tid] + s_m0 - s_m[tid]));
+        s_end[tid] = expf((float)(s_F[C - 1] - s_F[tid] + s_i[tid] - s_m[C - 1]));
         if (tid < n) b.tops[(size_t)(t0 + tid) * p.heads + h] = s_m[tid];
     }
     {
@@ -187,19 +200,31 @@ __global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p
         s = lb_warp_sumf(s);
         if (lane == 0) b.sums[(size_t)(t0 + t) * p.heads + h] = s;
     }
-    // keys decayed to the chunk's end and their sum, queries decayed from its start: a thread per channel and part of the tokens
-    const float end = s_m[C - 1], over = s_keep[C - 1];
-    for (int i = tid; i < n * dim; i += 256) {
-        const int t = i / dim, d = i - t * dim;
-        const size_t at = (size_t)(t0 + t) * HD + h * dim + d;
-        const float kd = sk[t * LD + d] * expf((float)(s_F[C - 1] - s_F[t] + s_i[t] - end));
-        b.c.qd[at] = sq[t * LD + d] * s_keep[t];
-        b.c.kd[at] = kd;
-        sk[t * LD + d] = kd;
+    // keys decayed to the chunk's end, queries decayed from its start
+    const float over = s_keep[C - 1];
+    for (int i = tid; i < n * D4; i += 256) {
+        const int t = i / D4, d = (i - t * D4) * 4;
+        const float e = s_end[t], g = s_keep[t];
+        const float4 q = *reinterpret_cast<const float4*>(sq + t * LD + d), k = *reinterpret_cast<const float4*>(sk + t * LD + d);
+        const float qd[4] = {q.x * g, q.y * g, q.z * g, q.w * g}, kd[4] = {k.x * e, k.y * e, k.z * e, k.w * e};
+        const size_t at = (size_t)(t0 + t) * HD + h * dim;
+        *reinterpret_cast<float4*>(sk + t * LD + d) = make_float4(kd[0], kd[1], kd[2], kd[3]);
+        if (vec) {
+            *reinterpret_cast<float4*>(b.c.qd + at + d) = make_float4(qd[0], qd[1], qd[2], qd[3]);
+            *reinterpret_cast<float4*>(b.c.kd + at + d) = make_float4(kd[0], kd[1], kd[2], kd[3]);
+        } else {
+#pragma unroll
+            for (int x = 0; x < 4; ++x)
+                if (d + x < dim) {
+                    b.c.qd[at + d + x] = qd[x];
+                    b.c.kd[at + d + x] = kd[x];
+                }
+        }
     }
     __syncthreads();
     for (int d = tid; d < dim; d += 256) {
         float s = 0.f;
+#pragma unroll 8
         for (int t = 0; t < n; ++t) s += sk[t * LD + d];
         const size_t at = ((size_t)ch * p.heads + h) * dim + d;
         b.norms[at] = s;
@@ -252,7 +277,8 @@ size_t prep_smem(int C, int dim) { return ((size_t)2 * C * lead(dim) + (size_t)C
 template <int C>
 int launch_prep(loom_b200_ctx* ctx, const LbMemory& p, const LbMemoryBlock& b, int T, int pos0) {
     LB_BIG_SMEM(ctx, lb_memory_prep_kernel<C>, 200 * 1024);
-    LB_LAUNCH(ctx, lb_memory_prep_kernel<C>, dim3(lb_ceil_div(T, C), p.heads), dim3(256), prep_smem(C, p.dim), p, b, T, pos0);
+    const bool vec = p.dim % 4 == 0 && lb_vec_rows(p.proj, p.ldp);
+    LB_LAUNCH(ctx, lb_memory_prep_kernel<C>, dim3(lb_ceil_div(T, C), p.heads), dim3(256), prep_smem(C, p.dim), p, b, T, pos0, vec);
     return 0;
 }
 
@@ -284,6 +310,7 @@ int lb_memory_block(loom_b200_ctx* ctx, const LbMemory& p, const LbMemoryBlock& 
     b.c.o = p.o;
     b.c.ldo = p.ldo;
     const int chunks = lb_ceil_div(T, b.c.C);
+    LB_LAUNCH(ctx, lb_memory_gates_kernel, dim3(lb_ceil_div(T * p.heads, 256)), dim3(256), 0, p, b, T);
     int rc = b.c.C == 64 ? launch_prep<64>(ctx, p, b, T, pos0) : b.c.C == 32 ? launch_prep<32>(ctx, p, b, T, pos0) : launch_prep<16>(ctx, p, b, T, pos0);
     if (rc) return rc;
     if ((rc = lb_chunk_states(ctx, b.c, T))) return rc;

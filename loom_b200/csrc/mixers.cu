@@ -36,9 +36,14 @@ __global__ void __launch_bounds__(256) lb_embed_image_kernel(const uint8_t* __re
     for (int c = threadIdx.x; c < slices * 8; c += blockDim.x) {
         float f[C];
         lb_unpack_chunk<WT>(*reinterpret_cast<const uint4*>(img + lb_img_chunk(ok ? t : 0, c, slices)), f);
+        if ((c + 1) * C <= width) {  // (rows of x are padded to eight columns)
 #pragma unroll
-        for (int e = 0; e < C; ++e)
-            if (c * C + e < width) out[c * C + e] = ok ? f[e] : 0.f;
+            for (int e = 0; e < C; e += 4) *reinterpret_cast<float4*>(out + c * C + e) = ok ? make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]) : make_float4(0.f, 0.f, 0.f, 0.f);
+        } else {
+#pragma unroll
+            for (int e = 0; e < C; ++e)
+                if (c * C + e < width) out[c * C + e] = ok ? f[e] : 0.f;
+        }
     }
 }
 
@@ -53,15 +58,15 @@ __device__ __forceinline__ float row_rstd(const float* row, int width, float eps
 }
 
 template <typename WT>
-__global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p, bool vec) {
+__global__ void __launch_bounds__(256) lb_norm_conv_kernel(const LbNormBlock p, bool vec) {
     constexpr int C = LbElem<WT>::kChunk;
     __shared__ float s_r[kNormTokens + kMaxTaps];
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * kNormTokens, t1 = min(p.T, t0 + kNormTokens);
-    const int back = p.conv_w ? p.taps - 1 : 0;
-    const float gain = p.gain ? *p.gain : 1.f;
+    const int back = p.taps - 1;
+    const float gain = *p.gain;
     for (int i = warp; i < t1 - t0 + back; i += 8) {
         const int t = t0 - back + i;
         if (t < 0) continue;
@@ -78,18 +83,7 @@ __global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p,
         lb_load_cols<C>(p.x + (size_t)src * p.ldx, k0, p.width, vec, f);
 #pragma unroll
         for (int e = 0; e < C; ++e) f[e] *= s_r[tt + back];
-        if (p.gain_w) {
-            float w[C];
-            lb_load_cols<C>(p.gain_w, k0, p.width, vec, w);
-#pragma unroll
-            for (int e = 0; e < C; ++e) f[e] *= w[e];
-        }
-        if (p.rows) {
-#pragma unroll
-            for (int e = 0; e < C; ++e)
-                if (k0 + e < p.width) p.rows[(size_t)t * p.ldx + k0 + e] = f[e];
-        }
-        if (p.conv_w && k0 < p.width) {
+        if (k0 < p.width) {
             float a[C], w[C], h[C];
 #pragma unroll
             for (int e = 0; e < C; ++e) a[e] = 0.f;
@@ -110,7 +104,62 @@ __global__ void __launch_bounds__(256) lb_norm_block_kernel(const LbNormBlock p,
 #pragma unroll
             for (int e = 0; e < C; ++e) f[e] += a[e];
         }
-        if (p.img) *reinterpret_cast<uint4*>(p.img + lb_img_chunk(t, c, p.slices)) = lb_pack_chunk<WT>(f);
+        *reinterpret_cast<uint4*>(p.img + lb_img_chunk(t, c, p.slices)) = lb_pack_chunk<WT>(f);
+    }
+}
+
+// the same without a convolution, a CTA per token with the row in registers as far as it fits
+template <typename WT>
+__global__ void __launch_bounds__(256) lb_norm_row_kernel(const LbNormBlock p, bool vec) {
+    constexpr int C = LbElem<WT>::kChunk, KEEP = 32 / C;
+    __shared__ float red[8];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int t = blockIdx.x, chunks = p.slices * 8;
+    const float* row = p.x + (size_t)(p.row_idx ? p.row_idx[t] : t) * p.ldx;
+    float f[KEEP][C], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < chunks) lb_load_cols<C>(row, c * C, p.width, vec, f[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if ((int)threadIdx.x + i * 256 < chunks)
+#pragma unroll
+            for (int e = 0; e < C; ++e) ss = fmaf(f[i][e], f[i][e], ss);
+    for (int k = KEEP * 256 * C + (int)threadIdx.x; k < p.width; k += 256) ss = fmaf(row[k], row[k], ss);
+    ss = lb_block_sumf(ss, red);
+    const float r = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)p.width), p.eps))) * (p.gain ? *p.gain : 1.f);
+    auto finish = [&](int c, float* g) {
+#pragma unroll
+        for (int e = 0; e < C; ++e) g[e] *= r;
+        if (p.gain_w) {
+            float w[C];
+            lb_load_cols<C>(p.gain_w, c * C, p.width, vec, w);
+#pragma unroll
+            for (int e = 0; e < C; ++e) g[e] *= w[e];
+        }
+        if (p.rows) {
+            float* out = p.rows + (size_t)t * p.ldx + c * C;
+            if (vec && (c + 1) * C <= p.width) {
+#pragma unroll
+                for (int e = 0; e < C; e += 4) *reinterpret_cast<float4*>(out + e) = make_float4(g[e], g[e + 1], g[e + 2], g[e + 3]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < C; ++e)
+                    if (c * C + e < p.width) out[e] = g[e];
+            }
+        }
+        if (p.img) *reinterpret_cast<uint4*>(p.img + lb_img_chunk(t, c, p.slices)) = lb_pack_chunk<WT>(g);
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if ((int)threadIdx.x + i * 256 < chunks) finish(threadIdx.x + i * 256, f[i]);
+    for (int c = threadIdx.x + KEEP * 256; c < chunks; c += 256) {
+        float g[C];
+        lb_load_cols<C>(row, c * C, p.width, vec, g);
+        finish(c, g);
     }
 }
 
@@ -479,8 +528,13 @@ int lb_embed_image(loom_b200_ctx* ctx, int dtype, const uint8_t* img, int slices
 
 int lb_norm_block(loom_b200_ctx* ctx, int dtype, const LbNormBlock& p) {
     LB_REQUIRE(ctx, p.taps >= 1 && p.taps <= kMaxTaps, "norm_block: %d taps (1..%d)", p.taps, kMaxTaps);
-    LB_TYPED(dtype, lb_norm_block_kernel<float>, lb_norm_block_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.T, kNormTokens)), dim3(256), 0, p,
-             lb_vec_rows(p.x, p.ldx) && (!p.gain_w || lb_vec_rows(p.gain_w, 4)) && (!p.conv_w || (lb_vec_rows(p.conv_w, p.ring_ld) && lb_vec_rows(p.ring, p.ring_ld))));
+    if (!p.conv_w) {
+        LB_TYPED(dtype, lb_norm_row_kernel<float>, lb_norm_row_kernel<__nv_bfloat16>, dim3(p.T), dim3(256), 0, p,
+                 lb_vec_rows(p.x, p.ldx) && (!p.gain_w || lb_vec_rows(p.gain_w, 4)) && (!p.rows || lb_vec_rows(p.rows, p.ldx)));
+        return 0;
+    }
+    LB_TYPED(dtype, lb_norm_conv_kernel<float>, lb_norm_conv_kernel<__nv_bfloat16>, dim3(lb_ceil_div(p.T, kNormTokens)), dim3(256), 0, p,
+             lb_vec_rows(p.x, p.ldx) && lb_vec_rows(p.conv_w, p.ring_ld) && lb_vec_rows(p.ring, p.ring_ld));
     return 0;
 }
 

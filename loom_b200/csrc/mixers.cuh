@@ -120,6 +120,7 @@ struct LbMemoryBlock {
     float* norms = nullptr;       // [chunks, heads, dim] what a chunk adds to the normaliser, then the normaliser in front of it
     float* sums = nullptr;        // [T, heads] sums of a token's weights inside its chunk
     float* tops = nullptr;        // [T, heads] running maximum
+    float *gate_i = nullptr, *gate_f = nullptr;  // [heads, T] log gates
     float* scale = nullptr;       // [T, heads] out: what the outputs still have to be multiplied by
 };
 // T tokens of one sequence (state, norm and top are its own)

@@ -30,57 +30,64 @@ __device__ __forceinline__ size_t value_at(int g, int v, int vrows, int row, int
     return lb_img_chunk(g * vrows + v, row / C, slices) + (size_t)(row % C) * sizeof(WT);
 }
 
-// A CTA takes the tokens of eight aligned positions: a warp per token for queries and keys, then a thread per value row.
+// Queries (per-head blocks for the tensor-core kernel) and keys: a warp per (token, head), heads in blockIdx.y.  Values: the last rows
+// of CTAs, a thread per value row and eight aligned positions.
 template <typename WT>
-__global__ void __launch_bounds__(256) lb_attention_store_kernel(const LbAttention p, int T, int kchunks, int qchunks, uint8_t* __restrict__ q_img, bool vec) {
+__global__ void __launch_bounds__(256) lb_attention_store_kernel(const LbAttention p, int T, int kchunks, int qchunks, uint8_t* __restrict__ q_img, int rows, bool vec) {
     constexpr int C = LbElem<WT>::kChunk;
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, first = (p.pos0 & ~7) + (int)blockIdx.x * 8;
     const int QD = p.heads * p.dim, KD = p.kv_heads * p.dim, vrows = vrows_of(p.vdim);
-    uint8_t *kc = p.k + (size_t)p.lane0 * p.k_lane, *vc = p.vt + (size_t)p.lane0 * p.vt_lane;
-    const int pos = first + warp, t = pos - p.pos0;
-    if (t >= 0 && t < T) {
-        const float* row = p.proj + (size_t)t * p.ldp;
+    if ((int)blockIdx.y < rows) {
+        const int i = (int)blockIdx.y + (q_img ? 0 : p.heads), pos = first + warp, t = pos - p.pos0;
+        if (t < 0 || t >= T) return;
+        const bool key = i >= p.heads;
+        const int h = key ? i - p.heads : i;
+        const float* x = p.proj + (size_t)t * p.ldp + (key ? QD + h * p.dim : h * p.dim);
+        constexpr int KEEP = 8;  // columns of a lane that stay in registers: a pair of float4 for 256 channels
+        float f[KEEP], by = 1.f;
+        const int c0 = lane * KEEP;
+        lb_load_cols<KEEP>(x, c0, p.dim, vec, f);  // (zero behind the last channel)
+        if (p.qk_norm) {
+            float ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < KEEP; ++e) ss = fmaf(f[e], f[e], ss);
+            for (int d = 32 * KEEP + lane; d < p.dim; d += 32) ss = fmaf(x[d], x[d], ss);
+            ss = lb_warp_sumf(ss);
+            by = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)p.dim), p.eps)));
+        }
+        uint8_t* kc = p.k + (size_t)p.lane0 * p.k_lane;
         const int r = pos % p.ring;
-        for (int i = q_img ? 0 : p.heads; i < p.heads + p.kv_heads; ++i) {
-            const bool key = i >= p.heads;
-            const int h = key ? i - p.heads : i, chunks = key ? kchunks : qchunks;
-            const float* x = row + (key ? QD + h * p.dim : h * p.dim);
-            const float by = p.qk_norm ? head_rstd(x, p.dim, p.eps, lane) : 1.f;
+        for (int c = c0;; c += 32 * KEEP) {
+#pragma unroll
+            for (int e = 0; e < KEEP; ++e) f[e] *= by;
             if (key) {
-                for (int c = lane; c < chunks; c += 32) {
-                    float f[C];
-                    lb_load_cols<C>(x, c * C, p.dim, vec, f);
 #pragma unroll
-                    for (int e = 0; e < C; ++e) f[e] *= by;
-                    *reinterpret_cast<uint4*>(kc + key_chunk(r, h, p.kv_heads, kchunks, c)) = lb_pack_chunk<WT>(f);
-                }
-            } else {
-                for (int c = lane; c < chunks; c += 32) {
-                    float f[8];
-                    lb_load_cols<8>(x, c * 8, p.dim, vec, f);
-#pragma unroll
-                    for (int e = 0; e < 8; ++e) f[e] *= by;
-                    *reinterpret_cast<uint4*>(q_img + key_chunk(t, h, p.heads, chunks, c)) = lb_pack_chunk<__nv_bfloat16>(f);
-                }
+                for (int e = 0; e < KEEP; e += C)
+                    if ((c + e) / C < kchunks) *reinterpret_cast<uint4*>(kc + key_chunk(r, h, p.kv_heads, kchunks, (c + e) / C)) = lb_pack_chunk<WT>(f + e);
+            } else if (c / 8 < qchunks) {
+                *reinterpret_cast<uint4*>(q_img + key_chunk(t, h, p.heads, qchunks, c / 8)) = lb_pack_chunk<__nv_bfloat16>(f);
             }
+            if (c + 32 * KEEP >= lb_round_up(p.dim, 16)) break;
+            lb_load_cols<KEEP>(x, c + 32 * KEEP, p.dim, vec, f);
         }
+        return;
     }
-    const int t0 = first - p.pos0, r0 = first % p.ring;
-    for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += 256) {
-        const int g = i / p.vdim, v = i - g * p.vdim;
-        float f[8];
+    uint8_t* vc = p.vt + (size_t)p.lane0 * p.vt_lane;
+    const int t0 = first - p.pos0, r0 = first % p.ring, i = ((int)blockIdx.y - rows) * 256 + threadIdx.x;
+    if (i >= p.kv_heads * p.vdim) return;
+    const int g = i / p.vdim, v = i - g * p.vdim;
+    float f[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[e] = t0 + e >= 0 && t0 + e < T ? p.proj[(size_t)(t0 + e) * p.ldp + QD + KD + i] : 0.f;
-        if (t0 >= 0 && t0 + 8 <= T) {
+    for (int e = 0; e < 8; ++e) f[e] = t0 + e >= 0 && t0 + e < T ? p.proj[(size_t)(t0 + e) * p.ldp + QD + KD + i] : 0.f;
+    if (t0 >= 0 && t0 + 8 <= T) {
 #pragma unroll
-            for (int e = 0; e < 8; e += C) *reinterpret_cast<uint4*>(vc + lb_img_chunk(g * vrows + v, (r0 + e) / C, p.slices)) = lb_pack_chunk<WT>(f + e);
-        } else {  // the eight positions hold tokens of other calls too
+        for (int e = 0; e < 8; e += C) *reinterpret_cast<uint4*>(vc + lb_img_chunk(g * vrows + v, (r0 + e) / C, p.slices)) = lb_pack_chunk<WT>(f + e);
+    } else {  // the eight positions hold tokens of other calls too
 #pragma unroll
-            for (int e = 0; e < 8; ++e)
-                if (t0 + e >= 0 && t0 + e < T) *reinterpret_cast<WT*>(vc + value_at<WT>(g, v, vrows, r0 + e, p.slices)) = (WT)f[e];
-        }
+        for (int e = 0; e < 8; ++e)
+            if (t0 + e >= 0 && t0 + e < T) *reinterpret_cast<WT*>(vc + value_at<WT>(g, v, vrows, r0 + e, p.slices)) = (WT)f[e];
     }
 }
 
@@ -341,12 +348,13 @@ size_t lb_attention_q_bytes(const LbAttention& p, int rows) { return (size_t)lb_
 
 int lb_attention_store(loom_b200_ctx* ctx, int dtype, const LbAttention& p, int T, uint8_t* q_img) {
     const int kch = lb_attention_kchunks(p.dim, dtype), qch = lb_attention_kchunks(p.dim, LOOM_B200_DTYPE_BF16);
-    const dim3 grid((p.pos0 + T - 1) / 8 - p.pos0 / 8 + 1);
+    const int rows = p.kv_heads + (q_img && dtype == LOOM_B200_DTYPE_BF16 ? p.heads : 0);
+    const dim3 grid((p.pos0 + T - 1) / 8 - p.pos0 / 8 + 1, rows + lb_ceil_div(p.kv_heads * p.vdim, 256));
     const bool vec = p.dim % 4 == 0 && lb_vec_rows(p.proj, p.ldp);
     if (dtype == LOOM_B200_DTYPE_BF16)
-        LB_LAUNCH(ctx, lb_attention_store_kernel<__nv_bfloat16>, grid, dim3(256), 0, p, T, kch, qch, q_img, vec);
+        LB_LAUNCH(ctx, lb_attention_store_kernel<__nv_bfloat16>, grid, dim3(256), 0, p, T, kch, qch, q_img, rows, vec);
     else
-        LB_LAUNCH(ctx, lb_attention_store_kernel<float>, grid, dim3(256), 0, p, T, kch, qch, nullptr, vec);
+        LB_LAUNCH(ctx, lb_attention_store_kernel<float>, grid, dim3(256), 0, p, T, kch, qch, nullptr, rows, vec);
     return 0;
 }
 

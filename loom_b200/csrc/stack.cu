@@ -151,6 +151,8 @@ size_t mixer_scratch(const LbLayer& l, int T, uint8_t* base, MixerScratch& m) {
         take(m.mem.sums, t * H);
         take(m.mem.tops, t * H);
         take(m.mem.scale, t * H);
+        take(m.mem.gate_i, t * H);
+        take(m.mem.gate_f, t * H);
     }
     m.delta.c = m.mem.c = m.c;
     return at;
