@@ -120,8 +120,6 @@ __global__ void __launch_bounds__(256) lb_delta_step_kernel(const LbDelta p, con
 
 // ---- token blocks ------------------------------------------------------------------------------------------------------
 
-constexpr int kRows = 8;  // tokens of a CTA
-
 // columns c .. c + 3 of a row of n
 template <bool VEC>
 __device__ __forceinline__ void store4(float* row, int c, int n, const float* f) {
@@ -134,18 +132,25 @@ __device__ __forceinline__ void store4(float* row, int c, int n, const float* f)
     }
 }
 
-// Convolution, activation and norms of the block's tokens, their gates: a warp per (head of q, k or v; token), four channels per
-// lane and pass.
-template <bool VEC>
+// Convolution, activation and norms of the block's tokens, their gates: a warp per (head of q, k or v; four tokens), four channels per
+// lane and pass.  TAPS taps (0: any number) stay in registers with the rows they are applied to.
+constexpr int kWarpTokens = 4;
+
+__device__ __forceinline__ float fast_siluf(float z) { return __fdividef(z, 1.f + expf(-z)); }
+
+template <bool VEC, int TAPS>
 __global__ void __launch_bounds__(256) lb_delta_tokens_kernel(const LbDelta p, const LbDeltaBlock b, int T, int pos0) {
+    constexpr int N = kWarpTokens;
     lb_pdl_launch_dependents();
     lb_pdl_wait();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, slots = 2 * p.kv_heads + p.heads, nch = lb_delta_channels(p), back = p.taps - 1;
-    const int t = blockIdx.x * kRows + warp, slot = blockIdx.y;
-    if (t >= T) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, slots = 2 * p.kv_heads + p.heads, nch = lb_delta_channels(p);
+    const int t0 = (blockIdx.x * 8 + warp) * N, slot = blockIdx.y;
+    if (t0 >= T) return;
     if (slot == slots) {  // the last row of CTAs makes the gates
-        const float* row = p.proj + (size_t)t * p.ldp;
-        for (int h = lane; h < p.heads; h += 32) {
+        for (int i = lane; i < N * p.heads; i += 32) {
+            const int t = t0 + i / p.heads, h = i % p.heads;
+            if (t >= T) break;
+            const float* row = p.proj + (size_t)t * p.ldp;
             b.beta[(size_t)t * p.heads + h] = write_strength(p, row, h);
             b.logg[(size_t)t * p.heads + h] = log_gate(p, row, h);
         }
@@ -153,35 +158,63 @@ __global__ void __launch_bounds__(256) lb_delta_tokens_kernel(const LbDelta p, c
     }
     const bool value = slot >= 2 * p.kv_heads;
     const int n = value ? p.vdim : p.dim, c0 = value ? 2 * p.kv_heads * p.dim + (slot - 2 * p.kv_heads) * p.vdim : slot * p.dim;
-    float* out = b.qkv + (size_t)t * nch + c0;
-    float ss = 0.f;
+    float* out = b.qkv + (size_t)t0 * nch + c0;
+    auto read = [&](int t, int c, float* y) {  // projections of the block's token t, of an earlier one (in the ring), or before the start
+        if (pos0 + t < 0 || t >= T)
+            y[0] = y[1] = y[2] = y[3] = 0.f;
+        else
+            lb_load_cols<4>(t >= 0 ? p.proj + (size_t)t * p.ldp + c0 : p.ring + (size_t)((pos0 + t) % p.taps) * nch + c0, c, n, VEC, y);
+    };
+    float ss[N] = {};
     for (int c = lane * 4; c < n; c += 128) {
-        float a[4] = {0.f, 0.f, 0.f, 0.f}, w[4], y[4];
-#pragma unroll 4
-        for (int j = 0; j <= back; ++j) {
-            const int ts = t - back + j;
-            if (pos0 + ts < 0) continue;
-            lb_load_cols<4>(p.conv_w + (size_t)j * nch + c0, c, n, VEC, w);
-            lb_load_cols<4>(ts >= 0 ? p.proj + (size_t)ts * p.ldp + c0 : p.ring + (size_t)((pos0 + ts) % p.taps) * nch + c0, c, n, VEC, y);
+        float a[N][4] = {};
+        if (TAPS > 0) {
+            constexpr int K = TAPS > 0 ? TAPS : 1;
+            float w[K][4], y[N + K - 1][4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) a[e] = fmaf(w[e], y[e], a[e]);
+            for (int j = 0; j < K; ++j) lb_load_cols<4>(p.conv_w + (size_t)j * nch + c0, c, n, VEC, w[j]);
+#pragma unroll
+            for (int j = 0; j < N + K - 1; ++j) read(t0 - (K - 1) + j, c, y[j]);
+#pragma unroll
+            for (int i = 0; i < N; ++i)
+#pragma unroll
+                for (int j = 0; j < K; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) a[i][e] = fmaf(w[j][e], y[i + j][e], a[i][e]);
+        } else {
+            for (int j = 0; j < p.taps; ++j) {  // tap j looks back taps - 1 - j positions
+                float w[4], y[4];
+                lb_load_cols<4>(p.conv_w + (size_t)j * nch + c0, c, n, VEC, w);
+#pragma unroll
+                for (int i = 0; i < N; ++i) {
+                    read(t0 + i - (p.taps - 1) + j, c, y);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) a[i][e] = fmaf(w[e], y[e], a[i][e]);
+                }
+            }
         }
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            a[e] = lb_siluf(a[e]);  // (zero behind the last channel)
-            ss = fmaf(a[e], a[e], ss);
+        for (int i = 0; i < N; ++i) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                a[i][e] = fast_siluf(a[i][e]);  // (zero behind the last channel)
+                ss[i] = fmaf(a[i][e], a[i][e], ss[i]);
+            }
+            if (t0 + i < T) store4<VEC>(out + (size_t)i * nch, c, n, a[i]);
         }
-        store4<VEC>(out, c, n, a);
     }
     if (value) return;
-    ss = lb_warp_sumf(ss);
-    const float r = __fdiv_rn(slot < p.kv_heads ? p.qscale : 1.f, sqrtf(ss + kUnitEps));
-    for (int c = lane * 4; c < n; c += 128) {  // (a thread reads back what it wrote)
-        float a[4];
-        lb_load_cols<4>(out, c, n, VEC, a);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) a[e] *= r;
-        store4<VEC>(out, c, n, a);
+    for (int i = 0; i < N; ++i) {
+        const float r = __fdiv_rn(slot < p.kv_heads ? p.qscale : 1.f, sqrtf(lb_warp_sumf(ss[i]) + kUnitEps));
+        if (t0 + i >= T) break;
+        for (int c = lane * 4; c < n; c += 128) {  // (a thread reads back what it wrote)
+            float a[4];
+            lb_load_cols<4>(out + (size_t)i * nch, c, n, VEC, a);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) a[e] *= r;
+            store4<VEC>(out + (size_t)i * nch, c, n, a);
+        }
     }
 }
 
@@ -451,10 +484,12 @@ __global__ void __launch_bounds__(256, 2) lb_delta_prep_kernel(const LbDelta p, 
 
 // ---- the states in front of the chunks, one after the other: CTA = (a few value columns, head) ---------------------------
 //
-// S <- G S + N - M S with M = Kd^T Wk (dim x dim) and N = Kd^T Wv.  Panels of rows of M and the columns of N travel while the panel
-// before is worked on; the old and the new state are in shared memory.  Two halves of the threads split the sum over the old state's
-// rows; a thread has 4 x 4 of the panel's results, its rows a quarter of the panel apart (neighbouring threads, neighbouring rows).
+// S <- G S + N - M S with M = Kd^T Wk (dim x dim) and N = Kd^T Wv.  Panels of up to 128 rows of M and the columns of N travel while
+// the panel before is worked on; the old and the new state are in shared memory.  A lane has two rows of the panel and all of the CTA's
+// columns, so that a row of the old state is one broadcast for a whole warp; two warps have the panel's rows, kScanSplit such pairs split
+// the sum over the old state's rows.
 constexpr size_t kScanSmem = 224 * 1024;
+constexpr int kScanRows = 2, kScanSplit = 4, kScanWarps = 2 * kScanSplit;
 
 __device__ __forceinline__ void copy_async(float* dst, const float* src, bool wide) {
     if (wide)
@@ -463,9 +498,9 @@ __device__ __forceinline__ void copy_async(float* dst, const float* src, bool wi
         asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(lb_smem_u32(dst)), "l"(src) : "memory");
 }
 
-size_t scan_smem(int dim, int panel, int cols) {
-    return ((size_t)2 * panel * lead(dim) + (size_t)4 * lb_round_up(dim, 4) * cols + (size_t)panel * cols) * sizeof(float);
-}
+// floats of a panel's buffer: the panel, later the warps' sums
+__host__ __device__ inline int scan_buffer(int dim, int panel, int cols) { return panel * (lead(dim) > kScanSplit * cols ? lead(dim) : kScanSplit * cols); }
+size_t scan_smem(int dim, int panel, int cols) { return ((size_t)2 * scan_buffer(dim, panel, cols) + (size_t)4 * lb_round_up(dim, 4) * cols) * sizeof(float); }
 struct ScanShape {
     int panel, cols;
 };
@@ -475,98 +510,118 @@ ScanShape scan_shape(int dim, int vdim, int heads, int sms) {
     int cols = lb_round_up(lb_ceil_div(vdim, per_head), 4);
     if (cols > 32) cols = 32;
     int want = 128;
-    while (want > 16 && want / 2 >= dim) want /= 2;
+    while (want > 32 && want / 2 >= dim) want /= 2;
     for (; cols >= 4; cols -= 4) {
         int panel = want;
-        while (panel > 8 && scan_smem(dim, panel, cols) > kScanSmem) panel /= 2;
+        while (panel > 4 && scan_smem(dim, panel, cols) > kScanSmem) panel /= 2;
         if (scan_smem(dim, panel, cols) > kScanSmem) continue;
-        if (panel >= 32 || panel == want || cols == 4) return {panel, cols};
+        if (panel >= 32 || cols == 4) return {panel, cols};
     }
     return {0, 0};
 }
 
-__global__ void __launch_bounds__(512) lb_delta_scan_kernel(const LbDeltaBlock b, int chunks, int panel, int cols, int fresh, bool wide_m, bool wide_n) {
+template <int COLS>
+__global__ void __launch_bounds__(kScanWarps * 32, 1) lb_delta_scan_kernel(const LbDeltaBlock b, int chunks, int panel, int fresh, bool wide_m, bool wide_n) {
     extern __shared__ __align__(16) float sm[];
+    constexpr int NT = kScanWarps * 32;
     const LbChunks& c = b.c;
-    const int dim = c.dim, vdim = c.vdim, LD = lead(dim), DP = lb_round_up(dim, 4), tid = threadIdx.x, nt = blockDim.x, h = blockIdx.y, v0 = blockIdx.x * cols;
-    float *sM = sm, *sN = sM + 2 * panel * LD, *sS = sN + 2 * DP * cols, *red = sS + 2 * DP * cols;
-    const int panels = lb_ceil_div(dim, panel), steps = chunks * panels, live = min(cols, vdim - v0);
-    for (int i = tid; i < 2 * panel * LD + (4 * DP + panel) * cols; i += nt) sm[i] = 0.f;
+    const int dim = c.dim, vdim = c.vdim, LD = lead(dim), DP = lb_round_up(dim, 4), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, v0 = blockIdx.x * COLS;
+    const int buffer = scan_buffer(dim, panel, COLS);
+    float *sM = sm, *sN = sM + 2 * buffer, *sS = sN + 2 * DP * COLS;
+    const int panels = lb_ceil_div(dim, panel), steps = chunks * panels, live = min(COLS, vdim - v0);
+    for (int i = tid; i < 2 * buffer + 4 * DP * COLS; i += NT) sm[i] = 0.f;
     __syncthreads();
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     float* S0 = c.state + (size_t)h * dim * vdim + v0;
     if (!fresh)
-        for (int i = tid; i < dim * cols; i += nt) {
-            const int d = i / cols, v = i % cols;
+        for (int i = tid; i < dim * COLS; i += NT) {
+            const int d = i / COLS, v = i % COLS;
             if (v < live) sS[i] = S0[(size_t)d * vdim + v];
         }
-    const int qm = wide_m ? 4 : 1, per = dim / qm, qn = wide_n ? 4 : 1, pn = live / qn;
+    const int qm = wide_m ? 4 : 1, qn = wide_n ? 4 : 1;
     auto fetch = [&](int step) {
         const int cc = step / panels, d0 = (step - cc * panels) * panel, rows = min(panel, dim - d0);
         const float* M = b.mix + (((size_t)cc * c.heads + h) * dim + d0) * dim;
-        float* dst = sM + (step & 1) * panel * LD;
-        for (int i = tid; i < rows * per; i += nt) {
-            const int r = i / per, e = (i - r * per) * qm;
-            copy_async(dst + r * LD + e, M + (size_t)r * dim + e, wide_m);
+        float* dst = sM + (step & 1) * buffer;
+        if (wide_m && dim == 128) {
+            dst += warp * LD + lane * 4;
+            M += warp * 128 + lane * 4;
+#pragma unroll 4
+            for (int r = warp; r < rows; r += kScanWarps, dst += kScanWarps * LD, M += kScanWarps * 128) copy_async(dst, M, true);
+        } else {
+            for (int r = warp; r < rows; r += kScanWarps)
+                for (int e = lane * qm; e < dim; e += 32 * qm) copy_async(dst + r * LD + e, M + (size_t)r * dim + e, wide_m);
         }
         if (d0 == 0) {
             const float* N = c.states + ((size_t)cc * c.heads + h) * dim * vdim + v0;
-            float* to = sN + (cc & 1) * DP * cols;
-            for (int i = tid; i < dim * pn; i += nt) {
-                const int d = i / pn, v = (i - d * pn) * qn;
-                copy_async(to + d * cols + v, N + (size_t)d * vdim + v, wide_n);
+            float* to = sN + (cc & 1) * DP * COLS;
+            for (int i = tid; i < dim * (COLS / qn); i += NT) {
+                const int d = i / (COLS / qn), v = (i - d * (COLS / qn)) * qn;
+                if (v < live) copy_async(to + d * COLS + v, N + (size_t)d * vdim + v, wide_n);
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    const int RG = panel / 4, CG = cols / 4, items = RG * CG, half = tid / items, item = tid - half * items, rg = item / CG, v = (item - rg * CG) * 4;
-    const int split = DP / 8 * 4, e0 = half == 0 ? 0 : split, e1 = half == 0 ? split : DP;
+    const int part = warp >> 1, row0 = (warp & 1) * 32 * kScanRows + lane, e0 = DP / 4 * part / kScanSplit * 4, e1 = DP / 4 * (part + 1) / kScanSplit * 4;
     fetch(0);
     for (int step = 0; step < steps; ++step) {
-        const int cc = step / panels, d0 = (step - cc * panels) * panel;
+        const int cc = step / panels, d0 = (step - cc * panels) * panel, rows = min(panel, dim - d0);
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // the panel is here, and everyone is done with the other buffer
         if (step + 1 < steps) fetch(step + 1);
-        const float *S = sS + (cc & 1) * DP * cols, *N = sN + (cc & 1) * DP * cols, *M = sM + (step & 1) * panel * LD + rg * LD;
-        float acc[4][4] = {};
-        if (half < 2) {
+        const float g = c.decay[(size_t)cc * c.heads + h];
+        const float *S = sS + (cc & 1) * DP * COLS, *N = sN + (cc & 1) * DP * COLS;
+        float* M = sM + (step & 1) * buffer;
+        uint64_t acc[kScanRows][COLS / 2] = {};  // pairs of columns
 #pragma unroll 2
-            for (int e = e0; e < e1; e += 4) {  // (rows behind the panel's last one hold finite leftovers and are not stored)
-                float4 m[4], s[4];
+        for (int e = e0; e < e1; e += 4) {
+            float m[kScanRows][4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) m[i] = *reinterpret_cast<const float4*>(M + i * RG * LD + e);
+            for (int i = 0; i < kScanRows; ++i) {
+                const float4 x = row0 + 32 * i < rows ? *reinterpret_cast<const float4*>(M + (row0 + 32 * i) * LD + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+                m[i][0] = x.x;
+                m[i][1] = x.y;
+                m[i][2] = x.z;
+                m[i][3] = x.w;
+            }
 #pragma unroll
-                for (int k = 0; k < 4; ++k) s[k] = *reinterpret_cast<const float4*>(S + (e + k) * cols + v);
+            for (int k = 0; k < 4; ++k) {
+                uint64_t mm[kScanRows];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const float mv[4] = {m[i].x, m[i].y, m[i].z, m[i].w};
+                for (int i = 0; i < kScanRows; ++i) mm[i] = lb_pack2(m[i][k], m[i][k]);
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) {
-                        acc[i][0] = fmaf(mv[k], s[k].x, acc[i][0]);
-                        acc[i][1] = fmaf(mv[k], s[k].y, acc[i][1]);
-                        acc[i][2] = fmaf(mv[k], s[k].z, acc[i][2]);
-                        acc[i][3] = fmaf(mv[k], s[k].w, acc[i][3]);
+                for (int v = 0; v < COLS; v += 4) {
+                    const ulonglong2 s = *reinterpret_cast<const ulonglong2*>(S + (e + k) * COLS + v);
+#pragma unroll
+                    for (int i = 0; i < kScanRows; ++i) {
+                        acc[i][v / 2] = lb_fma2(mm[i], s.x, acc[i][v / 2]);
+                        acc[i][v / 2 + 1] = lb_fma2(mm[i], s.y, acc[i][v / 2 + 1]);
                     }
                 }
             }
         }
-        if (half == 1)
+        __syncthreads();  // the panel has been read: its buffer takes the warps' sums [part][column / 4][row][4]
 #pragma unroll
-            for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + (rg + i * RG) * cols + v) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+        for (int i = 0; i < kScanRows; ++i)
+            if (row0 + 32 * i < rows)
+#pragma unroll
+                for (int v = 0; v < COLS; v += 4)
+                    *reinterpret_cast<ulonglong2*>(M + ((part * (COLS / 4) + v / 4) * panel + row0 + 32 * i) * 4) = make_ulonglong2(acc[i][v / 2], acc[i][v / 2 + 1]);
         __syncthreads();
-        if (half != 0) continue;
-        const float g = c.decay[(size_t)cc * c.heads + h];
-        float* next = sS + ((cc + 1) & 1) * DP * cols;
+        float* next = sS + ((cc + 1) & 1) * DP * COLS;
         float* out = c.states + ((size_t)cc * c.heads + h) * dim * vdim + v0;
+        for (int i = tid; i < rows * (COLS / 4); i += NT) {
+            const int q = i / rows, r = i - q * rows, v = q * 4, d = d0 + r;
+            float4 x = *reinterpret_cast<const float4*>(M + (q * panel + r) * 4);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int r = rg + i * RG, d = d0 + r;
-            if (d >= dim) continue;
-            const float4 x = *reinterpret_cast<const float4*>(red + r * cols + v), old = *reinterpret_cast<const float4*>(S + d * cols + v),
-                         add = *reinterpret_cast<const float4*>(N + d * cols + v);
-            *reinterpret_cast<float4*>(next + d * cols + v) = make_float4(fmaf(g, old.x, add.x - (acc[i][0] + x.x)), fmaf(g, old.y, add.y - (acc[i][1] + x.y)),
-                                                                          fmaf(g, old.z, add.z - (acc[i][2] + x.z)), fmaf(g, old.w, add.w - (acc[i][3] + x.w)));
+            for (int w = 1; w < kScanSplit; ++w) {
+                const float4 y = *reinterpret_cast<const float4*>(M + ((w * (COLS / 4) + q) * panel + r) * 4);
+                x = make_float4(x.x + y.x, x.y + y.y, x.z + y.z, x.w + y.w);
+            }
+            const float4 old = *reinterpret_cast<const float4*>(S + d * COLS + v), add = *reinterpret_cast<const float4*>(N + d * COLS + v);
+            *reinterpret_cast<float4*>(next + d * COLS + v) =
+                make_float4(fmaf(g, old.x, add.x - x.x), fmaf(g, old.y, add.y - x.y), fmaf(g, old.z, add.z - x.z), fmaf(g, old.w, add.w - x.w));
             const float o[4] = {old.x, old.y, old.z, old.w};
             if (wide_n)
                 store4<true>(out + (size_t)d * vdim, v, live, o);
@@ -575,11 +630,33 @@ __global__ void __launch_bounds__(512) lb_delta_scan_kernel(const LbDeltaBlock b
         }
     }
     __syncthreads();
-    const float* last = sS + (chunks & 1) * DP * cols;
-    for (int i = tid; i < dim * cols; i += nt) {
-        const int d = i / cols, x = i % cols;
+    const float* last = sS + (chunks & 1) * DP * COLS;
+    for (int i = tid; i < dim * COLS; i += NT) {
+        const int d = i / COLS, x = i % COLS;
         if (x < live) S0[(size_t)d * vdim + x] = last[i];
     }
+}
+
+template <int COLS>
+int launch_scan(loom_b200_ctx* ctx, const LbDeltaBlock& b, int chunks, int panel, bool fresh) {
+    LB_BIG_SMEM(ctx, lb_delta_scan_kernel<COLS>, kScanSmem);
+    LB_LAUNCH(ctx, lb_delta_scan_kernel<COLS>, dim3(lb_ceil_div(b.c.vdim, COLS), b.c.heads), dim3(kScanWarps * 32), scan_smem(b.c.dim, panel, COLS), b, chunks, panel, fresh ? 1 : 0,
+              b.c.dim % 4 == 0, b.c.vdim % 4 == 0);
+    return 0;
+}
+int run_scan(loom_b200_ctx* ctx, const LbDeltaBlock& b, int chunks, bool fresh) {
+    const ScanShape s = scan_shape(b.c.dim, b.c.vdim, b.c.heads, ctx->sm_count);
+    switch (s.cols) {
+        case 4: return launch_scan<4>(ctx, b, chunks, s.panel, fresh);
+        case 8: return launch_scan<8>(ctx, b, chunks, s.panel, fresh);
+        case 12: return launch_scan<12>(ctx, b, chunks, s.panel, fresh);
+        case 16: return launch_scan<16>(ctx, b, chunks, s.panel, fresh);
+        case 20: return launch_scan<20>(ctx, b, chunks, s.panel, fresh);
+        case 24: return launch_scan<24>(ctx, b, chunks, s.panel, fresh);
+        case 28: return launch_scan<28>(ctx, b, chunks, s.panel, fresh);
+        case 32: return launch_scan<32>(ctx, b, chunks, s.panel, fresh);
+    }
+    return lb_fail(ctx, LOOM_B200_ERR_UNSUPPORTED, "delta rule: %d key channels", b.c.dim);
 }
 
 size_t prep_smem(int C, int dim) {
@@ -624,11 +701,13 @@ int lb_delta_block(loom_b200_ctx* ctx, const LbDelta& p, const LbDeltaBlock& bin
     b.c.ldo = p.ldo;
     const int chunks = lb_ceil_div(T, b.c.C);
     const bool vec = p.dim % 4 == 0 && p.vdim % 4 == 0 && lb_vec_rows(p.proj, p.ldp);
-    const dim3 tokens(lb_ceil_div(T, kRows), 2 * p.kv_heads + p.heads + 1);
-    if (vec)
-        LB_LAUNCH(ctx, lb_delta_tokens_kernel<true>, tokens, dim3(256), 0, p, b, T, pos0);
+    const dim3 tokens(lb_ceil_div(T, 8 * kWarpTokens), 2 * p.kv_heads + p.heads + 1);
+    if (vec && p.taps == 4)
+        LB_LAUNCH(ctx, (lb_delta_tokens_kernel<true, 4>), tokens, dim3(256), 0, p, b, T, pos0);
+    else if (vec)
+        LB_LAUNCH(ctx, (lb_delta_tokens_kernel<true, 0>), tokens, dim3(256), 0, p, b, T, pos0);
     else
-        LB_LAUNCH(ctx, lb_delta_tokens_kernel<false>, tokens, dim3(256), 0, p, b, T, pos0);
+        LB_LAUNCH(ctx, (lb_delta_tokens_kernel<false, 0>), tokens, dim3(256), 0, p, b, T, pos0);
     if (p.taps > 1) LB_LAUNCH(ctx, lb_delta_commit_kernel, dim3(lb_ceil_div(lb_delta_channels(p), 256), p.taps - 1), dim3(256), 0, p, T, pos0);
     int rc = b.c.C == 64 ? launch_prep<64>(ctx, p, b, T, vec) : b.c.C == 32 ? launch_prep<32>(ctx, p, b, T, vec) : launch_prep<16>(ctx, p, b, T, vec);
     if (rc) return rc;
@@ -639,10 +718,6 @@ int lb_delta_block(loom_b200_ctx* ctx, const LbDelta& p, const LbDeltaBlock& bin
     m.ldv = p.heads * p.dim;
     m.states = b.mix;
     if ((rc = lb_chunk_states(ctx, m, T))) return rc;
-    const ScanShape sh = scan_shape(p.dim, p.vdim, p.heads, ctx->sm_count);
-    const int threads = lb_round_up(2 * (sh.panel / 4) * (sh.cols / 4), 32);
-    LB_BIG_SMEM(ctx, lb_delta_scan_kernel, kScanSmem);
-    LB_LAUNCH(ctx, lb_delta_scan_kernel, dim3(lb_ceil_div(p.vdim, sh.cols), p.heads), dim3(threads), scan_smem(p.dim, sh.panel, sh.cols), b, chunks, sh.panel, sh.cols,
-              pos0 == 0 ? 1 : 0, p.dim % 4 == 0, p.vdim % 4 == 0);
+    if ((rc = run_scan(ctx, b, chunks, pos0 == 0))) return rc;
     return lb_chunk_out(ctx, b.c, T);
 }

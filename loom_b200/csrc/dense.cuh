@@ -116,6 +116,18 @@ __device__ __forceinline__ float lb_warp_sumf(float v) {
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
 }
+// two floats in a 64-bit register and their fused multiply-add, one instruction for both
+__device__ __forceinline__ uint64_t lb_pack2(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ void lb_unpack2(uint64_t r, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(r)); }
+__device__ __forceinline__ uint64_t lb_fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
 // sum over all warps of a block; red holds one float per warp, every thread gets the result
 __device__ __forceinline__ float lb_block_sumf(float v, float* red) {
     v = lb_warp_sumf(v);

@@ -105,9 +105,19 @@ __global__ void __launch_bounds__(256) lb_memory_gates_kernel(const LbMemory p, 
     b.gate_f[(size_t)h * T + t] = gf;
 }
 
+__device__ __forceinline__ void put4(float* row, int d, int n, bool vec, const float* f) {
+    if (vec) {
+        *reinterpret_cast<float4*>(row + d) = make_float4(f[0], f[1], f[2], f[3]);
+    } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+            if (d + e < n) row[d + e] = f[e];
+    }
+}
+
 // CTA = (chunk, head): maxima, weights, and the operands of the products over chunks
 template <int C>
-__global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p, const LbMemoryBlock b, int T, int pos0, bool vec) {
+__global__ void __launch_bounds__(256, 3) lb_memory_prep_kernel(const LbMemory p, const LbMemoryBlock b, int T, int pos0, bool vec) {
     extern __shared__ __align__(16) float sm[];
     __shared__ Run s_run[8];
     __shared__ double s_F[C];
@@ -115,7 +125,7 @@ __global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p
     constexpr int NI = C / 16, LC = C + 4;
     const int ch = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, dim = p.dim, LD = lead(dim);
     const int HD = p.heads * dim, t0 = ch * C, n = min(C, T - t0), D4 = lb_round_up(dim, 4) / 4;
-    float *sq = sm, *sk = sq + C * LD, *sa = sk + C * LD;
+    float *sk = sm, *sq = sk + C * LD, *sa = sq;  // sa [C][LC]: the weights, in place of the queries
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const float *gi = b.gate_i + (size_t)h * T, *gf = b.gate_f + (size_t)h * T;
@@ -166,6 +176,7 @@ __global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p
         s_end[tid] = expf((float)(s_F[C - 1] - s_F[tid] + s_i[tid] - s_m[C - 1]));
         if (tid < n) b.tops[(size_t)(t0 + tid) * p.heads + h] = s_m[tid];
     }
+    __syncthreads();
     {
         const int ty = tid >> 4, tx = tid & 15;
         float qk[NI][NI] = {};
@@ -181,6 +192,13 @@ __global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p
 #pragma unroll
                 for (int j = 0; j <= i; ++j) qk[i][j] = fmaf(q[i].x, k[j].x, fmaf(q[i].y, k[j].y, fmaf(q[i].z, k[j].z, fmaf(q[i].w, k[j].w, qk[i][j]))));
         }
+        for (int i = tid; i < n * D4; i += 256) {  // queries decayed from the chunk's start
+            const int t = i / D4, d = (i - t * D4) * 4;
+            const float4 q = *reinterpret_cast<const float4*>(sq + t * LD + d);
+            const float f[4] = {q.x * s_keep[t], q.y * s_keep[t], q.z * s_keep[t], q.w * s_keep[t]};
+            put4(b.c.qd + (size_t)(t0 + t) * HD + h * dim, d, dim, vec, f);
+        }
+        __syncthreads();
         float* A = b.c.weights + ((size_t)ch * p.heads + h) * C * C;
 #pragma unroll
         for (int i = 0; i < NI; ++i)
@@ -200,26 +218,14 @@ __global__ void __launch_bounds__(256, 2) lb_memory_prep_kernel(const LbMemory p
         s = lb_warp_sumf(s);
         if (lane == 0) b.sums[(size_t)(t0 + t) * p.heads + h] = s;
     }
-    // keys decayed to the chunk's end, queries decayed from its start
+    // keys decayed to the chunk's end
     const float over = s_keep[C - 1];
     for (int i = tid; i < n * D4; i += 256) {
         const int t = i / D4, d = (i - t * D4) * 4;
-        const float e = s_end[t], g = s_keep[t];
-        const float4 q = *reinterpret_cast<const float4*>(sq + t * LD + d), k = *reinterpret_cast<const float4*>(sk + t * LD + d);
-        const float qd[4] = {q.x * g, q.y * g, q.z * g, q.w * g}, kd[4] = {k.x * e, k.y * e, k.z * e, k.w * e};
-        const size_t at = (size_t)(t0 + t) * HD + h * dim;
-        *reinterpret_cast<float4*>(sk + t * LD + d) = make_float4(kd[0], kd[1], kd[2], kd[3]);
-        if (vec) {
-            *reinterpret_cast<float4*>(b.c.qd + at + d) = make_float4(qd[0], qd[1], qd[2], qd[3]);
-            *reinterpret_cast<float4*>(b.c.kd + at + d) = make_float4(kd[0], kd[1], kd[2], kd[3]);
-        } else {
-#pragma unroll
-            for (int x = 0; x < 4; ++x)
-                if (d + x < dim) {
-                    b.c.qd[at + d + x] = qd[x];
-                    b.c.kd[at + d + x] = kd[x];
-                }
-        }
+        const float4 k = *reinterpret_cast<const float4*>(sk + t * LD + d);
+        const float f[4] = {k.x * s_end[t], k.y * s_end[t], k.z * s_end[t], k.w * s_end[t]};
+        *reinterpret_cast<float4*>(sk + t * LD + d) = make_float4(f[0], f[1], f[2], f[3]);
+        put4(b.c.kd + (size_t)(t0 + t) * HD + h * dim, d, dim, vec, f);
     }
     __syncthreads();
     for (int d = tid; d < dim; d += 256) {
@@ -272,7 +278,10 @@ __global__ void __launch_bounds__(256) lb_memory_scale_kernel(const LbMemory p, 
     if (lane == 0) b.scale[i] = __fdiv_rn(1.f, fmaxf(fabsf(d), expf(-b.tops[i])) + kDenEps);
 }
 
-size_t prep_smem(int C, int dim) { return ((size_t)2 * C * lead(dim) + (size_t)C * (C + 4)) * sizeof(float); }
+size_t prep_smem(int C, int dim) {
+    const size_t q = lead(dim) > C + 4 ? lead(dim) : C + 4;
+    return (size_t)C * (lead(dim) + q) * sizeof(float);
+}
 
 template <int C>
 int launch_prep(loom_b200_ctx* ctx, const LbMemory& p, const LbMemoryBlock& b, int T, int pos0) {
