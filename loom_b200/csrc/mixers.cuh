@@ -143,9 +143,11 @@ struct LbAttention {
     uint8_t *k = nullptr, *vt = nullptr;  // [lane] caches
     size_t k_lane = 0, vt_lane = 0;
     int ring = 0, slices = 0;     // slices: K slices of a row of vt
+    bool mma = false;             // the step runs on the tensor cores (lb_attention_step_mma)
     const int* pos = nullptr;     // position of every token (one token per sequence), or null: token t is at pos0 + t of lane0
     int pos0 = 0, lane0 = 0;
 };
+bool lb_attention_step_mma(int dim, int vdim, int dtype);
 int lb_attention_kchunks(int dim, int dtype);
 size_t lb_attention_k_bytes(int kv_heads, int dim, int ring, int dtype);
 size_t lb_attention_vt_bytes(int kv_heads, int vdim, int ring, int dtype);

@@ -91,10 +91,91 @@ __global__ void __launch_bounds__(256) lb_attention_store_kernel(const LbAttenti
     }
 }
 
-// One token per sequence: CTA = (split of the visible positions, HB query heads of a kv head, token).  Tiles of 64 positions: four
-// threads per key for the scores, a warp per head for the running softmax, then four threads per value row and K slice for the
-// weighted sum.  The split with the newest position takes its key and value from the projections and puts them into the cache.
-// The last CTA of a (token, heads) to arrive merges the splits; nothing waits.
+// ---- the step: one token per sequence ----------------------------------------------------------------------------------------
+//
+// CTA = (split of the visible positions, HB query heads of a kv head, token).  The split with the newest position takes its key and
+// value from the projections and puts them into the cache.  Partial results are [token][kv head and block][split][HB] {vdim sums,
+// maximum, sum}; the last CTA of a (token, heads) to arrive merges them, nothing waits.
+
+// where the CTA works
+struct StepPlace {
+    int split, g, hb, m, h0, nh, pos, seq, low, active, j0, j1;
+    bool newest;  // (otherwise every position is in the cache)
+};
+template <int HB>
+__device__ __forceinline__ StepPlace step_place(const LbAttention& p, int splits) {
+    StepPlace w;
+    const int per = p.heads / p.kv_heads, nb = lb_ceil_div(per, HB);
+    w.split = blockIdx.x;
+    w.g = blockIdx.y / nb;
+    w.hb = blockIdx.y % nb;
+    w.m = blockIdx.z;
+    w.h0 = w.g * per + w.hb * HB;
+    w.nh = min(HB, per - w.hb * HB);
+    w.pos = p.pos ? p.pos[w.m] : p.pos0 + w.m;
+    w.seq = p.pos ? p.lane0 + w.m : p.lane0;
+    w.low = p.chunk ? w.pos - w.pos % p.chunk : 0;
+    const int first = w.low / kTile, ntiles = w.pos / kTile - first + 1;  // every tile has a visible position
+    w.active = min(splits, ntiles);
+    w.j0 = first + (int)((long long)ntiles * w.split / w.active);
+    w.j1 = first + (int)((long long)ntiles * (w.split + 1) / w.active);
+    w.newest = p.pos && w.split == w.active - 1;
+    return w;
+}
+
+__device__ __forceinline__ float* partial_row(const LbAttention& p, float* part, int group, int splits, int split, int HB) {
+    return part + ((size_t)group * splits + split) * HB * (p.vdim + 2);
+}
+
+// after every thread of the CTA has written its part of the partial result; sw: HB * 64 floats
+template <int HB>
+__device__ __forceinline__ void merge_splits(const LbAttention& p, float* part, unsigned* count, int group, int splits, int active, int h0, int nh, const float* gate, float* sw,
+                                             float* o) {
+    __shared__ bool s_last;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = p.vdim + 2;
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) {
+        s_last = atomicAdd(count + group, 1u) == (unsigned)active - 1;
+        if (s_last) count[group] = 0;
+    }
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+    const float* all = partial_row(p, part, group, splits, 0, HB);
+    for (int h = warp; h < nh; h += 8) {
+        float mx = -INFINITY, den = 0.f, top[2], sum[2];  // (at most 64 splits)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int s = lane + 32 * i;
+            top[i] = s < active ? __ldcg(all + ((size_t)s * HB + h) * row + p.vdim) : -INFINITY;
+            sum[i] = s < active ? __ldcg(all + ((size_t)s * HB + h) * row + p.vdim + 1) : 0.f;
+            mx = fmaxf(mx, top[i]);
+        }
+        mx = lb_warp_max(mx);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            top[i] = expf(top[i] - mx);
+            den = fmaf(top[i], sum[i], den);
+        }
+        den = lb_warp_sumf(den);
+        float r = __fdiv_rn(1.f, den);
+        if (p.head_gate) r *= lb_sigmoidf(gate[h0 + h]);
+        sw[h * 64 + lane] = top[0] * r;
+        sw[h * 64 + lane + 32] = top[1] * r;
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * p.vdim; i += kStepThreads) {
+        const int h = i / p.vdim, v = i - h * p.vdim;
+        float a = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < active; ++s) a = fmaf(sw[h * 64 + s], __ldcg(all + ((size_t)s * HB + h) * row + v), a);
+        o[(h0 + h) * p.vdim + v] = a;
+    }
+}
+
+// Any precision and head size, plain multiply-adds.  Tiles of 64 positions: four threads per key for the scores, a warp per head for the
+// running softmax, then four threads per value row and K slice for the weighted sum.
 template <typename WT, int HB>
 __global__ void __launch_bounds__(kStepThreads) lb_attention_step_kernel(const LbAttention p, int kchunks, int splits, float* __restrict__ part, unsigned* __restrict__ count,
                                                                          float* __restrict__ out, int ldo) {
@@ -102,18 +183,13 @@ __global__ void __launch_bounds__(kStepThreads) lb_attention_step_kernel(const L
     constexpr int C = LbElem<WT>::kChunk, S = LbElem<WT>::kSlice, KS = kTile / S;  // KS: K slices of a tile
     __shared__ __align__(16) float s_w[HB][kTile];
     __shared__ float s_max[HB], s_sum[HB], s_fac[HB], s_new[HB], s_rq[HB], s_rk;
-    __shared__ bool s_last;
     lb_pdl_launch_dependents();
     lb_pdl_wait();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int per = p.heads / p.kv_heads, nb = lb_ceil_div(per, HB), split = blockIdx.x, g = blockIdx.y / nb, hb = blockIdx.y % nb, m = blockIdx.z;
-    const int h0 = g * per + hb * HB, nh = min(HB, per - hb * HB);
-    const int pos = p.pos ? p.pos[m] : p.pos0 + m, seq = p.pos ? p.lane0 + m : p.lane0;
-    const int low = p.chunk ? pos - pos % p.chunk : 0, tile_lo = low / kTile, ntiles = pos / kTile - tile_lo + 1;
-    const int active = min(splits, ntiles);
+    const StepPlace w = step_place<HB>(p, splits);
+    const int split = w.split, g = w.g, hb = w.hb, m = w.m, h0 = w.h0, nh = w.nh, pos = w.pos, seq = w.seq, low = w.low, active = w.active, j0 = w.j0, j1 = w.j1;
+    const bool newest = w.newest;
     if (split >= active) return;
-    const int j0 = tile_lo + (int)((long long)ntiles * split / active), j1 = tile_lo + (int)((long long)ntiles * (split + 1) / active);
-    const bool newest = p.pos && split == active - 1;  // (otherwise every position is in the cache)
     const int vrows = vrows_of(p.vdim), QD = p.heads * p.dim, KD = p.kv_heads * p.dim, kcols = kchunks * C;
     float *sq = reinterpret_cast<float*>(sm), *so = sq + HB * kcols;              // queries [HB][kcols]; sums [HB][vrows]
     uint4* skey = reinterpret_cast<uint4*>(so + HB * vrows);                      // the newest key's chunks
@@ -248,6 +324,7 @@ __global__ void __launch_bounds__(kStepThreads) lb_attention_step_kernel(const L
     }
     const float* gate = row + QD + KD + p.kv_heads * p.vdim;
     float* o = out + (size_t)m * ldo;
+    const int group = m * gridDim.y + blockIdx.y;
     if (active == 1) {
         for (int i = tid; i < nh * p.vdim; i += kStepThreads) {
             const int h = i / p.vdim, v = i - h * p.vdim;
@@ -256,56 +333,251 @@ __global__ void __launch_bounds__(kStepThreads) lb_attention_step_kernel(const L
         }
         return;
     }
-    // ---- partial sums [token][kv head and block][split][HB][vdim + 2], merged by the last to arrive ----
-    const int prow = p.vdim + 2, group = m * gridDim.y + blockIdx.y;
-    float* mine = part + ((size_t)group * splits + split) * HB * prow;
+    float* mine = partial_row(p, part, group, splits, split, HB);
     for (int i = tid; i < nh * p.vdim; i += kStepThreads) {
         const int h = i / p.vdim, v = i - h * p.vdim;
-        mine[h * prow + v] = so[h * vrows + v];
+        mine[h * (p.vdim + 2) + v] = so[h * vrows + v];
     }
     if (tid < nh) {
-        mine[tid * prow + p.vdim] = s_max[tid];
-        mine[tid * prow + p.vdim + 1] = s_sum[tid];
+        mine[tid * (p.vdim + 2) + p.vdim] = s_max[tid];
+        mine[tid * (p.vdim + 2) + p.vdim + 1] = s_sum[tid];
     }
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) {
-        s_last = atomicAdd(count + group, 1u) == (unsigned)active - 1;
-        if (s_last) count[group] = 0;
+    merge_splits<HB>(p, part, count, group, splits, active, h0, nh, gate, sq, o);
+}
+
+__device__ __forceinline__ void mma_bf16(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+// 16 rows x one 16-byte chunk per lane column: which k of a chunk an MMA takes is the same for both operands, so the order cancels
+__device__ __forceinline__ void mma_chunk(float* d, const uint4& a0, const uint4& a1, const uint4& b) {
+    mma_bf16(d, a0.x, a1.x, a0.y, a1.y, b.x, b.y);
+    mma_bf16(d, a0.z, a1.z, a0.w, a1.w, b.z, b.w);
+}
+// value = hi + lo, both bf16: the pair carries sixteen bits of the float
+__device__ __forceinline__ void split_bf16(const float* f, uint4& hi, uint4& lo) {
+    float h[8], l[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        h[i] = __bfloat162float(__float2bfloat16_rn(f[i]));
+        l[i] = f[i] - h[i];
     }
-    __syncthreads();
-    if (!s_last) return;
-    __threadfence();
-    const float* all = part + (size_t)group * splits * HB * prow;
-    float* sw = sq;  // [HB][64] share of every split
-    for (int h = warp; h < nh; h += 8) {
-        float mx = -INFINITY, den = 0.f;
-        for (int s = lane; s < active; s += 32) mx = fmaxf(mx, __ldcg(all + ((size_t)s * HB + h) * prow + p.vdim));
-        mx = lb_warp_max(mx);
-        for (int s = lane; s < active; s += 32) {
-            const float w = expf(__ldcg(all + ((size_t)s * HB + h) * prow + p.vdim) - mx);
-            sw[h * 64 + s] = w;
-            den = fmaf(w, __ldcg(all + ((size_t)s * HB + h) * prow + p.vdim + 1), den);
+    hi = lb_pack_chunk<__nv_bfloat16>(h);
+    lo = lb_pack_chunk<__nv_bfloat16>(l);
+}
+
+// bf16, up to sixteen query heads of a kv head per CTA on the tensor cores (MMA rows that no head uses cost nothing that is scarce here):
+// keys and values go from global memory straight into the B fragments.  A warp has eight of a tile's 64 keys for the scores and every
+// eighth group of eight value rows for the weighted sum; queries and softmax weights are bf16 pairs.  The next tile's keys and values
+// are requested as soon as this tile's fragments have been used.
+constexpr int kMmaHeads = 16;
+
+template <int NK, int NG>  // key chunks per lane (dim <= 32 NK), groups of value rows per warp (vdim <= 64 NG)
+__global__ void __launch_bounds__(kStepThreads, 2) lb_attention_step_mma_kernel(const LbAttention p, int kchunks, int splits, float* __restrict__ part, unsigned* __restrict__ count,
+                                                                                float* __restrict__ out, int ldo) {
+    constexpr int HB = kMmaHeads, SL = kTile + 4;
+    __shared__ __align__(16) uint4 s_q[2][NK * 4][HB + 2], s_key[NK * 4], s_p[2][kTile / 8][HB + 2];  // (rows padded against bank conflicts)
+    __shared__ __align__(16) float s_s[HB][SL];  // (the merge uses 64 a head)
+    __shared__ float s_max[HB], s_sum[HB], s_fac[HB];
+    __shared__ __nv_bfloat16 s_val[NG * 64];
+    lb_pdl_launch_dependents();
+    lb_pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const StepPlace w = step_place<HB>(p, splits);
+    if (w.split >= w.active) return;
+    const int vrows = vrows_of(p.vdim), QD = p.heads * p.dim, KD = p.kv_heads * p.dim;
+    const float* row = p.proj + (size_t)w.m * p.ldp;
+    uint8_t *kc = p.k + (size_t)w.seq * p.k_lane, *vc = p.vt + (size_t)w.seq * p.vt_lane;
+    uint4 kr[NK], vr[NG][2];
+    auto load_keys = [&](int j) {
+        const uint8_t* src = kc + key_chunk((j * kTile) % p.ring + warp * 8 + g, w.g, p.kv_heads, kchunks, 0);
+#pragma unroll
+        for (int i = 0; i < NK; ++i)
+            if (4 * i + t < kchunks) kr[i] = *reinterpret_cast<const uint4*>(src + (size_t)(4 * i + t) * 128);
+    };
+    auto load_values = [&](int j) {
+        const int c0 = (j * kTile) % p.ring / 8;
+#pragma unroll
+        for (int i = 0; i < NG; ++i)
+            if ((warp + 8 * i) * 8 < vrows)
+#pragma unroll
+                for (int x = 0; x < 2; ++x) vr[i][x] = *reinterpret_cast<const uint4*>(vc + lb_img_chunk(w.g * vrows + (warp + 8 * i) * 8 + g, c0 + t + 4 * x, p.slices));
+    };
+#pragma unroll
+    for (int i = 0; i < NK; ++i) kr[i] = make_uint4(0, 0, 0, 0);
+#pragma unroll
+    for (int i = 0; i < NG; ++i) vr[i][0] = vr[i][1] = make_uint4(0, 0, 0, 0);
+    load_keys(w.j0);
+    load_values(w.j0);
+    // queries, and the newest key, a warp per row and eight columns per lane
+    for (int i = warp; i < HB + (w.newest ? 1 : 0); i += 8) {
+        const bool key = i == HB;
+        const float* x = key ? row + QD + w.g * p.dim : row + (w.h0 + i) * p.dim;
+        float f[8], by = key || i < w.nh ? 1.f : 0.f;
+        if (by != 0.f) {
+            lb_load_cols<8>(x, lane * 8, p.dim, false, f);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = 0.f;
         }
-        den = lb_warp_sumf(den);
-        float r = __fdiv_rn(1.f, den);
-        if (p.head_gate) r *= lb_sigmoidf(gate[h0 + h]);
-        __syncwarp();
-        for (int s = lane; s < active; s += 32) sw[h * 64 + s] *= r;
+        if (p.qk_norm && by != 0.f) {
+            float ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss = fmaf(f[e], f[e], ss);
+            ss = lb_warp_sumf(ss);
+            by = __fdiv_rn(1.f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)p.dim), p.eps)));
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] *= by;
+        if (lane >= NK * 4) continue;
+        if (!key) {
+            split_bf16(f, s_q[0][lane][i], s_q[1][lane][i]);
+        } else {
+            s_key[lane] = lb_pack_chunk<__nv_bfloat16>(f);
+            if (w.hb == 0 && lane < kchunks) *reinterpret_cast<uint4*>(kc + key_chunk(w.pos % p.ring, w.g, p.kv_heads, kchunks, lane)) = s_key[lane];
+        }
     }
+    if (w.newest)
+        for (int v = tid; v < p.vdim; v += kStepThreads) {
+            const __nv_bfloat16 x = __float2bfloat16_rn(row[QD + KD + w.g * p.vdim + v]);
+            s_val[v] = x;
+            if (w.hb == 0) *reinterpret_cast<__nv_bfloat16*>(vc + value_at<__nv_bfloat16>(w.g, v, vrows, w.pos % p.ring, p.slices)) = x;
+        }
+    if (tid < HB) {
+        s_max[tid] = p.sink && w.split == 0 ? 0.f : -INFINITY;
+        s_sum[tid] = p.sink && w.split == 0 ? 1.f : 0.f;
+    }
+    float o[NG][4];
+#pragma unroll
+    for (int i = 0; i < NG; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     __syncthreads();
-    for (int i = tid; i < nh * p.vdim; i += kStepThreads) {
-        const int h = i / p.vdim, v = i - h * p.vdim;
-        float a = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < active; ++s) a = fmaf(sw[h * 64 + s], __ldcg(all + ((size_t)s * HB + h) * prow + v), a);
-        o[(h0 + h) * p.vdim + v] = a;
+    for (int j = w.j0; j < w.j1; ++j) {
+        const int base = j * kTile, at = w.newest && w.pos / kTile == j ? w.pos - base : -1;  // the newest position's place in the tile
+        // ---- scores of keys warp * 8 + 0..7 ----
+        {
+            float bias[4] = {0.f, 0.f, 0.f, 0.f}, d[4] = {0.f, 0.f, 0.f, 0.f};
+            const int key0 = base + warp * 8 + 2 * t;  // d: heads g (0, 1) and g + 8 (2, 3), keys key0 and key0 + 1
+            if (p.bias)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int h = g + 8 * (e >> 1), dist = min(max(w.pos - key0 - (e & 1), 0), p.bias_len - 1);
+                    if (h < w.nh) bias[e] = __ldg(p.bias + (size_t)(w.h0 + h) * p.bias_ld + kBiasFront + dist);
+                }
+            if (at >= 0 && warp * 8 + g == at)
+#pragma unroll
+                for (int i = 0; i < NK; ++i)
+                    if (4 * i + t < kchunks) kr[i] = s_key[4 * i + t];
+#pragma unroll
+            for (int i = 0; i < NK; ++i)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) mma_chunk(d, s_q[half][4 * i + t][g], s_q[half][4 * i + t][g + 8], kr[i]);
+            if (j + 1 < w.j1) load_keys(j + 1);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int key = key0 + (e & 1);
+                s_s[g + 8 * (e >> 1)][warp * 8 + 2 * t + (e & 1)] = key >= w.low && key <= w.pos ? fmaf(d[e], p.scale, bias[e]) : -INFINITY;
+            }
+        }
+        __syncthreads();
+        // ---- running softmax: sixteen threads per head, four positions each ----
+        {
+            const int h = tid >> 4, q = tid & 15;
+            const float4 x = *reinterpret_cast<const float4*>(&s_s[h][q * 4]);
+            float mx = fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w));
+#pragma unroll
+            for (int off = 8; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+            const float old = s_max[h], nm = fmaxf(old, mx);
+            float e[4] = {expf(x.x - nm), expf(x.y - nm), expf(x.z - nm), expf(x.w - nm)}, sum = (e[0] + e[1]) + (e[2] + e[3]);
+#pragma unroll
+            for (int off = 8; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+            __syncwarp();
+            if (q == 0) {
+                const float f = expf(old - nm);
+                s_max[h] = nm;
+                s_fac[h] = f;
+                s_sum[h] = fmaf(s_sum[h], f, sum);
+            }
+            float l[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float hi = __bfloat162float(__float2bfloat16_rn(e[i]));
+                l[i] = e[i] - hi;
+                e[i] = hi;
+            }
+            *(reinterpret_cast<uint2*>(&s_p[0][q >> 1][h]) + (q & 1)) = make_uint2(lb_pack_bf16(e[0], e[1]), lb_pack_bf16(e[2], e[3]));
+            *(reinterpret_cast<uint2*>(&s_p[1][q >> 1][h]) + (q & 1)) = make_uint2(lb_pack_bf16(l[0], l[1]), lb_pack_bf16(l[2], l[3]));
+        }
+        __syncthreads();
+        // ---- weighted sum: chunk t + 4 x holds positions 8 (t + 4 x) ... of this lane's value rows ----
+        {
+            const float f0 = s_fac[g], f1 = s_fac[g + 8];
+            if (at >= 0) {  // the newest position's values are not in the cache yet
+                const int c = at >> 3;
+#pragma unroll
+                for (int i = 0; i < NG; ++i) {
+                    const int v = (warp + 8 * i) * 8 + g;
+                    const uint32_t put = (uint32_t)__bfloat16_as_ushort(s_val[v < p.vdim ? v : 0]) << (16 * (at & 1)), keep = ~(0xffffu << (16 * (at & 1)));
+#pragma unroll
+                    for (int x = 0; x < 2; ++x) {
+                        const int word = c == t + 4 * x && v < p.vdim ? (at & 7) >> 1 : -1;
+                        uint4& y = vr[i][x];
+                        y.x = word == 0 ? (y.x & keep) | put : y.x;
+                        y.y = word == 1 ? (y.y & keep) | put : y.y;
+                        y.z = word == 2 ? (y.z & keep) | put : y.z;
+                        y.w = word == 3 ? (y.w & keep) | put : y.w;
+                    }
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < NG; ++i) {
+                o[i][0] *= f0;
+                o[i][1] *= f0;
+                o[i][2] *= f1;
+                o[i][3] *= f1;
+            }
+#pragma unroll
+            for (int half = 0; half < 2; ++half)
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    const uint4 a0 = s_p[half][t + 4 * x][g], a1 = s_p[half][t + 4 * x][g + 8];
+#pragma unroll
+                    for (int i = 0; i < NG; ++i) mma_chunk(o[i], a0, a1, vr[i][x]);
+                }
+            if (j + 1 < w.j1) load_values(j + 1);
+        }
+        __syncthreads();
     }
+    const float* gate = row + QD + KD + p.kv_heads * p.vdim;
+    float* dst = out + (size_t)w.m * ldo;
+    const int group = w.m * gridDim.y + blockIdx.y;
+    float* mine = partial_row(p, part, group, splits, w.split, HB);
+#pragma unroll
+    for (int hb = 0; hb < 2; ++hb) {
+        const int h = g + 8 * hb;
+        if (h >= w.nh) continue;
+        const float r = w.active > 1 ? 1.f : __fdiv_rn(p.head_gate ? lb_sigmoidf(gate[w.h0 + h]) : 1.f, s_sum[h]);
+        float* y = w.active > 1 ? mine + h * (p.vdim + 2) : dst + (w.h0 + h) * p.vdim;
+#pragma unroll
+        for (int i = 0; i < NG; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int v = (warp + 8 * i) * 8 + 2 * t + e;
+                if (v < p.vdim) y[v] = o[i][2 * hb + e] * r;
+            }
+    }
+    if (w.active == 1) return;
+    if (tid < w.nh) {
+        mine[tid * (p.vdim + 2) + p.vdim] = s_max[tid];
+        mine[tid * (p.vdim + 2) + p.vdim + 1] = s_sum[tid];
+    }
+    merge_splits<HB>(p, part, count, group, splits, w.active, w.h0, w.nh, gate, &s_s[0][0], dst);
 }
 
 // query heads of a CTA of the step
 int heads_block(const LbAttention& p) {
     const int per = p.heads / p.kv_heads;
+    if (p.mma) return kMmaHeads;
     return per >= 8 ? 8 : per > 2 ? 4 : per;
 }
 int groups_of(const LbAttention& p) { return p.kv_heads * lb_ceil_div(p.heads / p.kv_heads, heads_block(p)); }
@@ -336,7 +608,16 @@ int step_heads(loom_b200_ctx* ctx, const LbAttention& p, int tokens, int kchunks
     return launch_step<WT, 8>(ctx, p, tokens, kchunks, part, count, out, ldo);
 }
 
+template <int NK, int NG>
+int launch_mma(loom_b200_ctx* ctx, const LbAttention& p, int tokens, int kchunks, float* part, unsigned* count, float* out, int ldo) {
+    const int splits = lb_attention_splits(ctx, p, tokens);
+    LB_LAUNCH(ctx, (lb_attention_step_mma_kernel<NK, NG>), dim3(splits, groups_of(p), tokens), dim3(kStepThreads), 0, p, kchunks, splits, part, count, out, ldo);
+    return 0;
+}
+
 }  // namespace
+
+bool lb_attention_step_mma(int dim, int vdim, int dtype) { return dtype == LOOM_B200_DTYPE_BF16 && dim <= 256 && vdim <= 256; }
 
 int lb_attention_kchunks(int dim, int dtype) { return lb_round_up(lb_ceil_div(dim, dtype == LOOM_B200_DTYPE_BF16 ? 8 : 4), 2); }
 
@@ -375,6 +656,11 @@ size_t lb_attention_counters(const LbAttention& p, int tokens) { return (size_t)
 int lb_attention_step(loom_b200_ctx* ctx, int dtype, const LbAttention& p, int tokens, float* part, unsigned* count, float* out, int ldo) {
     const int kch = lb_attention_kchunks(p.dim, dtype);
     LB_REQUIRE(ctx, tokens > 0 && tokens <= 65535, "attention: %d tokens", tokens);
+    if (p.mma) {
+        const bool k4 = p.dim <= 128, v2 = p.vdim <= 128;
+        if (k4) return v2 ? launch_mma<4, 2>(ctx, p, tokens, kch, part, count, out, ldo) : launch_mma<4, 4>(ctx, p, tokens, kch, part, count, out, ldo);
+        return v2 ? launch_mma<8, 2>(ctx, p, tokens, kch, part, count, out, ldo) : launch_mma<8, 4>(ctx, p, tokens, kch, part, count, out, ldo);
+    }
     return dtype == LOOM_B200_DTYPE_BF16 ? step_heads<__nv_bfloat16>(ctx, p, tokens, kch, part, count, out, ldo) : step_heads<float>(ctx, p, tokens, kch, part, count, out, ldo);
 }
 

@@ -110,6 +110,7 @@ LbAttention attention_of(const LbStack* st, const LbLayer& l, const float* proj,
     p.vt_lane = l.vt_lane;
     p.ring = l.ring;
     p.slices = lb_slices_of(l.ring, st->d.dtype);
+    p.mma = lb_attention_step_mma(s.dim, s.vdim, st->d.dtype);
     return p;
 }
 

@@ -314,6 +314,19 @@ def test_unequal_sequences_together_and_alone(ctx, dtype):
 
 
 @both
+@pytest.mark.parametrize("heads,kv,dim,vdim", [(17, 1, 24, 16), (40, 2, 16, 8), (2, 2, 1, 1), (3, 1, 130, 129), (2, 1, 264, 20), (2, 2, 20, 270), (8, 4, 256, 200)])
+def test_head_counts_and_sizes(ctx, heads, kv, dim, vdim, dtype):
+    """Groups of more heads than a CTA takes, heads too large for the tensor-core kernels, and tiny ones."""
+    cfg = dk.config(40, 60, [dk.attention(heads, kv, dim, vdim, 90, 30, dim ** -0.5, None)])
+    m = Model(ctx, cfg, 23, dtype, max_seq=220)
+    tok = dk.tokens_of(cfg, 200, 11)
+    want, _ = m.oracle(tok)
+    for got in (m.whole(tok), m.cut(tok, [85, 3, 1, 1, 70, 1])):
+        assert close(dtype, got, want)
+    m.close()
+
+
+@both
 def test_sequences_far_enough_apart_to_split_their_keys(ctx, dtype):
     """Steps whose sequences see many tiles, one, and none but their own token."""
     cfg = dk.config(48, 60, [dk.attention(8, 2, 24, 40, 1000, 200, 0.5, None), dk.attention(3, 3, 16, 16, 90, 40, 0.5, None)])
