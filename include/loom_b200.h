@@ -434,13 +434,13 @@ typedef struct loom_b200_layer_spec {
     int experts, top;
     double limit;          /* clamp of the gated unit */
     int kv_heads;          /* attention, delta rule: heads of k (and of v in attention, of q in the delta rule); divides heads */
-    int chunk;             /* attention: position i sees j <= i with i / chunk == j / chunk; 0: every j <= i */
+    int chunk;             /* attention: length of the stretches, counted from the first position, that attend within themselves; 0: the whole past */
     int buckets;           /* attention: rows of the distance bias, 0 for none */
     double bias_max;       /* attention: distance from which on the last bucket is used */
-    int qk_norm;           /* attention: q and k divided by their root mean square, per head */
-    int sink;              /* attention: one added to the softmax's denominator (a score of 0 without a value) */
+    int qk_norm;           /* attention: RMS norm of every q and k head, no weights */
+    int sink;              /* attention: a key of score 0 and value 0 in every softmax */
     int head_gate;         /* attention: every head's output times the sigmoid of one projected number */
-    int conv;              /* delta rule: taps of the convolutions (the last belongs to the current token) */
+    int conv;              /* delta rule: taps of the convolutions, newest last */
     double gate_cap;       /* matrix memory: gates pass cap * tanh(z / cap) */
 } loom_b200_layer_spec;
 
